@@ -11,7 +11,8 @@
 // Visible to the query at position p: the keys j <= p with p - j < window or j < keep_first (window 0:
 // every j <= p).  The tiles a block visits are those that hold kept first keys, then those of the
 // window of its rows.  A sink per head joins the denominator.  The result goes out in float32 (for a
-// kernel that combines several maps) or in bfloat16 times a gate per (token, head).
+// kernel that combines several maps) or in bfloat16 times a gate per (token, head) or per element (the sigmoid of a
+// column's sums).
 #include "common.cuh"
 
 #if !defined(WICK_DK) || !defined(WICK_DV)
@@ -87,6 +88,9 @@ struct Params {
     bf16* out_bf16;                // [n, heads, DV], or null
     const float* gate;             // [n, gate_heads] or null: a factor of the bfloat16 result (head hv -> column hv)
     const float* sink;             // [heads] or null
+    const float* gate_parts;       // float32 partial sums [gate_splits, n, gate_cols] or null: sigmoid of column gate_col + hv DV + j is a
+    int64_t gate_stride;           //   factor of element j of head hv's bfloat16 result
+    int gate_splits, gate_cols, gate_col;
     const int *cu_seqlens, *start, *page_table;
     int n_seqs, table_width, n_tiles, heads, window, keep_first;
     float scale;
@@ -279,6 +283,19 @@ attn_flex_kernel(const Params P) {
         } else {
             if (P.gate) inv *= P.gate[t * P.heads + head];
             bf16* op = P.out_bf16 + (t * P.heads + head) * DV + col;
+            if (P.gate_parts) {
+                const float* gp = P.gate_parts + t * P.gate_cols + P.gate_col + head * DV + col;
+#pragma unroll
+                for (int d = 0; d < ND; ++d) {
+                    float z0 = gp[d * 8], z1 = gp[d * 8 + 1];
+                    for (int s = 1; s < P.gate_splits; ++s) {
+                        z0 += gp[s * P.gate_stride + d * 8];
+                        z1 += gp[s * P.gate_stride + d * 8 + 1];
+                    }
+                    o[d][2 * half] *= 1.0f / (1.0f + expf(-z0));
+                    o[d][2 * half + 1] *= 1.0f / (1.0f + expf(-z1));
+                }
+            }
 #pragma unroll
             for (int d = 0; d < ND; ++d) *reinterpret_cast<uint32_t*>(op + d * 8) = pack_bf16(o[d][2 * half] * inv, o[d][2 * half + 1] * inv);
         }
@@ -328,7 +345,8 @@ WICK_API int wick_attn_flex_sizes(int* dk, int* dv) {
 //   address, tile_elems, const_off, hdiv, hmul, hmod, hmul2, row_stride, len, paged.
 WICK_API int wick_attn_flex_bf16(const void* q, const int64_t* src, void* out_f32, void* out_bf16, const float* gate, const float* sink,
                                  const int* cu_seqlens, int n_seqs, const int* start, const int* page_table, int table_width,
-                                 int n_tiles, int heads, int window, int keep_first, float scale, void* s) {
+                                 int n_tiles, int heads, int window, int keep_first, float scale, const float* gate_parts, int gate_splits,
+                                 int64_t gate_stride, int gate_cols, int gate_col, void* s) {
     using namespace flex;
     Params P;
     P.q = (const bf16*)q;
@@ -355,6 +373,8 @@ WICK_API int wick_attn_flex_bf16(const void* q, const int64_t* src, void* out_f3
     P.out_bf16 = (bf16*)out_bf16;
     P.gate = gate;
     P.sink = sink;
+    WICK_REQUIRE(!gate_parts || (out_bf16 && gate_splits >= 1 && gate_col >= 0 && gate_col + heads * DV <= gate_cols), "attn_flex: bad gate columns");
+    P.gate_parts = gate_parts; P.gate_stride = gate_stride; P.gate_splits = gate_splits; P.gate_cols = gate_cols; P.gate_col = gate_col;
     P.cu_seqlens = cu_seqlens; P.start = start; P.page_table = page_table;
     P.n_seqs = n_seqs; P.table_width = table_width; P.n_tiles = n_tiles; P.heads = heads; P.window = window; P.keep_first = keep_first;
     P.scale = scale;

@@ -516,11 +516,12 @@ attn_multi_merge_kernel(const float* __restrict__ partial, TO* __restrict__ out,
 // One block per token.  The row [query latent (qr) | latent (r) | key part (dr) | gates (Hg)] is summed
 // into shared memory; the two RMS norms follow (a block sum each); then the normed query latent goes out
 // in the activation type, the normed latent and the turned key part go to the position's row of the
-// cache ([page][64][r + dr]), and sigmoid(gate) goes out in float32.
+// cache ([page][64][r + dr]), and sigmoid(gate) goes out in float32.  A row of the sums has `cols` numbers; what lies
+// behind the gates of the heads is somebody else's.
 //   pairing 0: (2i, 2i + 1) turn together; 1: (i, i + dr / 2).
 template <typename T>
 __global__ void __launch_bounds__(256)
-latent_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, int qr, int r, int dr, int Hg,
+latent_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, int cols, int qr, int r, int dr, int Hg,
                      const float* __restrict__ q_w, const float* __restrict__ kv_w, float eps,
                      const float* __restrict__ cos_t, const float* __restrict__ sin_t, int pairing, T* __restrict__ cq_out,
                      float* __restrict__ gate_out, T* __restrict__ rows, T* __restrict__ flat_c, T* __restrict__ flat_kr,
@@ -536,8 +537,8 @@ latent_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_
     const int t = blockIdx.x, tid = threadIdx.x;
     const int W = qr + r + dr + Hg;
     for (int j = tid; j < W; j += blockDim.x) {
-        float v = parts[(int64_t)t * W + j];
-        for (int s = 1; s < splits; ++s) v += parts[s * split_stride + (int64_t)t * W + j];
+        float v = parts[(int64_t)t * cols + j];
+        for (int s = 1; s < splits; ++s) v += parts[s * split_stride + (int64_t)t * cols + j];
         row[j] = v;
     }
     __syncthreads();
@@ -692,16 +693,20 @@ latent_absorb_kernel(const float* __restrict__ parts, int splits, int64_t split_
 
 // One block per (TT tokens, head).  The head's weighted sums of latent rows (r numbers a token) wait in
 // shared memory; a warp makes one output element for all TT tokens at a time: row x of the head's e x r
-// block of Wuv, read once (lane l its elements l, l + 32, ...; the 32 sums by the butterfly), times the gate.
+// block of Wuv, read once (lane l its elements l, l + 32, ...; the 32 sums by the butterfly), times the gate: a number
+// per head (`gate`), or a number per element, the sigmoid of the sum of `gate_parts` at the element's column.  Lane tt ends
+// token tt's element.
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_expand_kernel(const float* __restrict__ y, const T* __restrict__ uv, const float* __restrict__ gate, int n, int H,
-                     int e, int r, T* __restrict__ out) {
+                     int e, int r, T* __restrict__ out, const float* __restrict__ gate_parts, int gate_splits, int64_t gate_stride,
+                     int gate_cols, int gate_col) {
     extern __shared__ __align__(16) float ys[];   // [r][TT]: a number of all TT tokens side by side
     pdl_trigger();
     pdl_wait();
     y = fresh(y);
     gate = fresh(gate);
+    gate_parts = fresh(gate_parts);
     const int t0 = blockIdx.x * LAT_TT, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
     const int n_t = min(LAT_TT, n - t0);
     for (int idx = tid; idx < LAT_TT * r; idx += blockDim.x) {
@@ -711,6 +716,15 @@ latent_expand_kernel(const float* __restrict__ y, const T* __restrict__ uv, cons
     __syncthreads();
     for (int x = blockIdx.z * n_warps + warp; x < e; x += gridDim.z * n_warps) {             // (the blocks along z share the rows)
         const T* w = uv + ((int64_t)h * e + x) * r;
+        float gt = 1.f;
+        if (lane < n_t) {
+            if (gate) gt = gate[(int64_t)(t0 + lane) * H + h];
+            if (gate_parts) {
+                float z = 0.f;
+                for (int s = 0; s < gate_splits; ++s) z += gate_parts[s * gate_stride + (int64_t)(t0 + lane) * gate_cols + gate_col + h * e + x];
+                gt = 1.0f / (1.0f + expf(-z));
+            }
+        }
         float acc[LAT_TT];
 #pragma unroll
         for (int tt = 0; tt < LAT_TT; ++tt) acc[tt] = 0.f;
@@ -723,14 +737,11 @@ latent_expand_kernel(const float* __restrict__ y, const T* __restrict__ uv, cons
         }
 #pragma unroll
         for (int tt = 0; tt < LAT_TT; ++tt) acc[tt] = warp_sum(acc[tt]);
-        if (lane == 0) {
+        float mine = acc[0];
 #pragma unroll
-            for (int tt = 0; tt < LAT_TT; ++tt)
-                if (tt < n_t) {
-                    const float gt = gate ? gate[(int64_t)(t0 + tt) * H + h] : 1.f;
-                    st(out + ((int64_t)(t0 + tt) * H + h) * e + x, acc[tt] * gt);
-                }
-        }
+        for (int tt = 1; tt < LAT_TT; ++tt)
+            if (lane == tt) mine = acc[tt];
+        if (lane < n_t) st(out + ((int64_t)(t0 + lane) * H + h) * e + x, mine * gt);
     }
 }
 
@@ -823,7 +834,7 @@ int attn_multi(const void* q, const void* store, void* out, float* partial, cons
 }
 
 template <typename T>
-int latent_finish(const float* parts, int splits, int n, int qr, int r, int dr, int Hg, const float* q_w, const float* kv_w,
+int latent_finish(const float* parts, int splits, int n, int cols, int qr, int r, int dr, int Hg, const float* q_w, const float* kv_w,
                   float eps, const float* cos_t, const float* sin_t, int pairing, void* cq_out, float* gate_out, void* rows,
                   void* flat_c, void* flat_kr, const int* page_table, int table_width, const int* seq_of_token, const int* positions,
                   cudaStream_t s) {
@@ -833,8 +844,9 @@ int latent_finish(const float* parts, int splits, int n, int qr, int r, int dr, 
     if (n == 0) return 0;
     const int W = qr + r + dr + Hg;
     const size_t smem = (size_t)W * sizeof(float);
+    WICK_REQUIRE(W <= cols, "latent_finish: rows of %d numbers, %d expected", cols, W);
     WICK_REQUIRE(smem <= 48 * 1024, "latent_finish: a row of %d numbers is beyond one block's shared memory", W);
-    WICK_CUDA(launch(latent_finish_kernel<T>, dim3(n), dim3(256), smem, s, parts, splits, (int64_t)n * W, qr, r, dr, Hg, q_w, kv_w, eps,
+    WICK_CUDA(launch(latent_finish_kernel<T>, dim3(n), dim3(256), smem, s, parts, splits, (int64_t)n * cols, cols, qr, r, dr, Hg, q_w, kv_w, eps,
                      cos_t, sin_t, pairing, (T*)cq_out, gate_out, (T*)rows, (T*)flat_c, (T*)flat_kr, page_table, table_width, seq_of_token,
                      positions));
     return check_launch("latent_finish");
@@ -864,13 +876,15 @@ int latent_query(const float* parts, int splits, int n, int H, int d, int dr, co
 }
 
 template <typename T>
-int latent_expand(const float* y, const void* uv, const float* gate, int n, int H, int e, int r, void* out, cudaStream_t s) {
+int latent_expand(const float* y, const void* uv, const float* gate, int n, int H, int e, int r, void* out, const float* gate_parts,
+                  int gate_splits, int64_t gate_stride, int gate_cols, int gate_col, cudaStream_t s) {
     WICK_REQUIRE(H > 0 && e > 0 && r > 0 && H <= 65535, "latent_expand: bad sizes");
+    WICK_REQUIRE(!gate_parts || (gate_splits >= 1 && gate_col >= 0 && gate_col + H * e <= gate_cols), "latent_expand: bad gate columns");
     if (n == 0) return 0;
     const size_t smem = (size_t)LAT_TT * r * sizeof(float);
     WICK_REQUIRE(smem <= 48 * 1024, "latent_expand: a latent of %d numbers is beyond one block's shared memory", r);
     WICK_CUDA(launch(latent_expand_kernel<T>, dim3(ceil_div(n, LAT_TT), H, min(64, ceil_div(e, 32))), dim3(256), smem, s, y, (const T*)uv, gate,
-                     n, H, e, r, (T*)out));
+                     n, H, e, r, (T*)out, gate_parts, gate_splits, gate_stride, gate_cols, gate_col));
     return check_launch("latent_expand");
 }
 
@@ -897,12 +911,12 @@ WICK_ATTN_MULTI(wick_attn_multi1_bf16, bf16, float, float, 1)
 WICK_ATTN_MULTI(wick_attn_multi1_f32, float, float, float, 1)
 
 #define WICK_LATENT(T, SUFFIX)                                                                                                   \
-    WICK_API int wick_latent_finish_##SUFFIX(const float* parts, int splits, int n, int qr, int r, int dr, int Hg,              \
+    WICK_API int wick_latent_finish_##SUFFIX(const float* parts, int splits, int n, int cols, int qr, int r, int dr, int Hg,  \
                                              const float* q_w, const float* kv_w, float eps, const float* cos_t,                \
                                              const float* sin_t, int pairing, void* cq_out, float* gate_out, void* rows,        \
                                              void* flat_c, void* flat_kr, const int* page_table, int table_width,               \
                                              const int* seq_of_token, const int* positions, void* s) {                          \
-        return latent_finish<T>(parts, splits, n, qr, r, dr, Hg, q_w, kv_w, eps, cos_t, sin_t, pairing, cq_out, gate_out, rows,  \
+        return latent_finish<T>(parts, splits, n, cols, qr, r, dr, Hg, q_w, kv_w, eps, cos_t, sin_t, pairing, cq_out, gate_out, rows,  \
                                 flat_c, flat_kr, page_table, table_width, seq_of_token, positions, (cudaStream_t)s);             \
     }                                                                                                                            \
     WICK_API int wick_latent_absorb_##SUFFIX(const float* parts, int splits, const void* uk, int n, int H, int d, int dr, int r, \
@@ -914,8 +928,10 @@ WICK_ATTN_MULTI(wick_attn_multi1_f32, float, float, float, 1)
         return latent_query<T>(parts, splits, n, H, d, dr, cos_t, sin_t, pairing, out, (cudaStream_t)s);                         \
     }                                                                                                                            \
     WICK_API int wick_latent_expand_##SUFFIX(const float* y, const void* uv, const float* gate, int n, int H, int e, int r,     \
-                                             void* out, void* s) {                                                              \
-        return latent_expand<T>(y, uv, gate, n, H, e, r, out, (cudaStream_t)s);                                                  \
+                                             void* out, const float* gate_parts, int gate_splits, int64_t gate_stride,          \
+                                             int gate_cols, int gate_col, void* s) {                                            \
+        return latent_expand<T>(y, uv, gate, n, H, e, r, out, gate_parts, gate_splits, gate_stride, gate_cols, gate_col,        \
+                                (cudaStream_t)s);                                                                                \
     }
 WICK_LATENT(bf16, bf16)
 WICK_LATENT(float, f32)

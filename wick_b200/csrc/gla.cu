@@ -1,4 +1,4 @@
-// Gated linear attention: a recurrence per head whose state is a matrix of key channels by value elements, with a decay
+// Linear attention with a decay per key channel: a recurrence per head whose state is a matrix of key channels by value elements, with a decay
 // per key channel and token, for steps of any shape over per-sequence state records.
 //
 // The input projection's float32 partial sums hold, per token, [q: H dk | k: H dk | v: H dv | g: H dv | low: r]
@@ -9,6 +9,9 @@
 //   scan    : S_t = diag(a_t) S_(t-1) + k_t v_t^T  (dk x dv per head);  o_t = S_t^T q_t
 //   out     : every head's o is divided by its root mean square over dv (eps inside the root) and multiplied by a weight
 //             of dv numbers that the heads share, then by silu(g); the result goes out in the activation type
+//
+// A second preparation (hgrn2) makes the same rows from [q: H dk | z: H dk | v: H dv]: q <- silu(q), with a learned lower
+// bound l per channel a = l + (1 - l) sigmoid(z + b) and k = 1 - a = (1 - l) sigmoid(-(z + b)); scan and norm follow (no gate).
 //
 // A sequence's record (float32) is the state as [H][dv][dk] (a column of S, the dk numbers that meet one element of v,
 // lies together).  Everything here is float32 arithmetic; a token's numbers depend on its own sequence alone.  A step of
@@ -134,6 +137,56 @@ gla_prepare_kernel(const float* __restrict__ parts, int splits, int64_t split_st
         const float sp = -z > 20.0f ? -z : log1pf(expf(-z));
         o[2 * HK + c] = expf(-sp * inv_tau);
     }
+}
+
+// grid (tokens, ceil(items / 256)), an item VEC neighbours: first the H dk key channels, then the H dv value elements.
+template <int VEC, bool ONE>
+__global__ void __launch_bounds__(256)
+hgrn2_prepare_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, int HK, int HV, const float* __restrict__ bias,
+                     const float* __restrict__ lower, float* __restrict__ out) {
+    pdl_trigger();
+    pdl_wait();
+    parts = fresh(parts);
+    const int64_t t = blockIdx.x;
+    const int c = ((int)blockIdx.y * (int)blockDim.x + (int)threadIdx.x) * VEC;
+    if (c >= HK + HV) return;
+    const float* row = parts + t * (2 * HK + HV);
+    float* o = out + t * (3 * HK + HV);
+    auto load = [&](int at, float (&v)[VEC]) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+        for (int s = 0; s < (ONE ? 1 : splits); ++s) {
+            const float* p = row + s * split_stride + at;
+            if (VEC == 4) {
+                const float4 d = *reinterpret_cast<const float4*>(p);
+                v[0] += d.x; v[VEC > 1 ? 1 : 0] += d.y; v[VEC > 2 ? 2 : 0] += d.z; v[VEC > 3 ? 3 : 0] += d.w;
+            } else {
+                v[0] += *p;
+            }
+        }
+    };
+    auto store = [&](int at, const float (&v)[VEC]) {
+        if (VEC == 4) *reinterpret_cast<float4*>(o + at) = make_float4(v[0], v[VEC > 1 ? 1 : 0], v[VEC > 2 ? 2 : 0], v[VEC > 3 ? 3 : 0]);
+        else o[at] = v[0];
+    };
+    float q[VEC], z[VEC], a[VEC], k[VEC];
+    if (c >= HK) {                                                       // (VEC divides HK)
+        load(HK + c, q);
+        store(2 * HK + c, q);
+        return;
+    }
+    load(c, q);
+    load(HK + c, z);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+        const float l = lower[c + i], x = z[i] + bias[c + i];
+        q[i] = q[i] / (1.0f + expf(-q[i]));
+        a[i] = l + (1.0f - l) / (1.0f + expf(-x));
+        k[i] = (1.0f - l) / (1.0f + expf(x));
+    }
+    store(c, q);
+    store(HK + c, k);
+    store(2 * HK + c, a);
 }
 
 // The sums of four columns over the LN threads that share them (see the state-space scan: the same exchange).
@@ -400,7 +453,8 @@ gla_chunk_join_kernel(float* __restrict__ chunk_state, const float* __restrict__
     *rec = S;
 }
 
-// grid (tokens, groups of heads), a warp per head: o / sqrt(mean(o^2) + eps) * w * silu(g), g from the projection's sums.
+// grid (tokens, groups of heads), a warp per head: o / sqrt(mean(o^2) + eps) * w * silu(g), g from the projection's sums (no
+// gate where there are none).
 template <typename T, bool ONE>
 __global__ void __launch_bounds__(256)
 gla_norm_gate_kernel(const float* __restrict__ y, const float* __restrict__ parts, int splits, int64_t split_stride, int cols,
@@ -417,9 +471,13 @@ gla_norm_gate_kernel(const float* __restrict__ y, const float* __restrict__ part
         ss = warp_sum(ss);
         const float f = 1.0f / sqrtf(ss / (float)P + eps);
         for (int j = lane; j < P; j += 32) {
-            const int64_t at = (int64_t)t * cols + g_col + h * P + j;
-            const float g = ONE ? parts[at] : gla_sum_parts(parts, splits, split_stride, at);
-            st(out + ((int64_t)t * H + h) * P + j, (row[j] * f) * w[j] * (g / (1.0f + expf(-g))));
+            float v = (row[j] * f) * w[j];
+            if (parts) {
+                const int64_t at = (int64_t)t * cols + g_col + h * P + j;
+                const float g = ONE ? parts[at] : gla_sum_parts(parts, splits, split_stride, at);
+                v *= g / (1.0f + expf(-g));
+            }
+            st(out + ((int64_t)t * H + h) * P + j, v);
         }
     }
 }
@@ -453,45 +511,10 @@ int gla_launch(const GlaArgs& a, int chunks, size_t smem, cudaStream_t s) {
     return gla_launch_mode<LN, 2>(a, chunks, smem, s);
 }
 
-}  // namespace wick
-
-using namespace wick;
-typedef __nv_bfloat16 bf16;
-
-// parts: float32 [splits, n, cols] laid out [q | k | v | g | low]; w2: float32 [H dk, rank]; b2: float32 [H dk] or null;
-// state: float32 [slots, H dv dk]; qkav: float32 [n, 3 H dk + H dv] and y: float32 [n, H dv], both written here.
-// max_q: the most tokens a sequence can bring (0: unknown).  chunks > 0: the sequences' tokens are scanned in chunks of
-// `chunk` tokens side by side; `chunks` is at least the number of chunks (n / chunk + n_seqs is enough), chunk_state float32
-// [chunks, H dv dk] and chunk_decay float32 [chunks, H dk] are scratch.
-WICK_API int wick_gla_mix(const float* parts, int splits, int n, int cols, int H, int dk, int dv, int rank, const float* w2,
-                          const float* b2, float q_scale, float tau, float* state, int64_t record, const int* slots, int n_seqs,
-                          const int* cu_seqlens, float* qkav, float* y, int max_q, int chunk, int chunks, float* chunk_state,
-                          float* chunk_decay, void* stream) {
-    cudaStream_t s = (cudaStream_t)stream;
-    WICK_REQUIRE(H > 0 && dk > 0 && dv > 0 && rank > 0 && tau > 0.f, "gla_mix: bad sizes");
-    WICK_REQUIRE(dk <= 32 * GLA_ROWS, "gla_mix: heads of %d key channels (up to %d are built)", dk, 32 * GLA_ROWS);
-    const int HK = H * dk, HV = H * dv, channels = 3 * HK + HV;
-    WICK_REQUIRE(cols == 2 * HK + 2 * HV + rank, "gla_mix: rows of %d numbers, %d expected", cols, 2 * HK + 2 * HV + rank);
-    WICK_REQUIRE(record == (int64_t)HV * dk, "gla_mix: records of another size");
-    WICK_REQUIRE(splits >= 1, "gla_mix: partial sums are needed");
-    WICK_REQUIRE(chunks == 0 || (chunk > 0 && chunk_state && chunk_decay && (int64_t)chunks >= n / chunk + n_seqs),
-                 "gla_mix: the chunked scan needs room for %d chunks", chunk > 0 ? n / chunk + n_seqs : 0);
-    WICK_REQUIRE((size_t)rank * 4 <= 48 * 1024, "gla_mix: a rank of %d is beyond one block's shared memory", rank);
-    if (n == 0 || n_seqs == 0) return 0;
-    const int64_t stride = (int64_t)n * cols;
-    // (long steps: eight tokens a block share a thread's row of W2; short ones: a block a token, for more blocks)
-    const int prep_tiles = ceil_div(HK, GLA_PREP_THREADS) + ceil_div(HV, GLA_PREP_THREADS);
-    const int pb = (n >= 512 && (size_t)rank * 8 * 4 <= 16 * 1024) ? 8 : 1;
-    size_t prep_smem = (size_t)pb * rank * 4;
-    const size_t staged = (size_t)GLA_PREP_THREADS * (rank | 1) * 4;
-    const int stage = prep_smem + staged <= 48 * 1024 ? 1 : 0;          // (else a thread reads its row of W2 from memory)
-    if (stage) prep_smem += staged;
-    auto prepare = pb == 8 ? (splits == 1 ? gla_prepare_kernel<8, true> : gla_prepare_kernel<8, false>)
-                           : (splits == 1 ? gla_prepare_kernel<1, true> : gla_prepare_kernel<1, false>);
-    WICK_CUDA(launch(prepare, dim3(ceil_div(n, pb), prep_tiles), dim3(GLA_PREP_THREADS), prep_smem, s, parts, splits, stride, cols, HK, HV,
-                     rank, w2, b2, q_scale, 1.0f / tau, qkav, n, stage));
-    if (check_launch("gla_prepare")) return 1;
-    const int N = dk, P = dv;
+// The scan of prepared rows, by whichever form the step's shape asks for.
+int gla_scan(float* qkav, int H, int dk, int dv, float* state, int64_t record, const int* slots, int n_seqs, const int* cu_seqlens,
+             float* y, int max_q, int chunk, int chunks, float* chunk_state, float* chunk_decay, cudaStream_t s) {
+    const int N = dk, P = dv, channels = 3 * H * dk + H * dv;
     int ln = 1;
     while (ln < 32 && (N + ln - 1) / ln > GLA_ROWS) ln *= 2;
     if (ln < 4 && N >= 16) ln = 4;                                       // (a thread keeps a few numbers, not a whole column)
@@ -517,11 +540,75 @@ WICK_API int wick_gla_mix(const float* parts, int splits, int n, int cols, int H
     }
 }
 
-// y: float32 [n, H dv]; parts as above (g from column g_col on); w: float32 [dv]; out: [n, H dv].
+}  // namespace wick
+
+using namespace wick;
+typedef __nv_bfloat16 bf16;
+
+// What both mixers' scans ask of their sizes.
+#define WICK_GLA_CHECKS(NAME)                                                                                                  \
+    WICK_REQUIRE(dk <= 32 * GLA_ROWS, NAME ": heads of %d key channels (up to %d are built)", dk, 32 * GLA_ROWS);               \
+    WICK_REQUIRE(record == (int64_t)H * dv * dk, NAME ": records of another size");                                            \
+    WICK_REQUIRE(splits >= 1, NAME ": partial sums are needed");                                                                \
+    WICK_REQUIRE(chunks == 0 || (chunk > 0 && chunk_state && chunk_decay && (int64_t)chunks >= n / chunk + n_seqs),            \
+                 NAME ": the chunked scan needs room for %d chunks", chunk > 0 ? n / chunk + n_seqs : 0)
+
+// parts: float32 [splits, n, cols] laid out [q | k | v | g | low]; w2: float32 [H dk, rank]; b2: float32 [H dk] or null;
+// state: float32 [slots, H dv dk]; qkav: float32 [n, 3 H dk + H dv] and y: float32 [n, H dv], both written here.
+// max_q: the most tokens a sequence can bring (0: unknown).  chunks > 0: the sequences' tokens are scanned in chunks of
+// `chunk` tokens side by side; `chunks` is at least the number of chunks (n / chunk + n_seqs is enough), chunk_state float32
+// [chunks, H dv dk] and chunk_decay float32 [chunks, H dk] are scratch.
+WICK_API int wick_gla_mix(const float* parts, int splits, int n, int cols, int H, int dk, int dv, int rank, const float* w2,
+                          const float* b2, float q_scale, float tau, float* state, int64_t record, const int* slots, int n_seqs,
+                          const int* cu_seqlens, float* qkav, float* y, int max_q, int chunk, int chunks, float* chunk_state,
+                          float* chunk_decay, void* stream) {
+    cudaStream_t s = (cudaStream_t)stream;
+    WICK_REQUIRE(H > 0 && dk > 0 && dv > 0 && rank > 0 && tau > 0.f, "gla_mix: bad sizes");
+    WICK_GLA_CHECKS("gla_mix");
+    const int HK = H * dk, HV = H * dv;
+    WICK_REQUIRE(cols == 2 * HK + 2 * HV + rank, "gla_mix: rows of %d numbers, %d expected", cols, 2 * HK + 2 * HV + rank);
+    WICK_REQUIRE((size_t)rank * 4 <= 48 * 1024, "gla_mix: a rank of %d is beyond one block's shared memory", rank);
+    if (n == 0 || n_seqs == 0) return 0;
+    const int64_t stride = (int64_t)n * cols;
+    // (long steps: eight tokens a block share a thread's row of W2; short ones: a block a token, for more blocks)
+    const int prep_tiles = ceil_div(HK, GLA_PREP_THREADS) + ceil_div(HV, GLA_PREP_THREADS);
+    const int pb = (n >= 512 && (size_t)rank * 8 * 4 <= 16 * 1024) ? 8 : 1;
+    size_t prep_smem = (size_t)pb * rank * 4;
+    const size_t staged = (size_t)GLA_PREP_THREADS * (rank | 1) * 4;
+    const int stage = prep_smem + staged <= 48 * 1024 ? 1 : 0;          // (else a thread reads its row of W2 from memory)
+    if (stage) prep_smem += staged;
+    auto prepare = pb == 8 ? (splits == 1 ? gla_prepare_kernel<8, true> : gla_prepare_kernel<8, false>)
+                           : (splits == 1 ? gla_prepare_kernel<1, true> : gla_prepare_kernel<1, false>);
+    WICK_CUDA(launch(prepare, dim3(ceil_div(n, pb), prep_tiles), dim3(GLA_PREP_THREADS), prep_smem, s, parts, splits, stride, cols, HK, HV,
+                     rank, w2, b2, q_scale, 1.0f / tau, qkav, n, stage));
+    if (check_launch("gla_prepare")) return 1;
+    return gla_scan(qkav, H, dk, dv, state, record, slots, n_seqs, cu_seqlens, y, max_q, chunk, chunks, chunk_state, chunk_decay, s);
+}
+
+// parts: float32 [splits, n, 2 H dk + H dv] laid out [q | z | v]; bias, lower: float32 [H dk]; the rest as above.
+WICK_API int wick_hgrn2_mix(const float* parts, int splits, int n, int H, int dk, int dv, const float* bias, const float* lower,
+                            float* state, int64_t record, const int* slots, int n_seqs, const int* cu_seqlens, float* qkav, float* y,
+                            int max_q, int chunk, int chunks, float* chunk_state, float* chunk_decay, void* stream) {
+    cudaStream_t s = (cudaStream_t)stream;
+    WICK_REQUIRE(H > 0 && dk > 0 && dv > 0, "hgrn2_mix: bad sizes");
+    WICK_GLA_CHECKS("hgrn2_mix");
+    if (n == 0 || n_seqs == 0) return 0;
+    const int HK = H * dk, HV = H * dv;
+    const int64_t stride = (int64_t)n * (2 * HK + HV);
+    const bool vec = ((HK | HV) & 3) == 0 && (((uintptr_t)parts | (uintptr_t)qkav) & 15) == 0;
+    auto prepare = vec ? (splits == 1 ? hgrn2_prepare_kernel<4, true> : hgrn2_prepare_kernel<4, false>)
+                       : (splits == 1 ? hgrn2_prepare_kernel<1, true> : hgrn2_prepare_kernel<1, false>);
+    WICK_CUDA(launch(prepare, dim3(n, ceil_div(HK + HV, vec ? 1024 : 256)), dim3(256), 0, s, parts, splits, stride, HK, HV, bias, lower,
+                     qkav));
+    if (check_launch("hgrn2_prepare")) return 1;
+    return gla_scan(qkav, H, dk, dv, state, record, slots, n_seqs, cu_seqlens, y, max_q, chunk, chunks, chunk_state, chunk_decay, s);
+}
+
+// y: float32 [n, H dv]; parts as above (g from column g_col on) or null (no gate); w: float32 [dv]; out: [n, H dv].
 #define WICK_GLA_NORM_GATE(NAME, T)                                                                                            \
     WICK_API int NAME(const float* y, const float* parts, int splits, int n, int cols, int g_col, int H, int dv, const float* w, \
                       float eps, void* out, void* s) {                                                                         \
-        WICK_REQUIRE(H > 0 && dv > 0 && g_col >= 0 && g_col + H * dv <= cols, "gla_norm_gate: bad sizes");                     \
+        WICK_REQUIRE(H > 0 && dv > 0 && (!parts || (g_col >= 0 && g_col + H * dv <= cols)), "gla_norm_gate: bad sizes");       \
         if (n == 0) return 0;                                                                                                  \
         const int warps = H >= 4 ? 4 : H;                                                                                      \
         auto kernel = splits == 1 ? gla_norm_gate_kernel<T, true> : gla_norm_gate_kernel<T, false>;                            \

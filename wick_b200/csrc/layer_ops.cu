@@ -11,6 +11,8 @@
 //                rms(.) * g (times a factor per element), optionally followed by the
 //                norm y = tanh(a x) * w + b or by a copy of x in the activation type
 //   gate rows :  g = gelu_tanh(z) * e, e a slice of the token's row in a table
+//   poly norm :  a r(z) + b r(z^2) + c r(z^3) + e, r(v) = v / sqrt(mean(v^2) + eps)
+//   pairs     :  an embedding row times a factor plus a row chosen by the token and the one before it
 #include "common.cuh"
 
 namespace wick {
@@ -288,6 +290,99 @@ embed_sinusoid_kernel(const T* __restrict__ table, const int* __restrict__ token
     }
 }
 
+// ---- an embedding with a factor and a row per pair of tokens -------------------------------------------------------
+// out[t] = table[token_t] * scale + pairs[r], r = (before * mul_prev + token_t * mul_cur) mod buckets, or the last row (number
+// `buckets`) at position 0.  `before` is the step's token before this one where that is the same sequence's, else the one an
+// earlier step left in `history` (int32 [page][64]); every token also leaves itself there.  (A step reads what earlier steps
+// wrote and writes its own positions: no position is read and written in one step.)  One block per token.
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_pairs_kernel(const T* __restrict__ table, const T* __restrict__ pairs, const int* __restrict__ tokens,
+                   const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ cu_seqlens,
+                   const int* __restrict__ page_table, int table_width, int* history, int64_t buckets, int64_t mul_prev,
+                   int64_t mul_cur, float scale, float* __restrict__ out, int width) {
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x, tok = tokens[t], pos = positions[t], b = seq_of_token[t];
+    const int* pages = page_table + (int64_t)b * table_width;
+    int64_t r = buckets;
+    if (pos > 0) {
+        const int before = t > cu_seqlens[b] ? tokens[t - 1] : history[(int64_t)pages[(pos - 1) / kPage] * kPage + (pos - 1) % kPage];
+        r = ((int64_t)before * mul_prev + (int64_t)tok * mul_cur) % buckets;
+    }
+    if (threadIdx.x == 0) history[(int64_t)pages[pos / kPage] * kPage + pos % kPage] = tok;
+    const T* row = table + (int64_t)tok * width;
+    const T* add = pairs + r * width;
+    for (int j = threadIdx.x; j < width; j += blockDim.x) out[(int64_t)t * width + j] = fmaf(ld(row + j), scale, ld(add + j));
+}
+
+// ---- PolyNorm ------------------------------------------------------------------------------------------------------
+// One block per row of ff numbers z (the partial sums in index order): the means of z^2, z^4 and z^6, then
+// a r(z) + b r(z^2) + c r(z^3) + e out in the activation type.  The row waits in shared memory between the two passes (keep) or
+// is added up again.  The block's size depends on ff alone.
+template <typename TOut, bool VEC>
+__global__ void __launch_bounds__(1024)
+poly_norm_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, const float* __restrict__ coef, float eps,
+                 TOut* __restrict__ out, int ff, int keep) {
+    extern __shared__ float smem[];
+    __shared__ float red[3][33];
+    float* row = smem;
+    pdl_trigger();
+    const float ca = coef[0], cb = coef[1], cc = coef[2], ce = coef[3];      // (weights: no kernel writes them)
+    pdl_wait();
+    parts = fresh(parts);
+    const int64_t at = (int64_t)blockIdx.x * ff;
+    constexpr int V = VEC ? 4 : 1;
+    auto load = [&](int j, float (&z)[V]) {
+        if (VEC) {
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            add_partials4(v, parts, splits, split_stride, at + j);
+            z[0] = v.x; z[V > 1 ? 1 : 0] = v.y; z[V > 2 ? 2 : 0] = v.z; z[V > 3 ? 3 : 0] = v.w;
+        } else {
+            float v = 0.f;
+            for (int s = 0; s < splits; ++s) v += parts[s * split_stride + at + j];
+            z[0] = v;
+        }
+    };
+    float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+    for (int j = threadIdx.x * V; j < ff; j += blockDim.x * V) {
+        float z[V];
+        load(j, z);
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+            if (keep) row[j + i] = z[i];
+            const float q = z[i] * z[i];
+            s2 += q;
+            s4 = fmaf(q, q, s4);
+            s6 = fmaf(q * q, q, s6);
+        }
+    }
+    // the three sums over the block in one go: warps' sums, then every warp adds those up
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    s2 = warp_sum(s2); s4 = warp_sum(s4); s6 = warp_sum(s6);
+    if (lane == 0) {
+        red[0][warp] = s2; red[1][warp] = s4; red[2][warp] = s6;
+    }
+    __syncthreads();
+    s2 = warp_sum(lane < nw ? red[0][lane] : 0.f);
+    s4 = warp_sum(lane < nw ? red[1][lane] : 0.f);
+    s6 = warp_sum(lane < nw ? red[2][lane] : 0.f);
+    const float inv = 1.0f / (float)ff;
+    const float fa = ca / sqrtf(fmaf(s2, inv, eps)), fb = cb / sqrtf(fmaf(s4, inv, eps)), fc = cc / sqrtf(fmaf(s6, inv, eps));
+    TOut* o = out + at;
+    for (int j = threadIdx.x * V; j < ff; j += blockDim.x * V) {
+        float z[V];
+        if (keep) {                                                       // (a thread reads back what it wrote itself)
+#pragma unroll
+            for (int i = 0; i < V; ++i) z[i] = row[j + i];
+        } else {
+            load(j, z);
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) st(o + j + i, fmaf(z[i], fmaf(z[i], fmaf(z[i], fc, fb), fa), ce));
+    }
+}
+
 // x[t][j] += (x0 ? x0[t][j] : 0) + (vec ? vec[j] : 0): what a pass over a range of layers begins with.
 __global__ void stream_offset_kernel(float* __restrict__ x, const float* __restrict__ x0, const float* __restrict__ vec, int64_t n,
                                      int width) {
@@ -380,6 +475,27 @@ int scaled_add_rmsnorm(float* x, const float* delta, int splits, float alpha, co
     WICK_CUDA(launch(scaled_add_rmsnorm_kernel<TOut>, dim3(n), dim3(threads), smem, s, x, delta, splits, (int64_t)n * width, alpha,
                      w, eps, (TOut*)out, n, width));
     return check_launch("scaled_add_rmsnorm");
+}
+
+template <typename TOut, bool VEC>
+int poly_norm_launch(const float* parts, int splits, const float* coef, float eps, void* out, int n, int ff, cudaStream_t s) {
+    size_t smem = (size_t)((ff + 3) & ~3) * sizeof(float);
+    const int keep = smem <= 100 * 1024;                                 // (two blocks of that size share an SM; longer rows are added up twice)
+    if (!keep) smem = 0;
+    static bool raised = false;
+    if (smem > 48 * 1024 && !raised) {
+        WICK_CUDA(cudaFuncSetAttribute(poly_norm_kernel<TOut, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024));
+        raised = true;
+    }
+    const int threads = min(1024, max(64, ((ff + 3) / 4 + 31) / 32 * 32));
+    WICK_CUDA(launch(poly_norm_kernel<TOut, VEC>, dim3(n), dim3(threads), smem, s, parts, splits, (int64_t)n * ff, coef, eps, (TOut*)out, ff,
+                     keep));
+    return check_launch("poly_norm");
+}
+template <typename TOut>
+int poly_norm(const float* parts, int splits, const float* coef, float eps, void* out, int n, int ff, cudaStream_t s) {
+    if ((ff & 3) == 0 && ((uintptr_t)parts & 15) == 0) return poly_norm_launch<TOut, true>(parts, splits, coef, eps, out, n, ff, s);
+    return poly_norm_launch<TOut, false>(parts, splits, coef, eps, out, n, ff, s);
 }
 
 }  // namespace wick
@@ -499,6 +615,31 @@ WICK_CONCAT_ACTIVATION(wick_concat_activation_f32, float)
     }
 WICK_EMBED_SINUSOID(wick_embed_sinusoid_bf16, bf16)
 WICK_EMBED_SINUSOID(wick_embed_sinusoid_f32, float)
+
+// history: int32 [pages][64]; pairs: [buckets + 1, width] in the table's type.
+#define WICK_EMBED_PAIRS(NAME, T)                                                                                            \
+    WICK_API int NAME(const void* table, const void* pairs, const int* tokens, const int* positions, const int* seq_of_token, \
+                      const int* cu_seqlens, const int* page_table, int table_width, int* history, int64_t buckets,          \
+                      int64_t mul_prev, int64_t mul_cur, float scale, float* out, int n, int width, void* s) {               \
+        WICK_REQUIRE(n >= 0 && width > 0 && buckets > 0 && mul_prev >= 0 && mul_cur >= 0, "embed_pairs: bad sizes");          \
+        if (n == 0) return 0;                                                                                                \
+        WICK_CUDA(launch(embed_pairs_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)s, (const T*)table, (const T*)pairs, tokens, \
+                         positions, seq_of_token, cu_seqlens, page_table, table_width, history, buckets, mul_prev, mul_cur,  \
+                         scale, out, width));                                                                                \
+        return check_launch("embed_pairs");                                                                                  \
+    }
+WICK_EMBED_PAIRS(wick_embed_pairs_bf16, bf16)
+WICK_EMBED_PAIRS(wick_embed_pairs_f32, float)
+
+// parts: float32 [splits, n, ff]; coef: float32 [4]; out: [n, ff].
+#define WICK_POLY_NORM(NAME, T)                                                                                              \
+    WICK_API int NAME(const float* parts, int splits, const float* coef, float eps, void* out, int n, int ff, void* s) {     \
+        WICK_REQUIRE(splits >= 1 && ff > 0, "poly_norm: bad sizes");                                                         \
+        if (n == 0) return 0;                                                                                                \
+        return poly_norm<T>(parts, splits, coef, eps, out, n, ff, (cudaStream_t)s);                                          \
+    }
+WICK_POLY_NORM(wick_poly_norm_bf16, bf16)
+WICK_POLY_NORM(wick_poly_norm_f32, float)
 
 // x: float32 [n, width], changed in place; x0: float32 [n, width] or null; vec: float32 [width] or null.
 WICK_API int wick_stream_offset(float* x, const float* x0, const float* vec, int n, int width, void* s) {

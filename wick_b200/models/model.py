@@ -104,10 +104,13 @@ class Model:
     # ---- sizes -------------------------------------------------------------
     def cache_needs(self) -> List[Optional[CacheNeed]]:
         """For each schedule entry, the cache storage it owns (None if it reads
-        another entry's or its mixer keeps nothing)."""
+        another entry's or its mixer keeps nothing); one more at the end for an
+        embedding that keeps something."""
         needs: List[Optional[CacheNeed]] = []
         for e in self.spec.schedule:
             needs.append(None if e.read_cache_of is not None else self.blocks[e.layer].mixer.cache_need())
+        if self.embedding.cache_need() is not None:
+            needs.append(self.embedding.cache_need())
         return needs
 
     def weight_bytes_per_step(self) -> int:
@@ -137,7 +140,9 @@ class Model:
         (float32 [tokens, width], everything added)."""
         if not self.loaded:
             raise RuntimeError("the model has no weights yet")
-        if getattr(self.embedding, "NEEDS_POSITIONS", False):
+        if self.embedding.cache_need() is not None:
+            h = Hidden(self.embedding.forward_step(batch, cache.view(len(self.spec.schedule), batch)))
+        elif getattr(self.embedding, "NEEDS_POSITIONS", False):
             h = Hidden(self.embedding.forward(batch.tokens, batch.positions))
         else:
             h = Hidden(self.embedding.forward(batch.tokens))

@@ -723,15 +723,15 @@ def latent_finish(parts: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, 
                   q_weight: torch.Tensor, kv_weight: Optional[torch.Tensor], eps: float, cos: Optional[torch.Tensor],
                   sin: Optional[torch.Tensor], pairing: str = "neighbours", rows: Optional[torch.Tensor],
                   page_table: torch.Tensor, seq_of_token: torch.Tensor, positions: torch.Tensor, flat: bool = False):
-    """From the float32 partial sums ``parts`` [splits, n, q_rank + kv_rank + rot_dim + gate_heads] of a latent
-    attention's down-projections: the query latent rms(.) * q_weight -> [n, q_rank] in ``dtype``; the latent
+    """From the float32 partial sums ``parts`` [splits, n, q_rank + kv_rank + rot_dim + gate_heads (+ more)] of a latent
+    attention's down-projections (columns behind these, a gate per element's, are left alone): the query latent rms(.) * q_weight -> [n, q_rank] in ``dtype``; the latent
     rms(.) * kv_weight and the key part, turned by the angles of ``cos`` / ``sin`` [n, rot_dim / 2], -> the token's
     row of ``rows`` (pages of [64][kv_rank + rot_dim]; None: nothing is stored); sigmoid of the gates -> float32
     [n, gate_heads] (None if there are none).  Returns (query latent, gates); with ``flat`` (and ``rows``) also the step's
     own latents [n, kv_rank] and key parts [n, rot_dim] as arrays of their own, in ``dtype``."""
     _cuda("parts", parts, torch.float32)
     W = q_rank + kv_rank + rot_dim + gate_heads
-    _need(parts.dim() == 3 and parts.shape[2] == W, f"parts must be [splits, n, {W}], is {tuple(parts.shape)}")
+    _need(parts.dim() == 3 and parts.shape[2] >= W, f"parts must be [splits, n, {W} or more], is {tuple(parts.shape)}")
     n = parts.shape[1]
     _cuda("q_weight", q_weight, torch.float32, (q_rank,))
     if kv_weight is not None:
@@ -752,7 +752,7 @@ def latent_finish(parts: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int, 
     if flat and rows is not None:
         flat_c = torch.empty((n, kv_rank), dtype=dtype, device=parts.device)
         flat_kr = torch.empty((n, rot_dim), dtype=dtype, device=parts.device)
-    _layer().call(f"wick_latent_finish_{_dt(cq)}", "piiiiiippfppippppppippp", _p(parts), parts.shape[0], n, q_rank, kv_rank, rot_dim,
+    _layer().call(f"wick_latent_finish_{_dt(cq)}", "piiiiiiippfppippppppippp", _p(parts), parts.shape[0], n, parts.shape[2], q_rank, kv_rank, rot_dim,
                   gate_heads, _p(q_weight), _p(kv_weight), float(eps), _p(cos) if use_rot else None, _p(sin) if use_rot else None,
                   PAIRINGS[pairing], _p(cq), _p(gate), _p(rows), _p(flat_c), _p(flat_kr), _p(page_table), page_table.shape[-1],
                   _p(seq_of_token), _p(positions), _stream())
@@ -777,6 +777,17 @@ def latent_query(q_parts: torch.Tensor, heads: int, d: int, rot_dim: int, *, cos
     _layer().call(f"wick_latent_query_{_dt(out)}", "piiiiippipp", _p(q_parts), q_parts.shape[0], n, heads, d, rot_dim,
                   _p(cos) if use_rot else None, _p(sin) if use_rot else None, PAIRINGS[pairing], _p(out), _stream())
     return out
+
+
+def _gate_parts(gate_parts: Optional[Tuple[torch.Tensor, int]], n: int, width: int):
+    """(partial sums or None, splits, columns, first column) of a gate with a number per element."""
+    if gate_parts is None:
+        return None, 0, 0, 0
+    parts, first = gate_parts
+    _cuda("gate_parts", parts, torch.float32)
+    _need(parts.dim() == 3 and parts.shape[1] == n and 0 <= first and first + width <= parts.shape[2],
+          f"gate_parts must be [splits, {n}, {first + width} or more], is {tuple(parts.shape)}")
+    return parts, parts.shape[0], parts.shape[2], int(first)
 
 
 # ---- prompt attention on the tensor cores with keys and values described by strides ---------------------------------
@@ -805,11 +816,13 @@ def flex_source(t: Optional[torch.Tensor] = None, *, tile_elems: int = 0, const_
 
 def attention_flex(q: torch.Tensor, k0: List[int], k1: List[int], v: List[int], batch, scale: float, *, dv: int, window: int = 0,
                    keep_first: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                   out_dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
+                   gate_parts: Optional[Tuple[torch.Tensor, int]] = None, out_dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
     """Attention of a prompt's tokens on the tensor cores.  q: bfloat16 [n, heads, dk]; a key row is ``k0``'s numbers
     followed by ``k1``'s (sources as :func:`flex_source` makes them; flat sources need sequences that start at position
     0), a value row ``v``'s.  Visible to the query at position p: the keys j <= p with p - j < window or j < keep_first
-    (window 0: every j <= p).  ``sink`` float32 [heads]; ``gate`` float32 [n, heads], a factor of the bfloat16 result.
+    (window 0: every j <= p).  ``sink`` float32 [heads]; ``gate`` float32 [n, heads], a factor of the bfloat16 result;
+    ``gate_parts`` = (float32 partial sums [splits, n, cols], first column): the bfloat16 result is multiplied element by
+    element by the sigmoid of the heads * dv columns' sums.
     Returns [n, heads, dv] in ``out_dtype`` (float32 or bfloat16)."""
     import numpy as np
     _cuda("q", q, torch.bfloat16)
@@ -821,12 +834,14 @@ def attention_flex(q: torch.Tensor, k0: List[int], k1: List[int], v: List[int], 
     if gate is not None:
         _cuda("gate", gate, torch.float32, (n, heads))
         _need(out_dtype == torch.bfloat16, "the gate is a factor of the bfloat16 result")
+    gp, g_splits, g_cols, g_col = _gate_parts(gate_parts, n, heads * dv)
+    _need(gp is None or (gate is None and out_dtype == torch.bfloat16), "one gate, a factor of the bfloat16 result")
     out = torch.empty((n, heads, dv), dtype=out_dtype, device=q.device)
     src = np.asarray(k0 + k1 + v, dtype=np.int64)
-    _flex(dk, dv).call("wick_attn_flex_bf16", "pppppppippiiiiifp", _p(q), src.ctypes.data, _p(out) if out_dtype == torch.float32 else None,
+    _flex(dk, dv).call("wick_attn_flex_bf16", "pppppppippiiiiifpiliip", _p(q), src.ctypes.data, _p(out) if out_dtype == torch.float32 else None,
                        _p(out) if out_dtype == torch.bfloat16 else None, _p(gate), _p(sink), _p(batch.cu_seqlens), batch.n_seqs,
                        _p(batch.start), _p(batch.page_table), batch.table_width, attention_tiles(batch), heads, int(window),
-                       int(keep_first), float(scale), _stream())
+                       int(keep_first), float(scale), _p(gp), g_splits, n * g_cols, g_cols, g_col, _stream())
     return out
 
 
@@ -863,8 +878,9 @@ def latent_absorb(q_parts: torch.Tensor, uk: torch.Tensor, heads: int, d: int, r
 
 
 def latent_expand(y: torch.Tensor, uv: torch.Tensor, gate: Optional[torch.Tensor], heads: int, v_dim: int, kv_rank: int, *,
-                  dtype: torch.dtype) -> torch.Tensor:
-    """out[t, h] = gate[t, h] * Wuv_h y[t, h].  y: float32 [n, heads, kv_rank] (a head's weighted sum of cached
+                  dtype: torch.dtype, gate_parts: Optional[Tuple[torch.Tensor, int]] = None) -> torch.Tensor:
+    """out[t, h] = gate[t, h] * Wuv_h y[t, h], or, with ``gate_parts`` = (float32 partial sums [splits, n, cols], first column),
+    element by element times the sigmoid of the heads * v_dim columns' sums.  y: float32 [n, heads, kv_rank] (a head's weighted sum of cached
     latents); ``uv``: [heads * v_dim, kv_rank] in ``dtype``; gate: float32 [n, heads] or None.  Returns [n, heads * v_dim]."""
     _cuda("y", y, torch.float32)
     n = y.shape[0]
@@ -872,8 +888,11 @@ def latent_expand(y: torch.Tensor, uv: torch.Tensor, gate: Optional[torch.Tensor
     _cuda("uv", uv, dtype, (heads * v_dim, kv_rank))
     if gate is not None:
         _cuda("gate", gate, torch.float32, (n, heads))
+    gp, g_splits, g_cols, g_col = _gate_parts(gate_parts, n, heads * v_dim)
+    _need(gp is None or gate is None, "one gate")
     out = torch.empty((n, heads * v_dim), dtype=dtype, device=y.device)
-    _layer().call(f"wick_latent_expand_{_dt(out)}", "pppiiiipp", _p(y), _p(uv), _p(gate), n, heads, v_dim, kv_rank, _p(out), _stream())
+    _layer().call(f"wick_latent_expand_{_dt(out)}", "pppiiiippiliip", _p(y), _p(uv), _p(gate), n, heads, v_dim, kv_rank, _p(out), _p(gp),
+                  g_splits, n * g_cols, g_cols, g_col, _stream())
     return out
 
 
@@ -1241,14 +1260,7 @@ def gla_mix(parts: torch.Tensor, *, heads: int, key_dim: int, v_dim: int, w2: to
     _cuda("records", records, torch.float32)
     _need(records.dim() == 2 and records.shape[1] == hv * key_dim, f"records must be [slots, {hv * key_dim}], are {tuple(records.shape)}")
     _need(n == batch.n_tokens, f"{n} rows, the batch has {batch.n_tokens} tokens")
-    qkav = torch.empty((n, 3 * hk + hv), dtype=torch.float32, device=parts.device)
-    y = torch.empty((n, hv), dtype=torch.float32, device=parts.device)
-    max_q = 1 if batch.is_decode else 0          # (0: unknown to the host, as in a captured prompt step)
-    chunk, chunks, chunk_state, chunk_decay = GLA_CHUNK, 0, None, None
-    if not batch.is_decode and n >= GLA_CHUNKED_FROM:
-        chunks = n // chunk + batch.n_seqs
-        chunk_state = torch.empty((chunks, hv * key_dim), dtype=torch.float32, device=parts.device)
-        chunk_decay = torch.empty((chunks, hk), dtype=torch.float32, device=parts.device)
+    qkav, y, max_q, chunk, chunks, chunk_state, chunk_decay = _gla_scratch(n, hk, hv, key_dim, batch, parts.device)
     _layer().call("wick_gla_mix", "piiiiiiippffplpipppiiippp", _p(parts), splits, n, cols, heads, key_dim, v_dim, rank, _p(w2), _p(b2),
                   float(q_scale), float(tau), _p(records), hv * key_dim, _p(batch.slots), batch.n_seqs, _p(batch.cu_seqlens),
                   _p(qkav), _p(y), max_q, chunk, chunks, _p(chunk_state), _p(chunk_decay), _stream(),
@@ -1256,19 +1268,57 @@ def gla_mix(parts: torch.Tensor, *, heads: int, key_dim: int, v_dim: int, w2: to
     return y
 
 
-def gla_norm_gate(y: torch.Tensor, parts: torch.Tensor, g_col: int, heads: int, v_dim: int, weight: torch.Tensor, eps: float,
+def hgrn2_mix(parts: torch.Tensor, *, heads: int, key_dim: int, v_dim: int, bias: torch.Tensor, lower: torch.Tensor,
+              records: torch.Tensor, batch) -> torch.Tensor:
+    """The same recurrence with a forget factor that also says how much is written.  ``parts``: the input projection's float32
+    partial sums [splits, n, 2 H dk + H dv], a row laid out [q: H dk | z: H dk | v: H dv].  q <- silu(q);
+    f = lower + (1 - lower) sigmoid(z + bias) per key channel (``bias``, ``lower`` float32 [H dk]); per head
+    S <- diag(f) S + (1 - f) v^T and o = S^T q.  ``records`` as for :func:`gla_mix`.  Returns o float32 [n, H dv]."""
+    _cuda("parts", parts, torch.float32)
+    hk, hv = heads * key_dim, heads * v_dim
+    _need(parts.dim() == 3 and parts.shape[2] == 2 * hk + hv, f"parts must be [splits, n, {2 * hk + hv}], are {tuple(parts.shape)}")
+    splits, n, cols = parts.shape
+    _cuda("bias", bias, torch.float32, (hk,))
+    _cuda("lower", lower, torch.float32, (hk,))
+    _cuda("records", records, torch.float32)
+    _need(records.dim() == 2 and records.shape[1] == hv * key_dim, f"records must be [slots, {hv * key_dim}], are {tuple(records.shape)}")
+    _need(n == batch.n_tokens, f"{n} rows, the batch has {batch.n_tokens} tokens")
+    qkav, y, max_q, chunk, chunks, chunk_state, chunk_decay = _gla_scratch(n, hk, hv, key_dim, batch, parts.device)
+    _layer().call("wick_hgrn2_mix", "piiiiippplpipppiiippp", _p(parts), splits, n, heads, key_dim, v_dim, _p(bias), _p(lower),
+                  _p(records), hv * key_dim, _p(batch.slots), batch.n_seqs, _p(batch.cu_seqlens), _p(qkav), _p(y), max_q, chunk,
+                  chunks, _p(chunk_state), _p(chunk_decay), _stream(), kernels=1 + (3 if chunks else 1))
+    return y
+
+
+def _gla_scratch(n: int, hk: int, hv: int, key_dim: int, batch, device):
+    """What a linear attention's kernels write on the way: the tokens' rows [q | k | a | v], o, and (steps of many tokens) the
+    chunks' states and decays."""
+    qkav = torch.empty((n, 3 * hk + hv), dtype=torch.float32, device=device)
+    y = torch.empty((n, hv), dtype=torch.float32, device=device)
+    max_q = 1 if batch.is_decode else 0          # (0: unknown to the host, as in a captured prompt step)
+    chunk, chunks, chunk_state, chunk_decay = GLA_CHUNK, 0, None, None
+    if not batch.is_decode and n >= GLA_CHUNKED_FROM:
+        chunks = n // chunk + batch.n_seqs
+        chunk_state = torch.empty((chunks, hv * key_dim), dtype=torch.float32, device=device)
+        chunk_decay = torch.empty((chunks, hk), dtype=torch.float32, device=device)
+    return qkav, y, max_q, chunk, chunks, chunk_state, chunk_decay
+
+
+def gla_norm_gate(y: torch.Tensor, parts: Optional[torch.Tensor], g_col: int, heads: int, v_dim: int, weight: torch.Tensor, eps: float,
                   dtype: torch.dtype) -> torch.Tensor:
     """Every head's ``v_dim`` numbers of y (float32 [n, H dv]) divided by their root mean square and multiplied by ``weight``
     (float32 [dv], shared by the heads), then by silu(g), g the columns from ``g_col`` on of the float32 partial sums
-    ``parts`` [splits, n, cols]; [n, H dv] in ``dtype``."""
+    ``parts`` [splits, n, cols] (``parts`` None: no gate); [n, H dv] in ``dtype``."""
     _cuda("y", y, torch.float32)
-    _cuda("parts", parts, torch.float32)
     n = y.shape[0]
     _need(tuple(y.shape) == (n, heads * v_dim), f"y must be [n, {heads * v_dim}]")
-    _need(parts.dim() == 3 and parts.shape[1] == n and parts.shape[2] >= g_col + heads * v_dim, "parts must hold the gate's columns")
+    if parts is not None:
+        _cuda("parts", parts, torch.float32)
+        _need(parts.dim() == 3 and parts.shape[1] == n and parts.shape[2] >= g_col + heads * v_dim, "parts must hold the gate's columns")
     _cuda("weight", weight, torch.float32, (v_dim,))
     out = torch.empty((n, heads * v_dim), dtype=dtype, device=y.device)
-    _layer().call(f"wick_gla_norm_gate_{_dt(out)}", "ppiiiiiipfpp", _p(y), _p(parts), parts.shape[0], n, parts.shape[2], int(g_col), heads,
+    _layer().call(f"wick_gla_norm_gate_{_dt(out)}", "ppiiiiiipfpp", _p(y), _p(parts), 1 if parts is None else parts.shape[0], n,
+                  0 if parts is None else parts.shape[2], int(g_col), heads,
                   v_dim, _p(weight), float(eps), _p(out), _stream())
     return out
 
@@ -1286,6 +1336,37 @@ def embed_sinusoid(table: torch.Tensor, tokens: torch.Tensor, positions: torch.T
     out = torch.empty((n, width), dtype=torch.float32, device=table.device)
     _layer().call(f"wick_embed_sinusoid_{_dt(table)}", "ppppfpiip", _p(table), _p(tokens), _p(positions), _p(freq), float(scale), _p(out),
                   n, width, _stream())
+    return out
+
+
+def embed_pairs(table: torch.Tensor, pairs: torch.Tensor, batch, history: torch.Tensor, scale: float, mul_prev: int, mul_cur: int
+                ) -> torch.Tensor:
+    """float32 [n, width]: rows of ``table`` at the step's tokens times ``scale``, plus row (before * mul_prev + token * mul_cur)
+    mod (rows - 1) of ``pairs`` (the last row for a token at position 0), ``before`` the sequence's token at the position before.
+    ``history``: int32 pages of 64 positions, the sequences' tokens; the step's own are written to it."""
+    _cuda("table", table)
+    _cuda("pairs", pairs, table.dtype)
+    width = table.shape[1]
+    _need(pairs.dim() == 2 and pairs.shape[1] == width and pairs.shape[0] >= 2, f"pairs must be [buckets + 1, {width}], is {tuple(pairs.shape)}")
+    _cuda("history", history, torch.int32)
+    _need(history[0].numel() == PAGE, f"history must hold pages of {PAGE} tokens, is {tuple(history.shape)}")
+    n = batch.n_tokens
+    out = torch.empty((n, width), dtype=torch.float32, device=table.device)
+    _layer().call(f"wick_embed_pairs_{_dt(table)}", "pppppppiplllfpiip", _p(table), _p(pairs), _p(batch.tokens), _p(batch.positions),
+                  _p(batch.seq_of_token), _p(batch.cu_seqlens), _p(batch.page_table), batch.table_width, _p(history),
+                  pairs.shape[0] - 1, int(mul_prev), int(mul_cur), float(scale), _p(out), n, width, _stream())
+    return out
+
+
+def poly_norm(parts: torch.Tensor, coefficients: torch.Tensor, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """a r(z) + b r(z^2) + c r(z^3) + e in ``dtype`` [n, ff]: z the sum (in index order) of the float32 partial sums ``parts``
+    [splits, n, ff], powers element by element, r(v) = v / sqrt(mean(v^2) + eps) over a row; ``coefficients`` float32 [4]."""
+    _cuda("parts", parts, torch.float32)
+    _need(parts.dim() == 3, "the product comes as partial sums [splits, n, ff]")
+    _cuda("coefficients", coefficients, torch.float32, (4,))
+    splits, n, ff = parts.shape
+    out = torch.empty((n, ff), dtype=dtype, device=parts.device)
+    _layer().call(f"wick_poly_norm_{_dt(out)}", "pipfpiip", _p(parts), splits, _p(coefficients), float(eps), _p(out), n, ff, _stream())
     return out
 
 

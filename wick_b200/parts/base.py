@@ -294,6 +294,15 @@ class Embedding(Part):
         """int32 [n] -> float32 [n, width]."""
         raise NotImplementedError
 
+    def cache_need(self) -> Optional[CacheNeed]:
+        """What an embedding that reads more than the token itself keeps in the cache; its
+        :meth:`forward_step` is then called instead of :meth:`forward`."""
+        return None
+
+    def forward_step(self, batch: "Any", cache: "Any") -> torch.Tensor:
+        """The step's tokens -> float32 [n, width], with the view of the embedding's own cache storage."""
+        raise NotImplementedError
+
 
 class Head(Part):
     category = "head"

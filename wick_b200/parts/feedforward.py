@@ -5,14 +5,19 @@ category       kind                    params
 =============  ======================  ==========================================
 ffn            ``none``                — (a layer without a feed-forward)
 ffn            ``mlp``                 width, intermediate, activation
-                                       (``relu2``: the square of relu),
-                                       names (up, down -> local names)
+                                       (``relu2``: the square of relu;
+                                       ``poly_norm``: see below, with eps),
+                                       names (up, down, coefficients -> local
+                                       names)
 ffn            ``table_moe``           width, vocab, experts, top, intermediate,
                                        shared (PartSpec of a feed-forward that
                                        runs for every token, or None),
                                        names (expert: a pattern with ``{i}``,
                                        gate, up, down, table, shared: a prefix)
 =============  ======================  ==========================================
+
+``poly_norm``, with four learned numbers a, b, c, e: a r(z) + b r(z^2) + c r(z^3) + e, the powers
+element by element and r(v) = v / sqrt(mean(v^2) + eps) over a token's inner numbers, evaluated in float32.
 
 ``table_moe``: a mixture of gated experts without a router.  An integer table
 [vocab, top] names, for every token id, the ``top`` different experts that its tokens
@@ -49,32 +54,44 @@ class MLP(FeedForward):
         super().__init__(params, ctx)
         self.width, self.intermediate = int(params["width"]), int(params["intermediate"])
         self.activation = str(params.get("activation", "relu2"))
-        if self.activation != "relu2":
-            raise ValueError(f"unsupported activation {self.activation} (relu2)")
-        names = dict(up="up_proj.weight", down="down_proj.weight")
+        if self.activation not in ("relu2", "poly_norm"):
+            raise ValueError(f"unsupported activation {self.activation} (relu2, poly_norm)")
+        self.eps = float(params["eps"]) if self.activation == "poly_norm" else 0.0
+        self.coefficients: Optional[torch.Tensor] = None        # poly_norm: the four numbers, float32
+        names = dict(up="up_proj.weight", down="down_proj.weight", coefficients="act.weight")
         names.update(params.get("names") or {})
         self.names = names
         self.up = Linear(self.intermediate, self.width, ctx)
         self.down = Linear(self.width, self.intermediate, ctx)
 
     def tensor_specs(self):
-        return [TensorSpec(self.names["up"], (self.intermediate, self.width)),
-                TensorSpec(self.names["down"], (self.width, self.intermediate))]
+        specs = [TensorSpec(self.names["up"], (self.intermediate, self.width)),
+                 TensorSpec(self.names["down"], (self.width, self.intermediate))]
+        if self.activation == "poly_norm":
+            specs.append(TensorSpec(self.names["coefficients"], (4,), "vector"))
+        return specs
 
     def load(self, fetch):
         self.up.load_rows([fetch(self.names["up"])])
         self.down.load_rows([fetch(self.names["down"])])
+        if self.activation == "poly_norm":
+            self.coefficients = self.ctx.hold(fetch(self.names["coefficients"]), "vector")
 
     def tensor(self, name):
         if name == self.names["up"]:
             return self.up.rows(0, self.intermediate)
+        if self.coefficients is not None and name == self.names["coefficients"]:
+            return self.coefficients
         return self.down.rows(0, self.width) if name == self.names["down"] else None
 
     def weight_bytes(self):
         return self.up.weight_bytes() + self.down.weight_bytes()
 
     def forward(self, x, batch):
-        a = ops.relu_squared_(self.up.forward(x, self.ctx.dtype))
+        if self.activation == "poly_norm":
+            a = ops.poly_norm(self.up.forward_delta(x), self.coefficients, self.eps, self.ctx.dtype)
+        else:
+            a = ops.relu_squared_(self.up.forward(x, self.ctx.dtype))
         return self.down.forward_delta(a)
 
 

@@ -8,7 +8,9 @@ mixer          ``latent_attention``    width, heads, head_dim (unrotated query /
                                        ones), v_dim, q_rank, kv_rank, scale, eps,
                                        position (PartSpec ``rotary_pairs`` over
                                        rot_dim elements, or None), window (None
-                                       or positions), sink, gate, own_kv,
+                                       or positions), sink, gate (None, ``head``
+                                       or True: a number a head, ``element``: a
+                                       number an element), own_kv,
                                        names (dq, dq_norm, uq, dkv, dkv_norm, uk,
                                        uv, sink, gate, o -> local names)
 =============  ======================  ==========================================
@@ -23,7 +25,9 @@ elements, values of size e, latent of r numbers):
 * head i's key at position j is [Wuk_i c_j | rotated part_j], its value Wuv_i c_j; the
   score is (q . key) * scale over the keys with 0 <= p - j < window; the weights are
   exp(s_j) / (sum exp(s_j) + exp(sink_i));
-* the head's result is multiplied by sigmoid(Wg h)_i; Wo follows.
+* the head's result is multiplied by sigmoid(Wg h)_i, one number of the head (Wg has H rows), or
+  element by element by the head's e numbers of sigmoid(Wg h) (``element``: H e rows, read as the
+  product's float32 sums by whoever writes the heads' results); Wo follows.
 
 A layer with ``own_kv`` False has no Wdkv: it is scheduled to read the cache of an earlier
 layer, and applies its own Wuk and Wuv to that layer's rows.
@@ -67,7 +71,12 @@ class LatentAttention(Mixer):
         self.scale = float(p["scale"]) if p.get("scale") is not None else (self.head_dim + self.rot_dim) ** -0.5
         self.eps = float(p.get("eps", 0.0))
         self.window = int(p.get("window") or 0)
-        self.has_sink, self.has_gate, self.own_kv = bool(p.get("sink", False)), bool(p.get("gate", False)), bool(p.get("own_kv", True))
+        self.has_sink, self.own_kv = bool(p.get("sink", False)), bool(p.get("own_kv", True))
+        gate = p.get("gate") or None
+        self.gate = "head" if gate is True else gate
+        if self.gate not in (None, "head", "element"):
+            raise ValueError(f"the gate is None, 'head' or 'element', not {gate!r}")
+        self.gate_rows = {None: 0, "head": self.heads, "element": self.heads * self.v_dim}[self.gate]
         self.position = build_part("position", p.get("position") or PartSpec("none"), ctx)
         if not isinstance(self.position, (RotaryPairs, NoPosition)):
             raise ValueError("this mixer's kernel turns pairs (rotary_pairs) or nothing")
@@ -80,7 +89,7 @@ class LatentAttention(Mixer):
         self.names = names
         # one product for everything that reads h: [dq | dkv (own_kv) | gate (gate)]
         self.kv_rows = self.row if self.own_kv else 0
-        self.down = Linear(self.q_rank + self.kv_rows + (self.heads if self.has_gate else 0), self.width, ctx)
+        self.down = Linear(self.q_rank + self.kv_rows + self.gate_rows, self.width, ctx)
         self.uq = Linear(self.heads * (self.head_dim + self.rot_dim), self.q_rank, ctx)
         self.o = Linear(self.width, self.heads * self.v_dim, ctx)
         self.uk = self.uv = self.q_weight = self.kv_weight = self.sink = None
@@ -95,14 +104,14 @@ class LatentAttention(Mixer):
         specs += [TensorSpec(nm["uk"], (H * self.head_dim, self.kv_rank)), TensorSpec(nm["uv"], (H * self.v_dim, self.kv_rank))]
         if self.has_sink:
             specs.append(TensorSpec(nm["sink"], (H,), "vector", init="around_zero"))
-        if self.has_gate:
-            specs.append(TensorSpec(nm["gate"], (H, self.width)))
+        if self.gate_rows:
+            specs.append(TensorSpec(nm["gate"], (self.gate_rows, self.width)))
         specs.append(TensorSpec(nm["o"], (self.width, H * self.v_dim)))
         return specs
 
     def load(self, fetch):
         nm, hold = self.names, self.ctx.hold
-        rows = [fetch(nm["dq"])] + ([fetch(nm["dkv"])] if self.own_kv else []) + ([fetch(nm["gate"])] if self.has_gate else [])
+        rows = [fetch(nm["dq"])] + ([fetch(nm["dkv"])] if self.own_kv else []) + ([fetch(nm["gate"])] if self.gate_rows else [])
         self.down.load_rows(rows)
         self.uq.load_rows([fetch(nm["uq"])])
         self.o.load_rows([fetch(nm["o"])])
@@ -128,8 +137,8 @@ class LatentAttention(Mixer):
             return self.down.rows(0, a)
         if self.own_kv and name == nm["dkv"]:
             return self.down.rows(a, b)
-        if self.has_gate and name == nm["gate"]:
-            return self.down.rows(b, b + self.heads)
+        if self.gate_rows and name == nm["gate"]:
+            return self.down.rows(b, b + self.gate_rows)
         if name == nm["uq"]:
             return self.uq.rows(0, self.uq.out_features)
         return self.o.rows(0, self.width) if name == nm["o"] else None
@@ -154,15 +163,17 @@ class LatentAttention(Mixer):
         n, H = x.shape[0], self.heads
         if cache is None or getattr(cache, "rows", None) is None:
             raise RuntimeError("this layer has no cached rows to read: its schedule entry must name the entry whose cache it reads")
-        parts = self.down.forward_delta(x)                # float32 [splits, n, q_rank (+ r + dr) (+ H)]
+        parts = self.down.forward_delta(x)                # float32 [splits, n, q_rank (+ r + dr) (+ the gate's rows)]
         rot = self.position if isinstance(self.position, RotaryPairs) else None
         cos, sin = rot.tables(batch) if rot else (None, None)
+        pairing = rot.pairing if rot else "neighbours"
+        gate_parts = (parts, self.q_rank + self.kv_rows) if self.gate == "element" else None
         expand = self.expands and self._from_position_zero(batch)
         memo_key = ("latent_rows", cache.rows.data_ptr())
         writes = write_cache and self.own_kv
         res = ops.latent_finish(parts, self.q_rank, self.kv_rank if self.own_kv else 0, self.rot_dim if self.own_kv else 0,
-                                H if self.has_gate else 0, dtype=self.ctx.dtype, q_weight=self.q_weight,
-                                kv_weight=self.kv_weight, eps=self.eps, cos=cos, sin=sin,
+                                H if self.gate == "head" else 0, dtype=self.ctx.dtype, q_weight=self.q_weight,
+                                kv_weight=self.kv_weight, eps=self.eps, cos=cos, sin=sin, pairing=pairing,
                                 rows=cache.rows if writes else None, page_table=batch.page_table,
                                 seq_of_token=batch.seq_of_token, positions=batch.positions, flat=writes and self._from_position_zero(batch))
         cq, gate = res[0], res[1]
@@ -172,17 +183,18 @@ class LatentAttention(Mixer):
         if expand and memo_key in batch.memo:
             c, kr = batch.memo[memo_key]
             d, e, dr = self.head_dim, self.v_dim, self.rot_dim
-            qb = ops.latent_query(q, H, d, dr, cos=cos, sin=sin, dtype=self.ctx.dtype)
+            qb = ops.latent_query(q, H, d, dr, cos=cos, sin=sin, pairing=pairing, dtype=self.ctx.dtype)
             kv = self.ukv.forward(c, self.ctx.dtype)      # [n, H d + H e]: every head's unrotated keys, then every head's values
             k0 = ops.flex_source(kv, hmul=d, row_stride=H * (d + e), length=d)
             k1 = ops.flex_source(kr, row_stride=dr, length=dr) if dr else ops.flex_source()
             v = ops.flex_source(kv, const_off=H * d, hmul=e, row_stride=H * (d + e), length=e)
-            out = ops.attention_flex(qb, k0, k1, v, batch, self.scale, dv=e, window=self.window, sink=self.sink, gate=gate)
+            out = ops.attention_flex(qb, k0, k1, v, batch, self.scale, dv=e, window=self.window, sink=self.sink, gate=gate,
+                                     gate_parts=gate_parts)
             return self.o.forward_delta(out.view(n, H * e))
-        q_lat = ops.latent_absorb(q, self.uk, H, self.head_dim, self.rot_dim, self.kv_rank, cos=cos, sin=sin)
+        q_lat = ops.latent_absorb(q, self.uk, H, self.head_dim, self.rot_dim, self.kv_rank, cos=cos, sin=sin, pairing=pairing)
         att = ops.attention_multi(q_lat, cache.rows, batch, self.scale, maps=1, kv_heads=1, v_dim=self.kv_rank,
                                   window=self.window, sink=self.sink, rows_of=self.row, out_dtype=torch.float32)
-        out = ops.latent_expand(att, self.uv, gate, H, self.v_dim, self.kv_rank, dtype=self.ctx.dtype)
+        out = ops.latent_expand(att, self.uv, gate, H, self.v_dim, self.kv_rank, dtype=self.ctx.dtype, gate_parts=gate_parts)
         return self.o.forward_delta(out)
 
 

@@ -1,4 +1,4 @@
-"""Gated linear attention as a mixer.
+"""Linear attentions with a decay per key channel as mixers.
 
 =============  ===========================  ==========================================
 category       kind                         params
@@ -10,9 +10,13 @@ mixer          ``gated_linear_attention``   width, heads, head_dim (key channels
                                             head_dim^(-1/2)), names (q, k, v, gate, o,
                                             norm, decay_in, decay_out, decay_bias ->
                                             local names)
+mixer          ``hgrn2``                    width, heads, head_dim (key channels of a
+                                            head), v_dim, eps, names (q, forget,
+                                            forget_bias, lower, v, norm, o -> local
+                                            names)
 =============  ===========================  ==========================================
 
-With h the mixer's input, H heads of dk key channels and dv value numbers:
+``gated_linear_attention``, with h the mixer's input, H heads of dk key channels and dv value numbers:
 
 * q = Wq h * q_scale, k = Wk h (H x dk each), v = Wv h (H x dv), g = Wg h (H x dv), low = W1 h (r numbers): one matrix
   product;
@@ -21,6 +25,14 @@ With h the mixer's input, H heads of dk key channels and dv value numbers:
 * per head S <- diag(a) S + k v^T (dk x dv; the decay acts on the rows that belong to key channels), o = S^T q;
 * every head's o is divided by its root mean square over dv (eps inside the root) and multiplied by a weight of dv numbers
   that the heads share; the heads side by side are multiplied by silu(g) and go through Wo.
+
+``hgrn2``, with the same letters:
+
+* q = silu(Wq h), z = Wf h + b (H x dk each), v = Wv h (H x dv): one matrix product;
+* the forget factor of a key channel is f = l + (1 - l) sigmoid(z), l the channel's learned lower bound;
+* per head S <- diag(f) S + (1 - f) v^T, o = S^T q: the recurrence above with the decay f and 1 - f (evaluated as
+  (1 - l) sigmoid(-z)) where it has a key;
+* the per-head norm above, no gate, Wo.
 
 The state is one float32 record per sequence (kind ``state`` of the cache: zero when a sequence starts), read and brought
 up to date by every step whatever its shape.  Everything between the two matrix products is float32, W2's product
@@ -113,4 +125,65 @@ class GatedLinearAttention(Mixer):
         return self.o.forward_delta(g)
 
 
+class Hgrn2(Mixer):
+    PROMPT_CAPTURABLE = True
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        p = params
+        self.width, self.heads = int(p["width"]), int(p["heads"])
+        self.key_dim, self.v_dim, self.eps = int(p["head_dim"]), int(p["v_dim"]), float(p["eps"])
+        if self.heads <= 0 or self.key_dim <= 0 or self.v_dim <= 0:
+            raise ValueError("heads, head_dim and v_dim must be positive")
+        self.hk, self.hv = self.heads * self.key_dim, self.heads * self.v_dim
+        names = dict(q="q_proj.weight", forget="f_proj.weight", forget_bias="f_proj.bias", lower="lower_bound", v="v_proj.weight",
+                     norm="norm.weight", o="o_proj.weight")
+        names.update(p.get("names") or {})
+        self.names = names
+        self.input = Linear(2 * self.hk + self.hv, self.width, ctx)          # rows: q, forget, v
+        self.o = Linear(self.width, self.hv, ctx)
+        self.bias = self.lower = self.norm_w = None
+
+    def tensor_specs(self):
+        nm = self.names
+        return [TensorSpec(nm["q"], (self.hk, self.width)), TensorSpec(nm["forget"], (self.hk, self.width)),
+                TensorSpec(nm["forget_bias"], (self.hk,), "vector", init="decay_bias"),
+                TensorSpec(nm["lower"], (self.hk,), "vector", init="unit_interval"), TensorSpec(nm["v"], (self.hv, self.width)),
+                TensorSpec(nm["norm"], (self.v_dim,), "vector"), TensorSpec(nm["o"], (self.width, self.hv))]
+
+    def load(self, fetch):
+        nm, hold = self.names, self.ctx.hold
+        self.input.load_rows([fetch(nm["q"]), fetch(nm["forget"]), fetch(nm["v"])])
+        self.o.load_rows([fetch(nm["o"])])
+        self.bias, self.lower, self.norm_w = (hold(fetch(nm[k]), "vector") for k in ("forget_bias", "lower", "norm"))
+
+    def tensor(self, name):
+        nm, hk = self.names, self.hk
+        spans = {nm["q"]: (0, hk), nm["forget"]: (hk, 2 * hk), nm["v"]: (2 * hk, 2 * hk + self.hv)}
+        if name in spans:
+            return self.input.rows(*spans[name])
+        if name == nm["o"]:
+            return self.o.rows(0, self.width)
+        return {nm["forget_bias"]: self.bias, nm["lower"]: self.lower, nm["norm"]: self.norm_w}.get(name)
+
+    def record_floats(self) -> int:
+        return self.hv * self.key_dim
+
+    def cache_need(self):
+        return CacheNeed("state", shape=(self.record_floats(),), dtype=torch.float32)
+
+    def weight_bytes(self):
+        return self.input.weight_bytes() + self.o.weight_bytes() + 4 * (2 * self.hk + self.v_dim)
+
+    def forward(self, x, batch, cache, write_cache):
+        if not write_cache:
+            raise RuntimeError("a linear-attention mixer keeps its own record; it cannot read another entry's")
+        parts = self.input.forward_delta(x)                         # float32 [splits, n, 2 H dk + H dv]
+        y = ops.hgrn2_mix(parts, heads=self.heads, key_dim=self.key_dim, v_dim=self.v_dim, bias=self.bias, lower=self.lower,
+                          records=cache.state, batch=batch)
+        g = ops.gla_norm_gate(y, None, 0, self.heads, self.v_dim, self.norm_w, self.eps, self.ctx.dtype)
+        return self.o.forward_delta(g)
+
+
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
+register_part("mixer", "hgrn2", Hgrn2)

@@ -7,7 +7,9 @@ category       kind                    params
 =============  ======================  ==========================================
 norm           ``rms``                 width, eps, offset (added to the stored
                                        weight, default 0), tensor (its local
-                                       name, default "weight"), optional
+                                       name, default "weight"), optional,
+                                       one_number (one weight for all elements),
+                                       factor (of the weight, default 1)
 norm           ``tanh``                width, tensor, names (bias, alpha ->
                                        local names), optional
 position       ``rotary_half_split``   head_dim, theta
@@ -23,10 +25,14 @@ block          ``prenorm_residual``    width and layer_scale (mixer, ffn -> loca
                                        (mixer, ffn -> local names, eps) where
                                        they are normed before the sum
 block          ``postnorm_residual``   alpha
+block          ``normed_sum_residual`` —
 embedding      ``table``               vocab, width, tensor, scale (a factor of
                                        the rows, default 1), position (None or
                                        {"kind": "sinusoid", "base": b}: a vector
-                                       per position that is added)
+                                       per position that is added), pairs (None
+                                       or {"tensor", "buckets", "mul_prev",
+                                       "mul_cur"}: a row per pair of tokens that
+                                       is added)
 head           ``linear``              vocab, width, tied, tensor, soft_cap
 =============  ======================  ==========================================
 
@@ -56,7 +62,9 @@ from .linear import Linear
 class RMSNorm(Norm):
     """x / sqrt(mean(x^2) + eps) * (offset + w).  ``offset`` 1 is the form whose weight is
     stored as its distance from one; the sum is made once, in float32, when the weight is
-    loaded.  ``optional``: the tensor may be absent; the norm then has no weight and must
+    loaded.  ``one_number``: the stored weight is a single number, the same for all elements.
+    ``factor``: a constant the weight is multiplied by (in float32, when it is loaded).
+    ``optional``: the tensor may be absent; the norm then has no weight and must
     not be run (its owner asks :attr:`present`)."""
 
     PROMPT_CAPTURABLE = True
@@ -66,6 +74,7 @@ class RMSNorm(Norm):
         self.width = int(params["width"])
         self.eps = float(params["eps"])
         self.offset = float(params.get("offset", 0.0))
+        self.one_number, self.factor = bool(params.get("one_number", False)), float(params.get("factor", 1.0))
         self.name = str(params.get("tensor", "weight"))
         self.optional = bool(params.get("optional", False))
         self.stored: Optional[torch.Tensor] = None      # as the checkpoint has it
@@ -77,7 +86,7 @@ class RMSNorm(Norm):
 
     def tensor_specs(self):
         init = "absent" if self.optional else ("around_zero" if self.offset else "")
-        return [TensorSpec(self.name, (self.width,), "vector", optional=self.optional, init=init)]
+        return [TensorSpec(self.name, () if self.one_number else (self.width,), "vector", optional=self.optional, init=init)]
 
     def load(self, fetch):
         w = fetch(self.name)
@@ -86,6 +95,10 @@ class RMSNorm(Norm):
             return
         self.stored = self.ctx.hold(w, "vector")
         self.weight = self.stored + self.offset if self.offset else self.stored
+        if self.factor != 1.0:
+            self.weight = self.weight * self.factor
+        if self.one_number:                          # (the kernels read a weight per element)
+            self.weight = self.weight.reshape(1).expand(self.width).contiguous()
 
     def tensor(self, name):
         return self.stored if name == self.name else None
@@ -500,11 +513,42 @@ class PostNormResidual(Block):
         return h
 
 
+class NormedSumResidual(Block):
+    """x <- x + norm1(mixer(x)); x <- x + norm2(ffn(x)): the sublayers read the stream itself and
+    their results are normed before the sum (a factor of the results is the norms' own).  Norm
+    and sum are one kernel, which also makes the copy of the new stream in the compute dtype that
+    the next sublayer's matrix products read; the layer's last sum stays pending with its norm.
+    A layer whose feed-forward is of kind ``none`` ends after its mixer."""
+
+    PROMPT_CAPTURABLE = True
+
+    def __init__(self, params, ctx, mixer, mixer_norm, ffn, ffn_norm):
+        super().__init__(params, ctx, mixer, mixer_norm, ffn, ffn_norm)
+        if not isinstance(mixer_norm, RMSNorm) or not isinstance(ffn_norm, RMSNorm):
+            raise ValueError("the kernel that norms a result and adds it to the stream is an RMS norm's")
+
+    def forward(self, h, batch, cache, write_cache):
+        dt = self.ctx.dtype
+        h.resolved(dt)
+        d = self.mixer.forward(h.act, batch, cache, write_cache)
+        h.defer(as_splits(d), rms=(self.mixer_norm.weight, self.mixer_norm.eps))
+        if not getattr(self.ffn, "IS_NONE", False):
+            h.resolved(dt)
+            d = self.ffn.forward(h.act, batch)
+            h.defer(as_splits(d), rms=(self.ffn_norm.weight, self.ffn_norm.eps))
+        if self.side is not None:
+            self.side.forward(h, batch)
+        return h
+
+
 # ---------------------------------------------------------------------------
 class TableEmbedding(Embedding):
-    """x = table[token] * scale (+ the position's vector).  ``position`` of kind ``sinusoid``: element 2 i of position p's
+    """x = table[token] * scale (+ the position's vector) (+ the pair's row).  ``position`` of kind ``sinusoid``: element 2 i of position p's
     vector is sin(p base^(-2i/width)), element 2 i + 1 the cosine of the same angle; the frequencies are evaluated in
-    float64 and rounded to float32 once, the angle is their float32 product with the position."""
+    float64 and rounded to float32 once, the angle is their float32 product with the position.  ``pairs``: row
+    (before * mul_prev + token * mul_cur) mod buckets of a second table of buckets + 1 rows is added as it is, ``before`` the
+    sequence's token at the position before; a sequence's first token takes the last row.  The tokens of earlier steps are
+    kept in the cache, one integer per position."""
 
     PROMPT_CAPTURABLE = True
 
@@ -513,6 +557,13 @@ class TableEmbedding(Embedding):
         self.vocab, self.width = int(params["vocab"]), int(params["width"])
         self.name = str(params.get("tensor", "weight"))
         self.weight: Optional[torch.Tensor] = None
+        self.pairs = dict(params["pairs"]) if params.get("pairs") else None
+        self.pair_rows: Optional[torch.Tensor] = None
+        if self.pairs is not None:
+            if params.get("position") is not None:
+                raise ValueError("an embedding adds the positions' vectors or the pairs' rows, not both")
+            if int(self.pairs["buckets"]) <= 0:
+                raise ValueError("a pair table has a positive number of buckets")
         self.scale = float(params.get("scale", 1.0))
         pos = params.get("position")
         self.freq: Optional[torch.Tensor] = None
@@ -525,15 +576,31 @@ class TableEmbedding(Embedding):
         self.NEEDS_POSITIONS = self.freq is not None or self.scale != 1.0
 
     def tensor_specs(self):
-        return [TensorSpec(self.name, (self.vocab, self.width))]
+        specs = [TensorSpec(self.name, (self.vocab, self.width))]
+        if self.pairs is not None:
+            specs.append(TensorSpec(self.pairs["tensor"], (int(self.pairs["buckets"]) + 1, self.width)))
+        return specs
 
     def load(self, fetch):
         self.weight = self.ctx.hold(fetch(self.name), "matrix")
+        if self.pairs is not None:
+            self.pair_rows = self.ctx.hold(fetch(self.pairs["tensor"]), "matrix")
 
     def tensor(self, name):
+        if self.pairs is not None and name == self.pairs["tensor"]:
+            return self.pair_rows
         return self.weight if name in (self.name, "weight") else None
 
+    def cache_need(self):
+        return CacheNeed("paged_rows", shape=(1,), dtype=torch.int32) if self.pairs is not None else None
+
+    def forward_step(self, batch, cache):
+        p = self.pairs
+        return ops.embed_pairs(self.weight, self.pair_rows, batch, cache.rows, self.scale, int(p["mul_prev"]), int(p["mul_cur"]))
+
     def forward(self, tokens, positions=None):
+        if self.pairs is not None:
+            raise RuntimeError("an embedding with a pair table reads the step's batch and its cache (forward_step)")
         if self.NEEDS_POSITIONS:
             return ops.embed_sinusoid(self.weight, tokens, positions, self.freq, self.scale)
         return ops.embed(self.weight, tokens)
@@ -599,5 +666,6 @@ register_part("mixer", "gqa_attention", GQAttention)
 register_part("ffn", "gated_mlp", GatedMLP)
 register_part("block", "prenorm_residual", PreNormResidual)
 register_part("block", "postnorm_residual", PostNormResidual)
+register_part("block", "normed_sum_residual", NormedSumResidual)
 register_part("embedding", "table", TableEmbedding)
 register_part("head", "linear", LinearHead)
