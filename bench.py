@@ -2,7 +2,7 @@
 """Decode and prefill throughput of wick_b200 on one B200, as one JSON line.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--model 8b|14b|32b]
-    python bench.py --design nibotar|tuguvik|fasunex|sunosun [--design-size 2k|4k]      (a line of its own, see below)
+    python bench.py --design nibotar|tuguvik|fasunex|sunosun|kikopel [--design-size 2k|4k]      (a line of its own, see below)
 
 The default run has the layer sizes of Qwen3-8B (36 layers, hidden 4096, 32
 heads over 8 kv heads of 128, intermediate 12288, vocabulary 151936) with random
@@ -43,6 +43,10 @@ linear attention and a gated linear attention alone; one-matrix experts chosen w
 beside Fasunex, the closest design here (its parallel mixer holds a state-space recurrence with a state of the same size),
 at equal size, with the same kind of ``parts``; the recurrences' scans are also held against the float32 rate of the CUDA
 cores, since that, not memory, bounds them in a prompt.
+``--design kikopel`` prints the line of the Kikopel design (three layers of latent attention with a gate per element to one of
+a linear attention whose forget factor says what is written; normed results, PolyNorm feed-forwards, a pair embedding) beside
+the two designs whose layers are the closest: Tuguvik (latent attention) and Sunosun (a linear attention of the same state),
+at equal size, with the same kind of ``parts``.
 """
 import argparse
 import json
@@ -117,7 +121,10 @@ class Clocks:
             out, _ = self.proc.communicate(timeout=5)
         except subprocess.TimeoutExpired:
             self.proc.kill()
-            out, _ = self.proc.communicate()
+            try:
+                out, _ = self.proc.communicate(timeout=5)
+            except subprocess.TimeoutExpired:          # (it does not die: go on without its samples)
+                return
         sm, mx, reasons = [], [], set()
         names = ["hw_slowdown", "hw_thermal_slowdown", "sw_thermal_slowdown", "sw_power_cap"]
         for line in out.splitlines():
@@ -271,6 +278,8 @@ def design_step_bytes(eng, z, name, batch, kv_tokens):
         kv_tokens = min(kv_tokens, batch * z["mask"])
     if name == "tuguvik":
         kv_tokens = min(kv_tokens, batch * (z["window"] + z["keep_first"]))
+    if name == "kikopel":
+        return kikopel_step_bytes(eng, z, batch, kv_tokens)
     if name == "fasunex":
         return fasunex_step_bytes(eng, z, batch, kv_tokens)
     if name == "sunosun":
@@ -482,7 +491,7 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
             e0.record(torch.cuda.current_stream())
             r = fn(*a, **kw)
             e1.record(torch.cuda.current_stream())
-            acc.setdefault(kind, []).append((e0, e1) + tuple(work(r, *a, **kw)))
+            acc.setdefault(kind(*a, **kw) if callable(kind) else kind, []).append((e0, e1) + tuple(work(r, *a, **kw)))
             return r
         return run
 
@@ -505,7 +514,8 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
     def attn_flex_work(r, q, k0, k1, v, batch, scale, **kw):
         n, heads, dk = q.shape
         row_bytes = 2 * (k0[8] + k1[8] + v[8]) * (heads if not k0[9] else 1)      # (flat sources hold every head's rows)
-        return 2.0 * ctx["pairs"] * heads * (dk + kw["dv"]), nbytes(q, r) + ctx["kv_rows"] * row_bytes
+        gate = 4 * n * heads * kw["dv"] if kw.get("gate_parts") is not None else 0
+        return 2.0 * ctx["pairs"] * heads * (dk + kw["dv"]), nbytes(q, r) + ctx["kv_rows"] * row_bytes + gate
 
     def attn_std_work(r, q, kv, batch, *a, **k):
         n, H, d = q.shape
@@ -520,16 +530,36 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
         return 2.0 * parts.shape[1] * H * d * rank, nbytes(parts, uk, r)
 
     def expand_work(r, y, uv, gate, H, e, rank, **k):
-        return 2.0 * y.shape[0] * H * e * rank, nbytes(y, uv, r)
+        gate_bytes = 4 * k["gate_parts"][0].shape[0] * y.shape[0] * H * e if k.get("gate_parts") is not None else 0
+        return 2.0 * y.shape[0] * H * e * rank, nbytes(y, uv, r) + gate_bytes
 
     def norm_work(r, x, delta=None, *a, **k):
         return 0.0, nbytes(x, delta) + (nbytes(x) if delta is not None and k.get("rows") is None else 0) + (nbytes(r) if r is not None and r is not x else 0)
 
-    for fname, kind, work in (("attention_multi", "attention", attn_multi_work), ("attention_flex", "attention", attn_flex_work),
+    def finish_work(r, parts, q_rank, kv_rank, rot_dim, gate_heads, **k):
+        n, row = parts.shape[1], kv_rank + rot_dim if k["rows"] is not None else 0
+        return 0.0, n * (4 * parts.shape[0] * (q_rank + kv_rank + rot_dim + gate_heads) + 2 * row) + nbytes(*r)
+
+    def hgrn2_work(r, parts, **k):
+        n, H, dk, dv = parts.shape[1], k["heads"], k["key_dim"], k["v_dim"]
+        return 4.0 * n * H * dk * dv, nbytes(parts, r) + 2 * 4 * n * (3 * H * dk + H * dv) + 2 * 4 * k["batch"].n_seqs * H * dk * dv
+
+    def pairs_work(r, table, pairs, *a, **k):
+        return 0.0, nbytes(r) + r.numel() * 2 * table.element_size()
+
+    def norm_gate_work(r, y, parts, *a, **k):
+        return 0.0, nbytes(y, r) + (parts.shape[0] * nbytes(y) if parts is not None else 0)
+
+    latent_multi = lambda *a, **k: "attention over latent rows" if k.get("rows_of") else "attention"
+    latent_flex = lambda q, k0, k1, *a, **k: "attention with keys from the latent" if k1[8] else "attention"
+    for fname, kind, work in (("attention_multi", latent_multi, attn_multi_work), ("attention_flex", latent_flex, attn_flex_work),
                               ("combine_maps", "attention", rows_work), ("latent_query", "finish", rows_work),
                               ("attention_prompt", "attention", attn_std_work),
                               ("attention_decode", "attention", attn_std_work), ("qkv_finish", "finish", rows_work),
-                              ("latent_finish", "finish", rows_work), ("qk_norm_rope_append", "finish", rows_work),
+                              ("latent_finish", "finish", finish_work), ("qk_norm_rope_append", "finish", rows_work),
+                              ("embed_pairs", "embedding", pairs_work), ("poly_norm", "activation", rows_work),
+                              ("hgrn2_mix", "recurrence (forget factors, scan)", hgrn2_work),
+                              ("gla_norm_gate", "recurrence's norm", norm_gate_work),
                               ("latent_absorb", "query into the rows' space", absorb_work),
                               ("latent_expand", "values out of the rows' space", expand_work), ("stream_update", "norm", norm_work),
                               ("rmsnorm", "norm", lambda r, x, *a, **k: norm_work(r, x, k.get("delta"), rows=k.get("rows"))),
@@ -540,11 +570,13 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
     for blk in eng.model.blocks:
         m = blk.mixer
         for attr, kind in (("qkv", "projections into the mixer"), ("down", "projections into the mixer"),
-                           ("uq", "projections into the mixer"), ("ukv", "keys and values from the latent"), ("o", "o product")):
+                           ("uq", "projections into the mixer"), ("ukv", "keys and values from the latent"),
+                           ("input", "projections into the mixer"), ("o", "o product")):
             if isinstance(getattr(m, attr, None), Linear):
                 product(kind, getattr(m, attr))
-        for attr in ("gate_up", "down"):
-            product("feed-forward", getattr(blk.ffn, attr))
+        for attr in ("gate_up", "up", "down"):
+            if isinstance(getattr(blk.ffn, attr, None), Linear):
+                product("feed-forward", getattr(blk.ffn, attr))
         if blk.side is not None:
             product("side input", blk.side.gate)
             product("side input", blk.side.proj)
@@ -568,7 +600,7 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
         return res
 
     out = {}
-    win, keep = (z["window"], z["keep_first"]) if name == "tuguvik" else (None, 0)
+    win, keep = {"tuguvik": (z["window"], z["keep_first"]), "kikopel": (z["window"], 0)}.get(name, (None, 0))
     seen = lambda p: p + 1 if win is None else min(p + 1, win + (keep if name == "tuguvik" else 0))   # (an upper bound for kept keys)
     ptoks = random_prompts(torch, z["vocab"], [PREFILL], 3)[0]
     ctx["pairs"], ctx["kv_rows"] = sum(seen(p) for p in range(PREFILL)), PREFILL
@@ -713,6 +745,9 @@ def fasunex_parts(torch, wick, pk, z, name, cfg_json):
     def norm_work(r, x, delta=None, *a, **k):
         return 0.0, nbytes(x, delta) + (nbytes(x) if delta is not None and k.get("rows") is None else 0) + (nbytes(r) if r is not None and r is not x else 0)
 
+    def norm_gate_work(r, y, parts, *a, **k):
+        return 0.0, nbytes(y, r) + parts.shape[0] * nbytes(y)
+
     def ffn_work(width, ff, top, share, shared_ff, mats=3, shared_mats=3):
         def work(r, x, *a, **k):
             n = x.shape[0]
@@ -724,8 +759,8 @@ def fasunex_parts(torch, wick, pk, z, name, cfg_json):
     for fname, kind, work in (("attention_masked", "attention", attn_work), ("qkv_finish", "finish", rows_work),
                               ("gate_rows_", "output gate", rows_work), ("ssm_mix", "recurrence (convolution, scan)", ssm_work),
                               ("ssm_gate_norm", "recurrence's gate and norm", rows_work), ("weighted_sum", "sum of the branches", rows_work),
-                              ("gla_mix", "recurrence (decays, scan)", gla_work), ("gla_norm_gate", "recurrence's gate and norm", rows_work),
-                              ("embed_sinusoid", "embedding", rows_work),
+                              ("gla_mix", "recurrence (decays, scan)", gla_work), ("gla_norm_gate", "recurrence's gate and norm", norm_gate_work),
+                              ("embed_sinusoid", "embedding", lambda r, table, *a, **k: (0.0, nbytes(r) + r.numel() * table.element_size())),
                               ("concat_activation", "pass input", rows_work), ("stream_update", "norm", norm_work),
                               ("scaled_add_rmsnorm", "norm", lambda r, x, delta, *a, **k: norm_work(r, x, delta)),
                               ("rmsnorm", "norm", lambda r, x, *a, **k: norm_work(r, x, k.get("delta"), rows=k.get("rows")))):
@@ -880,6 +915,61 @@ def sunosun_compare(args) -> int:
     return 0 if all(m["finite"] for m in models.values()) else 1
 
 
+# ---- --design kikopel ----------------------------------------------------------
+# Kikopel beside Tuguvik (attention through a latent of the same size, the same window, a feed-forward of as many numbers) and
+# beside Sunosun (a linear attention with a state of the same size): the same width, heads, layers and vocabulary.  Three
+# layers of latent attention to one of the recurrence; the feed-forward has two matrices where Tuguvik's has three, so its
+# inner size is half as large again.
+def kikopel_configs(z):
+    d = z["dim"]
+    latent = dict(heads=z["heads"], dim=d, rot_dim=z["rot_dim"], vdim=d, q_rank=z["q_rank"], kv_rank=z["kv_rank"],
+                  scale=(d + z["rot_dim"]) ** -0.5, mask={"size": z["window"]}, rot={"dims": z["rot_dim"], "base": 10000.0})
+    hgrn2 = dict(heads=z["width"] // 128, dim=128, vdim=128)
+    layers = [dict(type="hgrn2" if i % 4 == 2 else "latent_attention", mixer=hgrn2 if i % 4 == 2 else latent,
+                   mlp={"kind": "dense", "ff": z["ff"] * 3 // 2}) for i in range(z["layers"])]
+    return dict(architecture="Kikopel", vocab=z["vocab"], width=z["width"], norm={"eps": 1e-5}, residual_mult=0.5,
+                embedding={"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 36313, "mul_cur": 27191}}, layers=layers)
+
+
+def kikopel_step_bytes(eng, z, batch, kv_tokens):
+    """Bytes a decode step of Kikopel has to read: the weights, the rows of the windows, and the recurrences' records (read and
+    written back)."""
+    n = eng.model.weight_bytes_per_step() + eng.cache.read_bytes(int(min(kv_tokens, batch * z["window"])), batch)
+    return n + sum(g.store.read_bytes(0, batch) for g in eng.cache.groups if g.need.kind == "state")
+
+
+def kikopel_compare(args) -> int:
+    import torch
+    import wick_b200 as wick
+    pk = peaks()
+    zt, zd = TUGUVIK_SIZES[args.design_size], DESIGN_SIZES[args.design_size]
+    cfgs = {"kikopel": (zt, kikopel_configs(zt), tuguvik_parts), "tuguvik": (zt, tuguvik_configs(zt)["tuguvik"], tuguvik_parts),
+            "sunosun": (zd, sunosun_configs(zd)["sunosun"], fasunex_parts)}
+    if args.design_parts:
+        z, cfg, parts_of = cfgs[args.design_parts]
+        print(json.dumps({args.design_parts: parts_of(torch, wick, pk, z, args.design_parts, cfg)}))
+        return 0
+    steps, warmup = min(args.steps, 64), max(args.warmup, 3)
+    with Clocks() as clk:
+        models = {name: design_model(torch, wick, pk, z, name, cfg, steps, warmup) for name, (z, cfg, _) in cfgs.items()}
+    env = dict(os.environ, WICK_B200_NO_PDL="1")
+    parts, errors = {}, {}
+    for name in cfgs:                                  # (a process each: the timing wrappers replace the module's functions)
+        r = subprocess.run([sys.executable, os.path.abspath(__file__), "--design", "kikopel", "--design-size", args.design_size,
+                            "--design-parts", name], env=env, capture_output=True, text=True)
+        for ln in r.stdout.splitlines():
+            if ln.startswith("{"):
+                parts.update(json.loads(ln))
+        if name not in parts:
+            errors[name] = r.stderr[-600:]
+    line = {"metric": f"Kikopel beside Tuguvik and Sunosun at equal size ({args.design_size}): prefill and decode tok/s, bf16",
+            "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": warmup, "dtype": "bf16", "sizes": zt,
+            "data": "synthetic: seeded random weights, seeded uniform random token ids", "models": models, "parts": parts,
+            "parts_error": errors or None, "clocks": clk.result, "peaks": pk, "fp32_tflops_nominal": FP32_TFLOPS_NOMINAL}
+    print(json.dumps(line))
+    return 0 if all(m["finite"] for m in models.values()) else 1
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -900,8 +990,8 @@ def main() -> int:
     ap.add_argument("--skip-prefill", action="store_true")
     ap.add_argument("--skip-decode", action="store_true", help="prefill only (for profiling)")
     ap.add_argument("--eager", action="store_true", help="no CUDA graphs (every kernel is a launch of its own)")
-    ap.add_argument("--design", default=None, choices=["nibotar", "tuguvik", "fasunex", "sunosun"],
-                    help="another line: this design beside Qwen3 (fasunex: beside Nibotar; sunosun: beside Fasunex) at equal size")
+    ap.add_argument("--design", default=None, choices=["nibotar", "tuguvik", "fasunex", "sunosun", "kikopel"],
+                    help="another line: this design beside Qwen3 (fasunex: beside Nibotar; sunosun: beside Fasunex; kikopel: beside Tuguvik and Sunosun) at equal size")
     ap.add_argument("--design-size", default="2k", choices=sorted(DESIGN_SIZES))
     ap.add_argument("--design-parts", nargs="?", const="both", default=None,
                     help="only the per-kernel times of --design (run by --design itself; tuguvik: of the model named)")
@@ -914,6 +1004,8 @@ def main() -> int:
         return fasunex_compare(args)
     if args.design == "sunosun":
         return sunosun_compare(args)
+    if args.design == "kikopel":
+        return kikopel_compare(args)
     if args.design:
         return design_compare(args)
     if args.gpus != 1:

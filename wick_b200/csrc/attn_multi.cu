@@ -459,55 +459,74 @@ attn_multi_tile_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO
     fold_warps<TO, MAPS, GROUP, MV_CHUNKS>(m, l, acc, ms, accs, out, partial, t, h0, H, e, sink, lam, eps, factor);
 }
 
-// One warp per (token, head): the records of the runs of keys (a run that held no key has the maximum -inf) are
-// folded in run order, map by map; the sink joins; the sums are divided; two maps are combined.
+// The records of the runs of keys (a run that held no key has the maximum -inf; at most 64 runs) are folded in run order, map by
+// map; the sink joins; the sums are divided; two maps are combined.  A lane reads one run's maximum and sum (or two), so that a
+// run's factor is a shuffle away and the runs' values come without a chain of loads.  One warp per (token, head); with one map a
+// warp takes one chunk of 128 values of a (token, head), since nothing but the factors joins the chunks.
 template <typename TO, int MAPS, int MV_CHUNKS>
 __global__ void __launch_bounds__(128)
 attn_multi_merge_kernel(const float* __restrict__ partial, TO* __restrict__ out, int n_heads_total, int H, int e, int runs,
                         const float* __restrict__ sink, float lam, float eps, float factor) {
+    constexpr unsigned ALL = 0xffffffffu;
+    constexpr int CPW = MAPS == 1 ? 1 : MV_CHUNKS;                            // chunks a warp takes
     pdl_trigger();
     pdl_wait();
     partial = fresh(partial);
     const int lane = threadIdx.x & 31;
-    const int th = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);      // token * H + head
+    const int e_pad = (e + 127) / 128 * 128, per = MAPS == 1 ? e_pad / 128 : 1;
+    const int64_t unit = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int th = (int)(unit / per), c0 = (int)(unit - (int64_t)th * per);      // token * H + head, first chunk
     if (th >= n_heads_total) return;
-    const int h = th % H, e_pad = (e + 127) / 128 * 128;
-    float y[MAPS][4 * MV_CHUNKS];
+    const int h = th % H;
+    float y[MAPS][4 * CPW];
 #pragma unroll
     for (int a = 0; a < MAPS; ++a) {
         const float* recs = partial + ((int64_t)th * MAPS + a) * runs * (4 + e_pad);
-        float big = sink ? sink[h] : -INFINITY;
-        for (int r = 0; r < runs; ++r) big = fmaxf(big, recs[(int64_t)r * (4 + e_pad)]);
-        float sum = sink ? expf(sink[h] - big) : 0.f;
+        float m[2], l[2];
 #pragma unroll
-        for (int c = 0; c < 4 * MV_CHUNKS; ++c) y[a][c] = 0.f;
-        for (int r = 0; r < runs; ++r) {
-            const float* rec = recs + (int64_t)r * (4 + e_pad);
-            const float mr = rec[0];
-            if (mr == -INFINITY) continue;
-            const float f = expf(mr - big);
-            sum += rec[1] * f;
+        for (int k = 0; k < 2; ++k) {
+            const int r = lane + 32 * k;
+            m[k] = r < runs ? recs[(int64_t)r * (4 + e_pad)] : -INFINITY;
+            l[k] = r < runs ? recs[(int64_t)r * (4 + e_pad) + 1] : 0.f;
+        }
+        const float big = fmaxf(warp_max(fmaxf(m[0], m[1])), sink ? sink[h] : -INFINITY);
+        float f[2], mine = 0.f;
 #pragma unroll
-            for (int c = 0; c < MV_CHUNKS; ++c)
-                if (128 * c < e_pad) {
-                    const float4 v = *reinterpret_cast<const float4*>(rec + 4 + 128 * c + 4 * lane);
-                    y[a][4 * c] = fmaf(v.x, f, y[a][4 * c]);
-                    y[a][4 * c + 1] = fmaf(v.y, f, y[a][4 * c + 1]);
-                    y[a][4 * c + 2] = fmaf(v.z, f, y[a][4 * c + 2]);
-                    y[a][4 * c + 3] = fmaf(v.w, f, y[a][4 * c + 3]);
+        for (int k = 0; k < 2; ++k) {
+            f[k] = m[k] == -INFINITY ? 0.f : expf(m[k] - big);
+            mine = fmaf(m[k] == -INFINITY ? 0.f : l[k], f[k], mine);
+        }
+        const float sum = warp_sum(mine) + (sink ? expf(sink[h] - big) : 0.f);
+#pragma unroll
+        for (int c = 0; c < 4 * CPW; ++c) y[a][c] = 0.f;
+        auto fold = [&](int r, float fr) {
+            const float* rec = recs + (int64_t)r * (4 + e_pad) + 4;
+#pragma unroll
+            for (int c = 0; c < CPW; ++c)
+                if (128 * (c0 + c) < e_pad) {
+                    const float4 v = *reinterpret_cast<const float4*>(rec + 128 * (c0 + c) + 4 * lane);
+                    y[a][4 * c] = fmaf(v.x, fr, y[a][4 * c]);
+                    y[a][4 * c + 1] = fmaf(v.y, fr, y[a][4 * c + 1]);
+                    y[a][4 * c + 2] = fmaf(v.z, fr, y[a][4 * c + 2]);
+                    y[a][4 * c + 3] = fmaf(v.w, fr, y[a][4 * c + 3]);
                 }
+        };
+#pragma unroll 4
+        for (int r = 0; r < runs; ++r) {
+            const float fr = __shfl_sync(ALL, r < 32 ? f[0] : f[1], r & 31);
+            if (fr != 0.f) fold(r, fr);               // (a run without a key left no values)
         }
         const float inv = 1.0f / sum;
 #pragma unroll
-        for (int c = 0; c < 4 * MV_CHUNKS; ++c) y[a][c] *= inv;
+        for (int c = 0; c < 4 * CPW; ++c) y[a][c] *= inv;
     }
-    finish_head<MAPS, MV_CHUNKS>(y, lane, e, lam, eps, factor);
+    finish_head<MAPS, CPW>(y, lane, e, lam, eps, factor);
     TO* o = out + (int64_t)th * e;
 #pragma unroll
-    for (int c = 0; c < MV_CHUNKS; ++c)
+    for (int c = 0; c < CPW; ++c)
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-            const int x = 128 * c + 4 * lane + i;
+            const int x = 128 * (c0 + c) + 4 * lane + i;
             if (x < e) st(o + x, y[0][4 * c + i]);
         }
 }
@@ -527,8 +546,8 @@ latent_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_
                      float* __restrict__ gate_out, T* __restrict__ rows, T* __restrict__ flat_c, T* __restrict__ flat_kr,
                      const int* __restrict__ page_table, int table_width,
                      const int* __restrict__ seq_of_token, const int* __restrict__ positions) {
-    extern __shared__ float row[];
-    __shared__ float red[40];
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[2 * 32];
     pdl_trigger();
     pdl_wait();
     parts = fresh(parts);
@@ -536,30 +555,58 @@ latent_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_
     sin_t = fresh(sin_t);
     const int t = blockIdx.x, tid = threadIdx.x;
     const int W = qr + r + dr + Hg;
-    for (int j = tid; j < W; j += blockDim.x) {
-        float v = parts[(int64_t)t * cols + j];
-        for (int s = 1; s < splits; ++s) v += parts[s * split_stride + (int64_t)t * cols + j];
-        row[j] = v;
+    const float* mine = parts + (int64_t)t * cols;
+    float ss[2] = {0.f, 0.f};                       // of the query latent, of the latent
+    if (((qr | r | cols) & 3) == 0 && (reinterpret_cast<size_t>(parts) & 15) == 0) {
+#pragma unroll 2
+        for (int j = tid * 4; j < W; j += blockDim.x * 4) {
+            float4 v = ld4(mine + j);               // (the last group may reach behind W: the row has cols numbers)
+            for (int s = 1; s < splits; ++s) {
+                const float4 d = ld4(mine + s * split_stride + j);
+                v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
+            }
+            *reinterpret_cast<float4*>(row + j) = v;
+            const float sq = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+            if (j < qr) ss[0] += sq;
+            else if (j < qr + r) ss[1] += sq;
+        }
+    } else {
+        for (int j = tid; j < W; j += blockDim.x) {
+            float v = mine[j];
+            for (int s = 1; s < splits; ++s) v += mine[s * split_stride + j];
+            row[j] = v;
+            if (j < qr) ss[0] = fmaf(v, v, ss[0]);
+            else if (j < qr + r) ss[1] = fmaf(v, v, ss[1]);
+        }
     }
-    __syncthreads();
-    float ss = 0.f;
-    for (int j = tid; j < qr; j += blockDim.x) ss = fmaf(row[j], row[j], ss);
-    ss = block_sum(ss, red);
-    const float fq = 1.0f / sqrtf(ss / (float)qr + eps);
-    for (int j = tid; j < qr; j += blockDim.x) st(cq_out + (int64_t)t * qr + j, (row[j] * fq) * q_w[j]);
+    block_sums(ss, red);                            // (its barrier also makes the row whole)
+    const float fq = 1.0f / sqrtf(ss[0] / (float)qr + eps);
+    if ((qr & 3) == 0) {
+        for (int j = tid * 4; j < qr; j += blockDim.x * 4)
+            st4(cq_out + (int64_t)t * qr + j, (row[j] * fq) * q_w[j], (row[j + 1] * fq) * q_w[j + 1], (row[j + 2] * fq) * q_w[j + 2],
+                (row[j + 3] * fq) * q_w[j + 3]);
+    } else {
+        for (int j = tid; j < qr; j += blockDim.x) st(cq_out + (int64_t)t * qr + j, (row[j] * fq) * q_w[j]);
+    }
     if (r > 0) {
-        ss = 0.f;
-        for (int j = tid; j < r; j += blockDim.x) ss = fmaf(row[qr + j], row[qr + j], ss);
-        ss = block_sum(ss, red);
         if (rows) {
-            const float fc = 1.0f / sqrtf(ss / (float)r + eps);
+            const float fc = 1.0f / sqrtf(ss[1] / (float)r + eps);
             const int pos = positions[t];
             const int pg = page_table[(int64_t)seq_of_token[t] * table_width + pos / kPage];
             T* dst = rows + ((int64_t)pg * kPage + pos % kPage) * (r + dr);
-            for (int j = tid; j < r; j += blockDim.x) {
-                const float c = (row[qr + j] * fc) * kv_w[j];
-                st(dst + j, c);
-                if (flat_c) st(flat_c + (int64_t)t * r + j, c);
+            if (((r | dr | qr) & 3) == 0) {
+                for (int j = tid * 4; j < r; j += blockDim.x * 4) {
+                    const float4 v = *reinterpret_cast<const float4*>(row + qr + j);
+                    const float a = (v.x * fc) * kv_w[j], b = (v.y * fc) * kv_w[j + 1], c = (v.z * fc) * kv_w[j + 2], d = (v.w * fc) * kv_w[j + 3];
+                    st4(dst + j, a, b, c, d);
+                    if (flat_c) st4(flat_c + (int64_t)t * r + j, a, b, c, d);
+                }
+            } else {
+                for (int j = tid; j < r; j += blockDim.x) {
+                    const float c = (row[qr + j] * fc) * kv_w[j];
+                    st(dst + j, c);
+                    if (flat_c) st(flat_c + (int64_t)t * r + j, c);
+                }
             }
             const int half = dr >> 1;
             const float* kr = row + qr + r;
@@ -594,7 +641,7 @@ latent_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_query_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, int H, int d, int dr,
-                    const float* __restrict__ cos_t, const float* __restrict__ sin_t, int pairing, T* __restrict__ out) {
+                    const float* __restrict__ cos_t, const float* __restrict__ sin_t, int pairing, T* __restrict__ out, int vec) {
     pdl_trigger();
     pdl_wait();
     parts = fresh(parts);
@@ -607,6 +654,41 @@ latent_query_kernel(const float* __restrict__ parts, int splits, int64_t split_s
         for (int s = 1; s < splits; ++s) v += parts[s * split_stride + at + j];
         return v;
     };
+    if (vec) {
+        // four plain numbers an item, or four pairs (half-split), or two pairs (neighbours)
+        auto sum4 = [&](int j) {
+            float4 v = ld4(parts + at + j);
+            for (int s = 1; s < splits; ++s) {
+                const float4 w = ld4(parts + s * split_stride + at + j);
+                v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+            }
+            return v;
+        };
+        const int d4 = d >> 2, items = d4 + (pairing == 0 ? dr >> 2 : half >> 2);
+        for (int idx = threadIdx.x; idx < H * items; idx += blockDim.x) {
+            const int h = idx / items, i = idx - h * items, base = h * dq;
+            if (i < d4 || !cos_t) {                                       // (without angles the rotated part is plain too)
+                const float4 v = sum4(base + 4 * i);
+                st4(out + at + base + 4 * i, v.x, v.y, v.z, v.w);
+                if (i >= d4 && pairing != 0) {
+                    const float4 w = sum4(base + 4 * i + half);
+                    st4(out + at + base + 4 * i + half, w.x, w.y, w.z, w.w);
+                }
+            } else if (pairing == 0) {
+                const int p = 2 * (i - d4), j = base + d + 2 * p;
+                const float4 v = sum4(j);
+                const float c0 = cos_t[(int64_t)t * half + p], s0 = sin_t[(int64_t)t * half + p];
+                const float c1 = cos_t[(int64_t)t * half + p + 1], s1 = sin_t[(int64_t)t * half + p + 1];
+                st4(out + at + j, v.x * c0 - v.y * s0, v.y * c0 + v.x * s0, v.z * c1 - v.w * s1, v.w * c1 + v.z * s1);
+            } else {
+                const int p = 4 * (i - d4), j = base + d + p;
+                const float4 u = sum4(j), v = sum4(j + half), c = ld4(cos_t + (int64_t)t * half + p), s = ld4(sin_t + (int64_t)t * half + p);
+                st4(out + at + j, u.x * c.x - v.x * s.x, u.y * c.y - v.y * s.y, u.z * c.z - v.z * s.z, u.w * c.w - v.w * s.w);
+                st4(out + at + j + half, v.x * c.x + u.x * s.x, v.y * c.y + u.y * s.y, v.z * c.z + u.z * s.z, v.w * c.w + u.w * s.w);
+            }
+        }
+        return;
+    }
     for (int idx = threadIdx.x; idx < H * per; idx += blockDim.x) {
         const int h = idx / per, i = idx - h * per;
         if (i < d) {
@@ -745,6 +827,166 @@ latent_expand_kernel(const float* __restrict__ y, const T* __restrict__ uv, cons
     }
 }
 
+// The two for steps of few tokens, where what counts is that the matrices come from memory with many loads on their way and over
+// many blocks.
+//   absorb: grid (tokens / 8, H, ceil(r / 64)), a block takes 64 columns of the head's block of Wuk: lane l two neighbouring ones,
+//           warp w the rows w, w + 8, ...; the warps' sums meet in shared memory.
+//   expand: grid (tokens / 8, H, ceil(e / 8)), a warp takes one row of the head's block of Wuv, lane l the pairs l, l + 32, ...
+// r is even here.
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_absorb_few_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, const T* __restrict__ uk, int n, int H,
+                         int d, int dr, int r, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int pairing,
+                         float* __restrict__ out) {
+    extern __shared__ __align__(16) float qh[];   // [d + dr][TT]: a number of all TT tokens side by side
+    __shared__ float sums[8][LAT_TT][64];
+    pdl_trigger();
+    const int t0 = blockIdx.x * LAT_TT, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int dq = d + dr, W = H * dq, n_t = min(LAT_TT, n - t0), j0 = blockIdx.z * 64 + 2 * lane;
+    const T* w = uk + (int64_t)h * d * r + j0;
+    constexpr int AHEAD = 16;                     // (weights: the first loads need not wait for the kernel before this one)
+    float2 wv[AHEAD];
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) {
+        const int x = warp + 8 * k;
+        wv[k] = x < d && j0 < r ? ld2(w + (int64_t)x * r) : make_float2(0.f, 0.f);
+    }
+    pdl_wait();
+    parts = fresh(parts);
+    cos_t = fresh(cos_t);
+    sin_t = fresh(sin_t);
+    for (int idx = tid; idx < LAT_TT * dq; idx += blockDim.x) {
+        const int tt = idx / dq, x = idx - tt * dq;
+        float v = 0.f;
+        if (tt < n_t) {
+            const int64_t at = (int64_t)(t0 + tt) * W + h * dq + x;
+            for (int s = 0; s < splits; ++s) v += parts[s * split_stride + at];
+        }
+        qh[x * LAT_TT + tt] = v;
+    }
+    __syncthreads();
+    if (blockIdx.z == 0) {
+        const int half = dr >> 1;
+        for (int idx = tid; idx < n_t * half; idx += blockDim.x) {
+            const int tt = idx / half, i = idx - tt * half;
+            const int p0 = pairing == 0 ? 2 * i : i, p1 = pairing == 0 ? 2 * i + 1 : i + half;
+            float u = qh[(d + p0) * LAT_TT + tt], v = qh[(d + p1) * LAT_TT + tt];
+            if (cos_t) {
+                const float cs = cos_t[(int64_t)(t0 + tt) * half + i], sn = sin_t[(int64_t)(t0 + tt) * half + i];
+                const float ru = u * cs - v * sn, rv = v * cs + u * sn;
+                u = ru;
+                v = rv;
+            }
+            float* o = out + ((int64_t)(t0 + tt) * H + h) * (r + dr) + r;
+            o[p0] = u;
+            o[p1] = v;
+        }
+        if ((dr & 1) && tid < n_t) out[((int64_t)(t0 + tid) * H + h) * (r + dr) + r + dr - 1] = qh[(d + dr - 1) * LAT_TT + tid];
+    }
+    float acc[LAT_TT][2];
+#pragma unroll
+    for (int tt = 0; tt < LAT_TT; ++tt) acc[tt][0] = acc[tt][1] = 0.f;
+    for (int x0 = 0; x0 < d; x0 += 8 * AHEAD) {
+#pragma unroll
+        for (int k = 0; k < AHEAD; ++k) {
+            const int x = x0 + warp + 8 * k;
+            if (x < d) {
+                const float4 qa = *reinterpret_cast<const float4*>(qh + x * LAT_TT), qb = *reinterpret_cast<const float4*>(qh + x * LAT_TT + 4);
+                const float q[LAT_TT] = {qa.x, qa.y, qa.z, qa.w, qb.x, qb.y, qb.z, qb.w};
+#pragma unroll
+                for (int tt = 0; tt < LAT_TT; ++tt) {
+                    acc[tt][0] = fmaf(q[tt], wv[k].x, acc[tt][0]);
+                    acc[tt][1] = fmaf(q[tt], wv[k].y, acc[tt][1]);
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < AHEAD; ++k) {
+            const int x = x0 + 8 * AHEAD + warp + 8 * k;
+            if (x < d && j0 < r) wv[k] = ld2(w + (int64_t)x * r);
+        }
+    }
+#pragma unroll
+    for (int tt = 0; tt < LAT_TT; ++tt) *reinterpret_cast<float2*>(&sums[warp][tt][2 * lane]) = make_float2(acc[tt][0], acc[tt][1]);
+    __syncthreads();
+    for (int idx = tid; idx < n_t * 64; idx += blockDim.x) {
+        const int tt = idx >> 6, c = idx & 63, j = blockIdx.z * 64 + c;
+        if (j >= r) continue;
+        float v = 0.f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v += sums[k][tt][c];
+        out[((int64_t)(t0 + tt) * H + h) * (r + dr) + j] = v;
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_expand_few_kernel(const float* __restrict__ y, const T* __restrict__ uv, const float* __restrict__ gate, int n, int H,
+                         int e, int r, T* __restrict__ out, const float* __restrict__ gate_parts, int gate_splits, int64_t gate_stride,
+                         int gate_cols, int gate_col) {
+    extern __shared__ __align__(16) float ys[];   // [TT][r]
+    pdl_trigger();
+    const int t0 = blockIdx.x * LAT_TT, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int n_t = min(LAT_TT, n - t0), x = blockIdx.z * 8 + warp;
+    const T* w = uv + ((int64_t)h * e + x) * r;
+    constexpr int AHEAD = 8;
+    float2 wv[AHEAD];
+#pragma unroll
+    for (int k = 0; k < AHEAD; ++k) {
+        const int j = 2 * (lane + 32 * k);
+        wv[k] = x < e && j < r ? ld2(w + j) : make_float2(0.f, 0.f);
+    }
+    pdl_wait();
+    y = fresh(y);
+    gate = fresh(gate);
+    gate_parts = fresh(gate_parts);
+    float gt = 1.f;
+    if (lane < n_t && x < e) {
+        if (gate) gt = gate[(int64_t)(t0 + lane) * H + h];
+        if (gate_parts) {
+            float z = 0.f;
+            for (int s = 0; s < gate_splits; ++s) z += gate_parts[s * gate_stride + (int64_t)(t0 + lane) * gate_cols + gate_col + h * e + x];
+            gt = 1.0f / (1.0f + expf(-z));
+        }
+    }
+    for (int tt = 0; tt < LAT_TT; ++tt)
+        for (int j = 2 * tid; j < r; j += 2 * blockDim.x)
+            *reinterpret_cast<float2*>(ys + tt * r + j) = tt < n_t ? ld2(y + ((int64_t)(t0 + tt) * H + h) * r + j) : make_float2(0.f, 0.f);
+    __syncthreads();
+    if (x >= e) return;
+    float acc[LAT_TT];
+#pragma unroll
+    for (int tt = 0; tt < LAT_TT; ++tt) acc[tt] = 0.f;
+    for (int b = 0; b < r; b += 64 * AHEAD) {
+#pragma unroll
+        for (int k = 0; k < AHEAD; ++k) {
+            const int j = b + 2 * (lane + 32 * k);
+            if (j < r) {
+#pragma unroll
+                for (int tt = 0; tt < LAT_TT; ++tt) {
+                    const float2 v = *reinterpret_cast<const float2*>(ys + tt * r + j);
+                    acc[tt] = fmaf(v.x, wv[k].x, fmaf(v.y, wv[k].y, acc[tt]));
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < AHEAD; ++k) {
+            const int j = b + 64 * AHEAD + 2 * (lane + 32 * k);
+            if (j < r) wv[k] = ld2(w + j);
+        }
+    }
+    float mine = 0.f;
+#pragma unroll
+    for (int tt = 0; tt < LAT_TT; ++tt) {
+        const float v = warp_sum(acc[tt]);
+        if (lane == tt) mine = v;
+    }
+    if (lane < n_t) st(out + ((int64_t)(t0 + lane) * H + h) * e + x, mine * gt);
+}
+
+constexpr int LAT_FEW = 64;                     // tokens up to which the two forms for few tokens are taken
+
 // ---------------------------------------------------------------------------
 template <typename T, typename TQ, typename TO, int MAPS, int GROUP, int MV_CHUNKS>
 int attn_multi_launch(const void* q, const void* store, void* out, float* partial, const int* seq_of_token, const int* positions,
@@ -774,7 +1016,7 @@ int attn_multi_launch(const void* q, const void* store, void* out, float* partia
                              H, G, dm, e, page_elems, k_row, v_off, v_row, scale, window, keep_first, sink, lam, eps, factor));
             if (int rc = check_launch("attn_multi_tile")) return rc;
             if (partial) {
-                WICK_CUDA(launch(attn_multi_merge_kernel<TO, MAPS, MV_CHUNKS>, dim3(ceil_div((int64_t)n * H, 4)), dim3(128), 0, s,
+                WICK_CUDA(launch(attn_multi_merge_kernel<TO, MAPS, MV_CHUNKS>, dim3(ceil_div((int64_t)n * H * (MAPS == 1 ? e_pad / 128 : 1), 4)), dim3(128), 0, s,
                                  (const float*)partial, (TO*)out, n * H, H, e, runs, sink, lam, eps, factor));
                 return check_launch("attn_multi_merge");
             }
@@ -793,7 +1035,7 @@ int attn_multi_launch(const void* q, const void* store, void* out, float* partia
                      page_elems, k_row, v_off, v_row, scale, window, keep_first, sink, lam, eps, factor));
     if (int rc = check_launch("attn_multi")) return rc;
     if (partial) {
-        WICK_CUDA(launch(attn_multi_merge_kernel<TO, MAPS, MV_CHUNKS>, dim3(ceil_div((int64_t)n * H, 4)), dim3(128), 0, s, (const float*)partial,
+        WICK_CUDA(launch(attn_multi_merge_kernel<TO, MAPS, MV_CHUNKS>, dim3(ceil_div((int64_t)n * H * (MAPS == 1 ? e_pad / 128 : 1), 4)), dim3(128), 0, s, (const float*)partial,
                          (TO*)out, n * H, H, e, runs, sink, lam, eps, factor));
         return check_launch("attn_multi_merge");
     }
@@ -843,7 +1085,7 @@ int latent_finish(const float* parts, int splits, int n, int cols, int qr, int r
     WICK_REQUIRE(!rows || (r > 0 && kv_w), "latent_finish: a cache row needs the latent and its norm weight");
     if (n == 0) return 0;
     const int W = qr + r + dr + Hg;
-    const size_t smem = (size_t)W * sizeof(float);
+    const size_t smem = (size_t)((W + 3) & ~3) * sizeof(float);
     WICK_REQUIRE(W <= cols, "latent_finish: rows of %d numbers, %d expected", cols, W);
     WICK_REQUIRE(smem <= 48 * 1024, "latent_finish: a row of %d numbers is beyond one block's shared memory", W);
     WICK_CUDA(launch(latent_finish_kernel<T>, dim3(n), dim3(256), smem, s, parts, splits, (int64_t)n * cols, cols, qr, r, dr, Hg, q_w, kv_w, eps,
@@ -859,6 +1101,11 @@ int latent_absorb(const float* parts, int splits, const void* uk, int n, int H, 
     WICK_REQUIRE(H <= 65535, "latent_absorb: too many heads");
     if (n == 0) return 0;
     const size_t smem = (size_t)LAT_TT * (d + dr) * sizeof(float);
+    if (n <= LAT_FEW && r % 2 == 0 && smem <= 28 * 1024 && ((uintptr_t)uk & 7) == 0 && ceil_div(r, 64) <= 65535) {
+        WICK_CUDA(launch(latent_absorb_few_kernel<T>, dim3(ceil_div(n, LAT_TT), H, ceil_div(r, 64)), dim3(256), smem, s, parts, splits,
+                         (int64_t)n * H * (d + dr), (const T*)uk, n, H, d, dr, r, cos_t, sin_t, pairing, out));
+        return check_launch("latent_absorb_few");
+    }
     WICK_REQUIRE(smem <= 48 * 1024, "latent_absorb: a head of %d numbers is beyond one block's shared memory", d + dr);
     WICK_CUDA(launch(latent_absorb_kernel<T>, dim3(ceil_div(n, LAT_TT), H, min(64, ceil_div(r, 128))), dim3(128), smem, s, parts, splits,
                      (int64_t)n * H * (d + dr), (const T*)uk, n, H, d, dr, r, cos_t, sin_t, pairing, out));
@@ -870,8 +1117,10 @@ int latent_query(const float* parts, int splits, int n, int H, int d, int dr, co
                  void* out, cudaStream_t s) {
     WICK_REQUIRE(H > 0 && d > 0 && dr >= 0 && splits >= 1, "latent_query: bad sizes");
     if (n == 0) return 0;
+    const int vec = (d & 3) == 0 && (pairing == 0 ? (dr & 3) == 0 : (dr & 7) == 0) &&
+                    (((uintptr_t)parts | (uintptr_t)cos_t | (uintptr_t)sin_t | (uintptr_t)out) & 15) == 0;
     WICK_CUDA(launch(latent_query_kernel<T>, dim3(n), dim3(256), 0, s, parts, splits, (int64_t)n * H * (d + dr), H, d, dr, cos_t, sin_t,
-                     pairing, (T*)out));
+                     pairing, (T*)out, vec));
     return check_launch("latent_query");
 }
 
@@ -882,6 +1131,11 @@ int latent_expand(const float* y, const void* uv, const float* gate, int n, int 
     WICK_REQUIRE(!gate_parts || (gate_splits >= 1 && gate_col >= 0 && gate_col + H * e <= gate_cols), "latent_expand: bad gate columns");
     if (n == 0) return 0;
     const size_t smem = (size_t)LAT_TT * r * sizeof(float);
+    if (n <= LAT_FEW && r % 2 == 0 && smem <= 48 * 1024 && (((uintptr_t)uv | (uintptr_t)y) & 7) == 0 && ceil_div(e, 8) <= 65535) {
+        WICK_CUDA(launch(latent_expand_few_kernel<T>, dim3(ceil_div(n, LAT_TT), H, ceil_div(e, 8)), dim3(256), smem, s, y, (const T*)uv, gate,
+                         n, H, e, r, (T*)out, gate_parts, gate_splits, gate_stride, gate_cols, gate_col));
+        return check_launch("latent_expand_few");
+    }
     WICK_REQUIRE(smem <= 48 * 1024, "latent_expand: a latent of %d numbers is beyond one block's shared memory", r);
     WICK_CUDA(launch(latent_expand_kernel<T>, dim3(ceil_div(n, LAT_TT), H, min(64, ceil_div(e, 32))), dim3(256), smem, s, y, (const T*)uv, gate,
                      n, H, e, r, (T*)out, gate_parts, gate_splits, gate_stride, gate_cols, gate_col));

@@ -74,15 +74,6 @@ __device__ __forceinline__ float sumsq4(float ss, float4 v) {
     return __fadd_rn(ss, __fadd_rn(__fadd_rn(__fadd_rn(__fmul_rn(v.x, v.x), __fmul_rn(v.y, v.y)), __fmul_rn(v.z, v.z)), __fmul_rn(v.w, v.w)));
 }
 __device__ __forceinline__ float normed(float v, float scale, float g) { return __fmul_rn(__fmul_rn(v, scale), g); }
-// Four neighbouring outputs at an index that is a multiple of 4.
-__device__ __forceinline__ void st4(float* p, float a, float b, float c, float d) { *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d); }
-__device__ __forceinline__ void st4(__nv_bfloat16* p, float a, float b, float c, float d) {
-    uint2 u;
-    __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
-    u.x = *reinterpret_cast<uint32_t*>(&lo);
-    u.y = *reinterpret_cast<uint32_t*>(&hi);
-    *reinterpret_cast<uint2*>(p) = u;
-}
 __device__ __forceinline__ float rms_scale(float ss, int width, float eps) { return 1.0f / sqrtf(__fadd_rn(__fdiv_rn(ss, (float)width), eps)); }
 
 // One block per output row i.  Source row r = rows ? rows[i] : i.  If delta is
@@ -240,8 +231,6 @@ __global__ void rope_table_kernel(const int* __restrict__ positions, const float
 }
 
 // Two neighbouring elements at an even index.
-__device__ __forceinline__ float2 ld2(const float* p) { return *reinterpret_cast<const float2*>(p); }
-__device__ __forceinline__ float2 ld2(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
 __device__ __forceinline__ void st2(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
 __device__ __forceinline__ void st2(__nv_bfloat16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
 

@@ -32,6 +32,30 @@ __device__ __forceinline__ void add_partials4(float4& v, const float* __restrict
     }
 }
 
+// v[u] = the partial sums of the thread's VPT groups of four of a row (group u: columns (u blockDim + thread) 4 .. + 3), added in
+// index order; the loads of all groups and of SU partial sums are on their way together.
+template <int VPT, int SU>
+__device__ __forceinline__ void row_partials(float4 (&v)[VPT], const float* __restrict__ row, int splits, int64_t split_stride, int width) {
+#pragma unroll
+    for (int u = 0; u < VPT; ++u) v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s0 = 0; s0 < splits; s0 += SU) {
+        float4 d[SU][VPT];
+#pragma unroll
+        for (int k = 0; k < SU; ++k)
+#pragma unroll
+            for (int u = 0; u < VPT; ++u) {
+                const int j = (u * (int)blockDim.x + (int)threadIdx.x) * 4;
+                d[k][u] = s0 + k < splits && j < width ? ld4(row + (s0 + k) * split_stride + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+        for (int k = 0; k < SU; ++k)
+#pragma unroll
+            for (int u = 0; u < VPT; ++u) {
+                v[u].x += d[k][u].x; v[u].y += d[k][u].y; v[u].z += d[k][u].z; v[u].w += d[k][u].w;
+            }
+    }
+}
+
 // One block per row; the row waits in shared memory between the two passes.  First pass:
 // v = alpha x + the partial sums (index order) and the sum of its squares (a thread's elements in
 // index order, then the block's sum in thread order); second pass: y = v * scale * w to x and out.
@@ -113,12 +137,17 @@ __global__ void soft_cap_kernel(float* __restrict__ z, int64_t n, float cap) {
 
 // float32 -> activation type (the residual stream as the input of a matrix product).
 template <typename T>
-__global__ void to_activation_kernel(const float* __restrict__ x, T* __restrict__ out, int64_t n) {
+__global__ void to_activation_kernel(const float* __restrict__ x, T* __restrict__ out, int64_t n, int vec) {
     pdl_trigger();
     pdl_wait();
     x = fresh(x);
-    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) st(out + i, x[i]);
+    const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (vec && i + 3 < n) {
+        const float4 v = ld4(x + i);
+        st4(out + i, v.x, v.y, v.z, v.w);
+    } else {
+        for (int64_t k = i; k < i + 4 && k < n; ++k) st(out + k, x[k]);
+    }
 }
 
 // One block per output row i; source row r = rows ? rows[i] : i.
@@ -234,6 +263,66 @@ stream_update_kernel(float* __restrict__ x, const float* __restrict__ delta, int
     }
 }
 
+// The same for rows of whole groups of four whose sums are normed (rms_w) and that end in a norm by the root mean square, in a copy
+// or in neither: a thread keeps VPT groups of the row's sums and of the stream in registers, all of their loads on their way
+// before the first reduction.
+template <typename TOut, int VPT>
+__global__ void __launch_bounds__(1024)
+stream_rms_kernel(float* __restrict__ x, const float* __restrict__ delta, int splits, int64_t split_stride, const float* __restrict__ scale,
+                  const float* __restrict__ rms_w, float rms_eps, const float* __restrict__ w, float out_eps, const int* __restrict__ rows,
+                  TOut* __restrict__ out, int width) {
+    __shared__ float red[2 * 32];
+    pdl_trigger();
+    pdl_wait();
+    x = fresh(x);
+    delta = fresh(delta);
+    const int i = blockIdx.x;
+    const int64_t r = rows ? rows[i] : i;
+    float* xr = x + r * width;
+    const float* dr = delta + r * width;
+    float4 xv[VPT], d[VPT];
+#pragma unroll
+    for (int u = 0; u < VPT; ++u) {
+        const int j = (u * (int)blockDim.x + (int)threadIdx.x) * 4;
+        const bool in = j < width;
+        xv[u] = in ? ld4(xr + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    row_partials<VPT, VPT <= 2 ? 4 : 1>(d, dr, splits, split_stride, width);
+    float ss[1] = {0.f};
+#pragma unroll
+    for (int u = 0; u < VPT; ++u)
+        ss[0] = fmaf(d[u].x, d[u].x, fmaf(d[u].y, d[u].y, fmaf(d[u].z, d[u].z, fmaf(d[u].w, d[u].w, ss[0]))));
+    block_sums(ss, red);
+    const float f = 1.0f / sqrtf(ss[0] / (float)width + rms_eps);
+    ss[0] = 0.f;
+#pragma unroll
+    for (int u = 0; u < VPT; ++u) {
+        const int j = (u * (int)blockDim.x + (int)threadIdx.x) * 4;
+        if (j >= width) continue;
+        const float4 g = ld4(rms_w + j);
+        float4 t = make_float4((d[u].x * f) * g.x, (d[u].y * f) * g.y, (d[u].z * f) * g.z, (d[u].w * f) * g.w);
+        if (scale) {
+            const float4 sc = ld4(scale + j);
+            t.x *= sc.x; t.y *= sc.y; t.z *= sc.z; t.w *= sc.w;
+        }
+        xv[u].x += t.x; xv[u].y += t.y; xv[u].z += t.z; xv[u].w += t.w;
+        const float4 v = xv[u];
+        if (!rows) st4(xr + j, v.x, v.y, v.z, v.w);
+        if (out && !w) st4(out + (int64_t)i * width + j, v.x, v.y, v.z, v.w);
+        ss[0] = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss[0]))));
+    }
+    if (!w) return;
+    block_sums(ss, red + 32);
+    const float q = 1.0f / sqrtf(ss[0] / (float)width + out_eps);
+#pragma unroll
+    for (int u = 0; u < VPT; ++u) {
+        const int j = (u * (int)blockDim.x + (int)threadIdx.x) * 4;
+        if (j >= width) continue;
+        const float4 g = ld4(w + j), v = xv[u];
+        st4(out + (int64_t)i * width + j, (v.x * q) * g.x, (v.y * q) * g.y, (v.z * q) * g.z, (v.w * q) * g.w);
+    }
+}
+
 // out[t, j] = gelu_tanh(z[t, j]) * table[tokens[t], offset + j]; gelu_tanh(z) = z/2 (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).
 template <typename T>
 __global__ void gelu_gate_rows_kernel(const float* __restrict__ z, const T* __restrict__ table, const int* __restrict__ tokens,
@@ -300,7 +389,7 @@ __global__ void __launch_bounds__(256)
 embed_pairs_kernel(const T* __restrict__ table, const T* __restrict__ pairs, const int* __restrict__ tokens,
                    const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ cu_seqlens,
                    const int* __restrict__ page_table, int table_width, int* history, int64_t buckets, int64_t mul_prev,
-                   int64_t mul_cur, float scale, float* __restrict__ out, int width) {
+                   int64_t mul_cur, float scale, float* __restrict__ out, int width, int vec) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x, tok = tokens[t], pos = positions[t], b = seq_of_token[t];
@@ -313,22 +402,73 @@ embed_pairs_kernel(const T* __restrict__ table, const T* __restrict__ pairs, con
     if (threadIdx.x == 0) history[(int64_t)pages[pos / kPage] * kPage + pos % kPage] = tok;
     const T* row = table + (int64_t)tok * width;
     const T* add = pairs + r * width;
-    for (int j = threadIdx.x; j < width; j += blockDim.x) out[(int64_t)t * width + j] = fmaf(ld(row + j), scale, ld(add + j));
+    float* o = out + (int64_t)t * width;
+    if (vec) {
+        for (int j = threadIdx.x * 4; j < width; j += blockDim.x * 4) {
+            const float4 a = ld4(row + j), b = ld4(add + j);
+            st4(o + j, fmaf(a.x, scale, b.x), fmaf(a.y, scale, b.y), fmaf(a.z, scale, b.z), fmaf(a.w, scale, b.w));
+        }
+    } else {
+        for (int j = threadIdx.x; j < width; j += blockDim.x) o[j] = fmaf(ld(row + j), scale, ld(add + j));
+    }
 }
 
 // ---- PolyNorm ------------------------------------------------------------------------------------------------------
 // One block per row of ff numbers z (the partial sums in index order): the means of z^2, z^4 and z^6, then
-// a r(z) + b r(z^2) + c r(z^3) + e out in the activation type.  The row waits in shared memory between the two passes (keep) or
-// is added up again.  The block's size depends on ff alone.
+// a r(z) + b r(z^2) + c r(z^3) + e out in the activation type.
+struct PolyCoef {
+    float a, b, c, e;
+};
+__device__ __forceinline__ void poly_powers(float z, float (&s)[3]) {
+    const float q = z * z;
+    s[0] += q;
+    s[1] = fmaf(q, q, s[1]);
+    s[2] = fmaf(q * q, q, s[2]);
+}
+__device__ __forceinline__ PolyCoef poly_factors(PolyCoef k, const float (&s)[3], int ff, float eps) {
+    const float inv = 1.0f / (float)ff;
+    return {k.a / sqrtf(fmaf(s[0], inv, eps)), k.b / sqrtf(fmaf(s[1], inv, eps)), k.c / sqrtf(fmaf(s[2], inv, eps)), k.e};
+}
+__device__ __forceinline__ float poly_value(float z, PolyCoef f) { return fmaf(z, fmaf(z, fmaf(z, f.c, f.b), f.a), f.e); }
+
+// Rows of whole groups of four: a thread keeps VPT groups in registers, so that all its loads of a partial sum are on their way at
+// once and nothing is read twice.
+template <typename TOut, int VPT>
+__global__ void __launch_bounds__(VPT >= 8 ? 512 : 1024)
+poly_norm_regs_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, const float* __restrict__ coef, float eps,
+                      TOut* __restrict__ out, int ff) {
+    __shared__ float red[3 * 32];
+    pdl_trigger();
+    const PolyCoef k = {coef[0], coef[1], coef[2], coef[3]};                 // (weights: no kernel writes them)
+    pdl_wait();
+    parts = fresh(parts);
+    const int64_t at = (int64_t)blockIdx.x * ff;
+    float4 z[VPT];
+    row_partials<VPT, VPT <= 2 ? 4 : 1>(z, parts + at, splits, split_stride, ff);
+    float sums[3] = {0.f, 0.f, 0.f};
+#pragma unroll
+    for (int u = 0; u < VPT; ++u) {
+        poly_powers(z[u].x, sums); poly_powers(z[u].y, sums); poly_powers(z[u].z, sums); poly_powers(z[u].w, sums);
+    }
+    block_sums(sums, red);
+    const PolyCoef f = poly_factors(k, sums, ff, eps);
+#pragma unroll
+    for (int u = 0; u < VPT; ++u) {
+        const int j = (u * (int)blockDim.x + (int)threadIdx.x) * 4;
+        if (j < ff) st4(out + at + j, poly_value(z[u].x, f), poly_value(z[u].y, f), poly_value(z[u].z, f), poly_value(z[u].w, f));
+    }
+}
+
+// Rows of any length: the row waits in shared memory between the two passes (keep) or is added up again.
 template <typename TOut, bool VEC>
 __global__ void __launch_bounds__(1024)
 poly_norm_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, const float* __restrict__ coef, float eps,
                  TOut* __restrict__ out, int ff, int keep) {
     extern __shared__ float smem[];
-    __shared__ float red[3][33];
+    __shared__ float red[3 * 32];
     float* row = smem;
     pdl_trigger();
-    const float ca = coef[0], cb = coef[1], cc = coef[2], ce = coef[3];      // (weights: no kernel writes them)
+    const PolyCoef co = {coef[0], coef[1], coef[2], coef[3]};                // (weights: no kernel writes them)
     pdl_wait();
     parts = fresh(parts);
     const int64_t at = (int64_t)blockIdx.x * ff;
@@ -344,31 +484,18 @@ poly_norm_kernel(const float* __restrict__ parts, int splits, int64_t split_stri
             z[0] = v;
         }
     };
-    float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+    float sums[3] = {0.f, 0.f, 0.f};
     for (int j = threadIdx.x * V; j < ff; j += blockDim.x * V) {
         float z[V];
         load(j, z);
 #pragma unroll
         for (int i = 0; i < V; ++i) {
             if (keep) row[j + i] = z[i];
-            const float q = z[i] * z[i];
-            s2 += q;
-            s4 = fmaf(q, q, s4);
-            s6 = fmaf(q * q, q, s6);
+            poly_powers(z[i], sums);
         }
     }
-    // the three sums over the block in one go: warps' sums, then every warp adds those up
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-    s2 = warp_sum(s2); s4 = warp_sum(s4); s6 = warp_sum(s6);
-    if (lane == 0) {
-        red[0][warp] = s2; red[1][warp] = s4; red[2][warp] = s6;
-    }
-    __syncthreads();
-    s2 = warp_sum(lane < nw ? red[0][lane] : 0.f);
-    s4 = warp_sum(lane < nw ? red[1][lane] : 0.f);
-    s6 = warp_sum(lane < nw ? red[2][lane] : 0.f);
-    const float inv = 1.0f / (float)ff;
-    const float fa = ca / sqrtf(fmaf(s2, inv, eps)), fb = cb / sqrtf(fmaf(s4, inv, eps)), fc = cc / sqrtf(fmaf(s6, inv, eps));
+    block_sums(sums, red);
+    const PolyCoef f = poly_factors(co, sums, ff, eps);
     TOut* o = out + at;
     for (int j = threadIdx.x * V; j < ff; j += blockDim.x * V) {
         float z[V];
@@ -379,7 +506,7 @@ poly_norm_kernel(const float* __restrict__ parts, int splits, int64_t split_stri
             load(j, z);
         }
 #pragma unroll
-        for (int i = 0; i < V; ++i) st(o + j + i, fmaf(z[i], fmaf(z[i], fmaf(z[i], fc, fb), fa), ce));
+        for (int i = 0; i < V; ++i) st(o + j + i, poly_value(z[i], f));
     }
 }
 
@@ -453,6 +580,15 @@ int stream_update(float* x, const float* delta, int splits, const float* scale, 
         WICK_CUDA(cudaFuncSetAttribute(stream_update_kernel<TOut>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
         raised = true;
     }
+    if (delta && rms_w && !b && (width & 3) == 0 && width <= 8192 &&
+        (((uintptr_t)x | (uintptr_t)delta | (uintptr_t)rms_w | (uintptr_t)scale | (uintptr_t)w | (uintptr_t)out) & 15) == 0) {
+        const bool many = n_out > 2 * sm_count();       // (few rows: more threads a row; many: more rows an SM)
+        auto kernel = many ? stream_rms_kernel<TOut, 4> : stream_rms_kernel<TOut, 2>;
+        const int vpt = many ? 4 : 2;
+        WICK_CUDA(launch(kernel, dim3(n_out), dim3((ceil_div(width, 4 * vpt) + 31) / 32 * 32), 0, s, x, delta, splits, (int64_t)n * width, scale,
+                         rms_w, rms_eps, w, out_eps, rows, (TOut*)out, width));
+        return check_launch("stream_rms");
+    }
     const int threads = min(1024, max(64, ((width + 3) / 4 + 31) / 32 * 32));
     WICK_CUDA(launch(stream_update_kernel<TOut>, dim3(n_out), dim3(threads), smem, s, x, delta, splits, (int64_t)n * width, scale,
                      rms_w, rms_eps, alpha, w, b, out_eps, rows, (TOut*)out, width));
@@ -492,9 +628,19 @@ int poly_norm_launch(const float* parts, int splits, const float* coef, float ep
                      keep));
     return check_launch("poly_norm");
 }
+template <typename TOut, int VPT>
+int poly_norm_regs(const float* parts, int splits, const float* coef, float eps, void* out, int n, int ff, cudaStream_t s) {
+    const int threads = max(32, (ceil_div(ff, 4 * VPT) + 31) / 32 * 32);
+    WICK_CUDA(launch(poly_norm_regs_kernel<TOut, VPT>, dim3(n), dim3(threads), 0, s, parts, splits, (int64_t)n * ff, coef, eps, (TOut*)out, ff));
+    return check_launch("poly_norm");
+}
 template <typename TOut>
 int poly_norm(const float* parts, int splits, const float* coef, float eps, void* out, int n, int ff, cudaStream_t s) {
-    if ((ff & 3) == 0 && ((uintptr_t)parts & 15) == 0) return poly_norm_launch<TOut, true>(parts, splits, coef, eps, out, n, ff, s);
+    const bool vec = (ff & 3) == 0 && (((uintptr_t)parts | (uintptr_t)out) & 15) == 0;
+    // (steps of few tokens: more threads a row; long ones: more rows an SM, each thread with more loads on their way)
+    if (vec && ff <= 8192 && n <= 2 * sm_count()) return poly_norm_regs<TOut, 2>(parts, splits, coef, eps, out, n, ff, s);
+    if (vec && ff <= 16384) return poly_norm_regs<TOut, 8>(parts, splits, coef, eps, out, n, ff, s);
+    if (vec) return poly_norm_launch<TOut, true>(parts, splits, coef, eps, out, n, ff, s);
     return poly_norm_launch<TOut, false>(parts, splits, coef, eps, out, n, ff, s);
 }
 
@@ -568,7 +714,8 @@ WICK_API int wick_soft_cap(float* z, int64_t n, float cap, void* s) {
 
 WICK_API int wick_to_activation_bf16(const float* x, void* out, int64_t n, void* s) {
     if (n == 0) return 0;
-    WICK_CUDA(launch(to_activation_kernel<bf16>, dim3(ceil_div(n, 256)), dim3(256), 0, (cudaStream_t)s, x, (bf16*)out, n));
+    const int vec = (((uintptr_t)x & 15) | ((uintptr_t)out & 7)) == 0;
+    WICK_CUDA(launch(to_activation_kernel<bf16>, dim3(ceil_div(n, 1024)), dim3(256), 0, (cudaStream_t)s, x, (bf16*)out, n, vec));
     return check_launch("to_activation");
 }
 
@@ -623,9 +770,10 @@ WICK_EMBED_SINUSOID(wick_embed_sinusoid_f32, float)
                       int64_t mul_prev, int64_t mul_cur, float scale, float* out, int n, int width, void* s) {               \
         WICK_REQUIRE(n >= 0 && width > 0 && buckets > 0 && mul_prev >= 0 && mul_cur >= 0, "embed_pairs: bad sizes");          \
         if (n == 0) return 0;                                                                                                \
+        const int vec = width % 4 == 0 && (((uintptr_t)table | (uintptr_t)pairs | (uintptr_t)out) & 15) == 0;                \
         WICK_CUDA(launch(embed_pairs_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)s, (const T*)table, (const T*)pairs, tokens, \
                          positions, seq_of_token, cu_seqlens, page_table, table_width, history, buckets, mul_prev, mul_cur,  \
-                         scale, out, width));                                                                                \
+                         scale, out, width, vec));                                                                           \
         return check_launch("embed_pairs");                                                                                  \
     }
 WICK_EMBED_PAIRS(wick_embed_pairs_bf16, bf16)
