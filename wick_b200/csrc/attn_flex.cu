@@ -285,15 +285,20 @@ attn_flex_kernel(const Params P) {
             bf16* op = P.out_bf16 + (t * P.heads + head) * DV + col;
             if (P.gate_parts) {
                 const float* gp = P.gate_parts + t * P.gate_cols + P.gate_col + head * DV + col;
+                float z[ND][2];                                 // (every block's loads of a partial sum are on their way together)
+#pragma unroll
+                for (int d = 0; d < ND; ++d) z[d][0] = gp[d * 8], z[d][1] = gp[d * 8 + 1];
+                for (int s = 1; s < P.gate_splits; ++s) {
+#pragma unroll
+                    for (int d = 0; d < ND; ++d) {
+                        z[d][0] += gp[s * P.gate_stride + d * 8];
+                        z[d][1] += gp[s * P.gate_stride + d * 8 + 1];
+                    }
+                }
 #pragma unroll
                 for (int d = 0; d < ND; ++d) {
-                    float z0 = gp[d * 8], z1 = gp[d * 8 + 1];
-                    for (int s = 1; s < P.gate_splits; ++s) {
-                        z0 += gp[s * P.gate_stride + d * 8];
-                        z1 += gp[s * P.gate_stride + d * 8 + 1];
-                    }
-                    o[d][2 * half] *= 1.0f / (1.0f + expf(-z0));
-                    o[d][2 * half + 1] *= 1.0f / (1.0f + expf(-z1));
+                    o[d][2 * half] *= 1.0f / (1.0f + expf(-z[d][0]));
+                    o[d][2 * half + 1] *= 1.0f / (1.0f + expf(-z[d][1]));
                 }
             }
 #pragma unroll
