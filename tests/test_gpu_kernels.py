@@ -726,3 +726,26 @@ def test_cuda_core_decode_attention_cuts_a_length_back_to_its_table(ops, dtype):
     want = ops.attention_decode(q, kv, fd_ok, 1 / math.sqrt(hd), scratch, max_kv_len=n)
     ops.check_status()
     assert torch.equal(out, want), "the first max_kv_len positions were attended to"
+
+
+def test_the_pair_product_behind_kernels_of_many_small_blocks():
+    """Hundreds of times in a row without a wait between: a kernel of 2,048 small blocks, then the product whose two blocks of
+    a pair share tensor memory and start some time apart behind it.  Every result is the first one's, bit for bit."""
+    from wick_b200 import ops as K
+    from wick_b200.ops import gemm_tc
+    g = torch.Generator(device="cuda").manual_seed(3)
+    n, ff, out = 2048, 1920, 1000
+    z = torch.randn((1, n, ff), generator=g, device="cuda")
+    co = torch.tensor([0.5, 0.3, 0.2, 0.1], device="cuda")
+    w = (0.02 * torch.randn((out, ff), generator=g, device="cuda")).to(torch.bfloat16)
+    plan = gemm_tc.plan_for(w)
+    first, same = None, torch.ones((), dtype=torch.bool, device="cuda")
+    for i in range(400):
+        y = plan.forward(K.poly_norm(z, co, 1e-5, torch.bfloat16), torch.float32)
+        if first is None:
+            first = y
+            ref = K.poly_norm(z, co, 1e-5, torch.bfloat16).float() @ w.float().T
+            assert (y - ref).abs().max() <= 2e-3 * ref.abs().max()
+        elif i % 50 == 0:
+            same &= (y == first).all()
+    assert bool(same)

@@ -128,13 +128,16 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
         }
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
-    if (warp == 1) {
+    // The pair allocates tensor memory together: the instruction of either block acts on both, so neither issues it before the
+    // other one runs.  (Issued earlier, it stopped the pair for good where the blocks of a pair started some time apart, behind a
+    // kernel of many small blocks.)
+    __syncthreads();
+    cluster_sync();
+    if (warp == 1)
         asm volatile("tcgen05.alloc.cta_group::2.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&tmem_base_slot)), "r"(tmem_cols));
-        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::2.sync.aligned;");
-    }
     tc_fence_before();
     __syncthreads();
-    cluster_sync();                            // the peer's barriers exist before anything arrives on them
+    cluster_sync();                            // both blocks hold their memory and barriers before anything is written to them
     tc_fence_after();
     const uint32_t tmem_base = tmem_base_slot;
     pdl_trigger();
@@ -296,6 +299,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
         while (global_ns() - t0 < 2000000ull) __nanosleep(1000);
         __syncthreads();
     }
+    if (warp == 1) asm volatile("tcgen05.relinquish_alloc_permit.cta_group::2.sync.aligned;");
     cluster_sync();                            // neither block leaves while the other may still read its shared memory
     if (warp == 1) {
         tc_fence_after();
