@@ -13,6 +13,8 @@
   (:func:`register_storage`): ``paged_kv`` groups [entries, pages, 2, kv_heads,
   64, head_dim]; ``paged_rows`` groups [entries, pages, 64, *shape], one row of
   fixed shape per position (a latent that keys and values are made from);
+  ``paged_blocks`` groups [entries, pages, kv_heads * rows * (head_dim + v_head_dim)], a key and a value for every
+  whole block of positions;
   ``state`` groups [entries, slots, *shape], a record of fixed
   size per sequence that is zeroed when the sequence opens.  All paged groups
   share the page ids (page p of a sequence is page p in each group).  Another
@@ -148,6 +150,30 @@ class PagedRows(Storage):
         return cached_tokens * self.bytes_per_token()
 
 
+class PagedBlocks(Storage):
+    """A key and a value for every whole block of the need's ``block`` positions, on the page that holds the block's last
+    position: [entries, pages, kv_heads * rows * (head_dim + v_head_dim)], a page [kv_heads, rows, head_dim] keys, then
+    [kv_heads, rows, v_head_dim] values, rows the most blocks that end on one page.  A mixer sees its entry's part as ``blocks``."""
+    kind = "paged_blocks"
+
+    def _page_elems(self) -> int:
+        n = self.need
+        return n.kv_heads * ((PAGE + n.block - 1) // n.block) * (n.head_dim + (n.head_dim if n.v_head_dim is None else n.v_head_dim))
+
+    def shape(self):
+        return (self.n_entries, self.n_pages, self._page_elems())
+
+    def view(self, idx, batch):
+        return CacheView(blocks=self.tensor[idx])
+
+    def bytes_per_token(self) -> float:
+        return self.n_entries * self._page_elems() * self.element_size() / PAGE
+
+    def read_bytes(self, cached_tokens, n_seqs):
+        n = self.need
+        return cached_tokens // n.block * self.n_entries * n.kv_heads * (n.head_dim + (n.head_dim if n.v_head_dim is None else n.v_head_dim)) * self.element_size()
+
+
 class StateRecords(Storage):
     """A record of fixed shape per sequence: [entries, slots, *shape], zero when a sequence starts."""
     kind = "state"
@@ -179,6 +205,7 @@ def register_storage(kind: str, cls: type) -> type:
 
 register_storage("paged_kv", PagedKV)
 register_storage("paged_rows", PagedRows)
+register_storage("paged_blocks", PagedBlocks)
 register_storage("state", StateRecords)
 
 
@@ -195,7 +222,7 @@ class _Group:
 
     def key(self):
         n = self.need
-        return (n.kind, n.kv_heads, n.head_dim, n.v_head_dim, n.window, tuple(n.shape), self.dtype)
+        return (n.kind, n.kv_heads, n.head_dim, n.v_head_dim, n.window, tuple(n.shape), n.block, self.dtype)
 
 
 class Cache:
@@ -244,7 +271,7 @@ class Cache:
     # ---- sizes -------------------------------------------------------------
     def bytes_per_token(self) -> int:
         """Bytes of keys and values that one cached position takes in all paged groups."""
-        return sum(g.store.bytes_per_token() for g in self.groups if isinstance(g.store, (PagedKV, PagedRows)))
+        return sum(g.store.bytes_per_token() for g in self.groups if isinstance(g.store, (PagedKV, PagedRows, PagedBlocks)))
 
     def read_bytes(self, cached_tokens: int, n_seqs: int) -> int:
         """Bytes one decode step reads from the cache: every group's share for ``n_seqs``

@@ -10,7 +10,9 @@
 //
 // Visible to the query at position p: the keys j <= p with p - j < window or j < keep_first (window 0:
 // every j <= p).  The tiles a block visits are those that hold kept first keys, then those of the
-// window of its rows.  A sink per head joins the denominator.  The result goes out in float32 (for a
+// window of its rows.  With blocks (block > 0) the query also sees the block b of `block` positions if
+// (b + 1) block <= p + 1 - window, as one key and value: tiles of 64 blocks per sequence in an array of pages that lie
+// like the sources' (which are then one paged source), visited first.  Scores may be soft-capped (cap tanh(s / cap)).  A sink per head joins the denominator.  The result goes out in float32 (for a
 // kernel that combines several maps) or in bfloat16 times a gate per (token, head) or per element (the sigmoid of a
 // column's sums).
 #include "common.cuh"
@@ -94,7 +96,20 @@ struct Params {
     const int *cu_seqlens, *start, *page_table;
     int n_seqs, table_width, n_tiles, heads, window, keep_first;
     float scale;
+    const bf16* pool;              // [n_seqs * pool_tiles] pages like the cache's, tile i of sequence b: page b * pool_tiles + i; or null
+    int pool_tiles, block;
+    float cap;                     // of the scores; 0: none
 };
+
+__device__ __forceinline__ int blocks_seen(int p, int window, int block) { return p + 1 > window ? (p + 1 - window) / block : 0; }
+// cap tanh(s / cap) = cap (1 - 2 / (1 + exp(2 s / cap)))
+__device__ __forceinline__ float soft_capped(float s, float two_over_cap, float cap) {
+    return cap * (1.0f - __fdividef(2.0f, 1.0f + __expf(s * two_over_cap)));
+}
+
+__device__ __forceinline__ const bf16* pool_tile_of(const Source& s, const Params& P, int hv, int b, int i) {
+    return P.pool + (int64_t)(b * P.pool_tiles + i) * s.tile_elems + s.const_off + (int64_t)(hv / s.hdiv) * s.hmul + (int64_t)(hv % s.hmod) * s.hmul2;
+}
 
 __global__ void __launch_bounds__(128, MIN_BLOCKS)
 attn_flex_kernel(const Params P) {
@@ -120,15 +135,18 @@ attn_flex_kernel(const Params P) {
     const int kt_lo = window > 0 ? max(0, p_first - window + 1) / kPage : 0;
     const int kt_hi = p_last / kPage;
     const int n_kept = min(kt_lo, (keep + kPage - 1) / kPage);
-    const int n_visit = n_kept + (kt_hi - kt_lo + 1);
-    auto tile_index = [&](int i) { return i < n_kept ? i : kt_lo + (i - n_kept); };
+    // (before them those with blocks that the last row sees)
+    const int n_pool = P.pool ? (blocks_seen(p_last, window, P.block) + kPage - 1) / kPage : 0;
+    const int n_visit = n_pool + n_kept + (kt_hi - kt_lo + 1);
+    auto tile_index = [&](int i) { return i < n_pool ? i : (i - n_pool < n_kept ? i - n_pool : kt_lo + (i - n_pool - n_kept)); };
 
     auto load_tiles = [&](int i) {
         const int kt = tile_index(i), buf = i & 1;
-        const int valid = kv_len - kt * kPage;                  // rows of the tile that hold a token
-        const bf16* p0 = tile_of(P.k0, head, b, tok0, kt, P.page_table, P.table_width);
+        const bool blocks = i < n_pool;
+        const int valid = blocks ? kPage : kv_len - kt * kPage; // rows of the tile that hold a token (places without a block hold zeros)
+        const bf16* p0 = blocks ? pool_tile_of(P.k0, P, head, b, kt) : tile_of(P.k0, head, b, tok0, kt, P.page_table, P.table_width);
         const bf16* p1 = P.k1.len ? tile_of(P.k1, head, b, tok0, kt, P.page_table, P.table_width) : nullptr;
-        const bf16* pv = tile_of(P.v, head, b, tok0, kt, P.page_table, P.table_width);
+        const bf16* pv = blocks ? pool_tile_of(P.v, P, head, b, kt) : tile_of(P.v, head, b, tok0, kt, P.page_table, P.table_width);
         bf16* kd = Ks + buf * kPage * DK;
         bf16* vd = Vs + buf * kPage * DV;
         const int c0 = P.k0.len >> 3;
@@ -159,6 +177,7 @@ attn_flex_kernel(const Params P) {
     const int pos_lo = s0 + q0 + min(r_lo, rows - 1), pos_hi = s0 + q0 + min(r_lo + 8, rows - 1);
     const int vis_lo = window > 0 ? pos_lo - window + 1 : 0, vis_hi = window > 0 ? pos_hi - window + 1 : 0;   // first key of the window
     const float sl2 = P.scale * 1.4426950408889634f;            // scores in units of log2(e)
+    const float two_over_cap = P.cap > 0.f ? 2.0f / P.cap : 0.f, cap2 = P.cap * 1.4426950408889634f;
     const float sink2 = P.sink ? P.sink[head] * 1.4426950408889634f : -INFINITY;
 
     float o[ND][4];
@@ -199,15 +218,26 @@ attn_flex_kernel(const Params P) {
         }
         // ---- mask, running maximum, probabilities ----
         const int key0 = kt * kPage + (lane & 3) * 2;
+        const bool blocks = i < n_pool;
+        // keys a row sees of this tile: first .. last (or below keep)
+        const int last_lo = blocks ? blocks_seen(pos_lo, window, P.block) - 1 : pos_lo, last_hi = blocks ? blocks_seen(pos_hi, window, P.block) - 1 : pos_hi;
+        const int first_lo = blocks ? 0 : vis_lo, first_hi = blocks ? 0 : vis_hi;
         float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
         for (int nb = 0; nb < 8; ++nb) {
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = key0 + nb * 8 + e;
-                float a = s[nb][e] * sl2, c = s[nb][2 + e] * sl2;
-                if (key > pos_lo || (key < vis_lo && key >= keep)) a = -INFINITY;
-                if (key > pos_hi || (key < vis_hi && key >= keep)) c = -INFINITY;
+                float a = s[nb][e], c = s[nb][2 + e];
+                if (P.cap > 0.f) {
+                    a = soft_capped(a * P.scale, two_over_cap, cap2);
+                    c = soft_capped(c * P.scale, two_over_cap, cap2);
+                } else {
+                    a *= sl2;
+                    c *= sl2;
+                }
+                if (key > last_lo || (key < first_lo && key >= keep)) a = -INFINITY;
+                if (key > last_hi || (key < first_hi && key >= keep)) c = -INFINITY;
                 s[nb][e] = a;
                 s[nb][2 + e] = c;
                 mx_lo = fmaxf(mx_lo, a);
@@ -351,7 +381,8 @@ WICK_API int wick_attn_flex_sizes(int* dk, int* dv) {
 WICK_API int wick_attn_flex_bf16(const void* q, const int64_t* src, void* out_f32, void* out_bf16, const float* gate, const float* sink,
                                  const int* cu_seqlens, int n_seqs, const int* start, const int* page_table, int table_width,
                                  int n_tiles, int heads, int window, int keep_first, float scale, const float* gate_parts, int gate_splits,
-                                 int64_t gate_stride, int gate_cols, int gate_col, void* s) {
+                                 int64_t gate_stride, int gate_cols, int gate_col, const void* pool, int pool_tiles, int block, float cap,
+                                 void* s) {
     using namespace flex;
     Params P;
     P.q = (const bf16*)q;
@@ -383,6 +414,9 @@ WICK_API int wick_attn_flex_bf16(const void* q, const int64_t* src, void* out_f3
     P.cu_seqlens = cu_seqlens; P.start = start; P.page_table = page_table;
     P.n_seqs = n_seqs; P.table_width = table_width; P.n_tiles = n_tiles; P.heads = heads; P.window = window; P.keep_first = keep_first;
     P.scale = scale;
+    WICK_REQUIRE(!pool || (((uintptr_t)pool & 15) == 0 && window > 0 && block > 0 && pool_tiles > 0 && P.k0.paged && P.v.paged && P.k1.len == 0 &&
+                           P.k0.tile_elems == P.v.tile_elems), "attn_flex: blocks need a window and one paged source");
+    P.pool = (const bf16*)pool; P.pool_tiles = pool_tiles; P.block = block; P.cap = cap;
     if (n_tiles == 0) return 0;
     const size_t smem = ((size_t)(QT + 2 * kPage) * DK + 2 * kPage * DV) * sizeof(bf16);
     static bool raised = false;

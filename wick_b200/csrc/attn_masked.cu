@@ -1,4 +1,5 @@
-// Attention with options, for any head sizes (run-time numbers): projection biases, an
+// Attention with options, for any head sizes (run-time numbers): projection biases, short
+// filters over time, values of unit root mean square, gates per head, an
 // RMS norm of q and k over spans of any length (a head, or the whole projection), a
 // rotation of neighbouring or of half-split pairs over the first dims of each head, values
 // blended with the values another layer made for the same token, key and value heads of
@@ -13,6 +14,7 @@
 // Scores, the softmax, its weights and the weighted sum are float32.  A token's work is the
 // same whatever else the step holds, up to the number of warps that share its keys.
 #include "common.cuh"
+#include "short_conv.cuh"
 
 namespace wick {
 
@@ -41,6 +43,51 @@ __device__ __forceinline__ int first_visible(int p, int mask, int size) {
 //   A span without a weight vector (q_span > 0, q_w null) is divided by its root mean square and no more.
 constexpr int FINISH_KEYS_ARE_VALUES = 1, FINISH_NORM_AFTER = 2;
 constexpr int MAX_SPANS = 512;                  // spans of the two norms together (a span per head at most)
+constexpr int MAX_V_HEADS = 256;                // value heads that the values' norm takes
+
+// What some attentions do besides.
+//   conv_w  : [taps][W] or null: the row is a causal filter over time of what was projected, channel by channel, the inputs
+//             before this token from the sequence's record ([taps - 1][W], oldest first), which moves on by this token (steps
+//             of one token per sequence only; a longer step runs the filter as a kernel of its own)
+//   v_norm  : every head's values are divided by their root mean square (v_eps inside the root)
+//   gate_out: [n, gate_heads], the sigmoids of the columns from gate_col on of gate_parts (sums laid out like parts, gate_cols a row)
+//   pool    : (steps of one token per sequence only) the token that completes a block of `block` positions leaves the block's mean key
+//             and value, of the numbers as the cache holds them: pages of pool_page elements, [G][rows][d] keys, then [G][rows][e]
+//             values, a block on the page of its last position
+template <typename T>
+struct FinishExtra {
+    const float* conv_w;
+    float* conv_rec;
+    int64_t record;
+    const int* slots;
+    int taps, v_norm;
+    float v_eps;
+    float* gate_out;
+    const float* gate_parts;
+    int gate_splits, gate_cols, gate_col, gate_heads;
+    T* pool;
+    int block, rows;
+    int64_t pool_page;
+};
+
+// Where block b of `block` positions lies: on the page that holds its last position, at this place.
+__device__ __forceinline__ int block_place(int b, int block, int page) { return b - (int)((int64_t)page * kPage / block); }
+
+// Element c of the block's mean (c counts the G d key numbers, then the G e value numbers) over positions first .. first + block - 1.
+template <typename T>
+__device__ __forceinline__ float block_mean(const T* kv, const int* table, int G, int d, int e, int first, int block, int c) {
+    const int64_t page_elems = (int64_t)G * kPage * (d + e);
+    const bool key = c < G * d;
+    const int size = key ? d : e, i = key ? c : c - G * d, g = i / size, x = i - g * size;
+    const T* at = kv + (key ? 0 : (int64_t)G * kPage * d) + (int64_t)g * kPage * size + x;
+    float sum = 0.f;
+#pragma unroll 8
+    for (int j = 0; j < block; ++j) {
+        const int p = first + j;
+        sum += ld(at + table[p / kPage] * page_elems + (int64_t)(p % kPage) * size);
+    }
+    return sum / (float)block;
+}
 
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -49,9 +96,10 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
                   int k_span, float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot_dims,
                   int pairing, int maps, float* __restrict__ v_keep, int v_mode, const float* __restrict__ lambda, T* __restrict__ q_out,
                   T* __restrict__ kv, const int* __restrict__ page_table, int table_width,
-                  const int* __restrict__ seq_of_token, const int* __restrict__ positions, int write_kv, int cols, int flags) {
+                  const int* __restrict__ seq_of_token, const int* __restrict__ positions, int write_kv, int cols, int flags,
+                  const FinishExtra<T> X) {
     extern __shared__ float row[];
-    __shared__ float partial[MAX_SPANS], span_scale[MAX_SPANS];
+    __shared__ float partial[MAX_SPANS], span_scale[MAX_SPANS], v_scale[MAX_V_HEADS];
     pdl_trigger();
     pdl_wait();
     parts = fresh(parts);
@@ -61,7 +109,8 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
     const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
     const bool keys_are_values = flags & FINISH_KEYS_ARE_VALUES, norm_after = flags & FINISH_NORM_AFTER;
     const int Wq = H * d, Wk = G * d, Wv = G * e, W = Wq + Wk + (keys_are_values ? 0 : Wv);
-    if ((W & 3) == 0 && (cols & 3) == 0 && (split_stride & 3) == 0) {
+    float* rec = X.conv_w ? X.conv_rec + (int64_t)X.slots[seq_of_token[t]] * X.record : nullptr;
+    if ((W & 3) == 0 && (cols & 3) == 0 && (split_stride & 3) == 0 && (X.record & 3) == 0) {
         // four neighbours a load, the loads of four partial sums issued together (a chain of dependent trips to
         // the L2 cache is what a step of few tokens would otherwise wait for); the sums in index order
         for (int j = tid * 4; j < W; j += blockDim.x * 4) {
@@ -80,6 +129,17 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
             if (bias) {
                 v.x += bias[j]; v.y += bias[j + 1]; v.z += bias[j + 2]; v.w += bias[j + 3];
             }
+            if (rec) {                           // (a place's old input moves one place down: read before it is written over)
+                float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 3
+                for (int k = 0; k < X.taps; ++k) {
+                    const float4 u = k < X.taps - 1 ? *reinterpret_cast<const float4*>(rec + (int64_t)k * W + j) : v;
+                    const float4 w = *reinterpret_cast<const float4*>(X.conv_w + (int64_t)k * W + j);
+                    if (k > 0) *reinterpret_cast<float4*>(rec + (int64_t)(k - 1) * W + j) = u;
+                    y.x = fmaf(w.x, u.x, y.x); y.y = fmaf(w.y, u.y, y.y); y.z = fmaf(w.z, u.z, y.z); y.w = fmaf(w.w, u.w, y.w);
+                }
+                v = y;
+            }
             *reinterpret_cast<float4*>(row + j) = v;
         }
     } else {
@@ -87,10 +147,35 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
             float v = parts[(int64_t)t * cols + j];
             for (int s = 1; s < splits; ++s) v += parts[s * split_stride + (int64_t)t * cols + j];
             if (bias) v += bias[j];
+            if (rec) {
+                float y = 0.f;
+                for (int k = 0; k < X.taps; ++k) {
+                    const float u = k < X.taps - 1 ? rec[(int64_t)k * W + j] : v;
+                    if (k > 0) rec[(int64_t)(k - 1) * W + j] = u;
+                    y = fmaf(X.conv_w[(int64_t)k * W + j], u, y);
+                }
+                v = y;
+            }
             row[j] = v;
         }
     }
+    for (int j = tid; j < X.gate_heads; j += blockDim.x) {
+        float z = 0.f;
+        for (int s = 0; s < X.gate_splits; ++s)
+            z += X.gate_parts[((int64_t)s * gridDim.x + t) * X.gate_cols + X.gate_col + j];
+        X.gate_out[(int64_t)t * X.gate_heads + j] = 1.0f / (1.0f + expf(-z));
+    }
     __syncthreads();
+    if (X.v_norm) {                                        // a warp per head
+        for (int g = warp; g < G; g += n_warps) {
+            const float* p = row + (keys_are_values ? Wq : Wq + Wk) + g * e;
+            float ss = 0.f;
+            for (int x = lane; x < e; x += 32) ss = fmaf(p[x], p[x], ss);
+            ss = warp_sum(ss);
+            if (lane == 0) v_scale[g] = 1.0f / sqrtf(ss / (float)e + X.v_eps);
+        }
+        __syncthreads();
+    }
     const int pos = positions[t];
     const float lam = v_mode == 2 ? *lambda : 0.f;
     T* page = nullptr;
@@ -104,6 +189,7 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
     // The values first (they read the row as projected): blended where asked, then stored.
     for (int j = tid; j < Wv; j += blockDim.x) {
         float v = row[(keys_are_values ? Wq : Wq + Wk) + j];
+        if (X.v_norm) v *= v_scale[j / e];
         if (v_mode == 1) v_keep[(int64_t)t * Wv + j] = v;
         if (v_mode == 2) v = (1.0f - lam) * v + lam * v_keep[(int64_t)t * Wv + j];
         if (write_kv) {
@@ -191,6 +277,55 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
             st(o + j0, u);
             if (two) st(o + j1, v);
         }
+    }
+    if (X.pool && (pos + 1) % X.block == 0) {
+        __syncthreads();                                   // (the token's own key and value are in the cache)
+        const int* table = page_table + (int64_t)seq_of_token[t] * table_width;
+        const int b = pos / X.block, pg = pos / kPage;
+        T* dst = X.pool + table[pg] * X.pool_page;
+        const int at = block_place(b, X.block, pg);
+        for (int c = tid; c < Wk + Wv; c += blockDim.x) {
+            const bool key = c < Wk;
+            const int size = key ? d : e, i = key ? c : c - Wk, g = i / size;
+            st(dst + (key ? 0 : (int64_t)G * X.rows * d) + ((int64_t)g * X.rows + at) * size + (i - g * size),
+               block_mean(kv, table, G, d, e, pos - X.block + 1, X.block, c));
+        }
+    }
+}
+
+// The blocks of `block` positions that a step completes: their mean keys and values go to the store (as above), and, with
+// `flat`, so do all blocks the sequences' tokens can see to arrays whose tiles of 64 blocks lie like cache pages: tile i of sequence b is
+// page b * flat_tiles + i of [G][64][d] keys, then [G][64][e] values (places beyond a sequence's whole blocks hold zeros).
+// grid (most blocks of a sequence, sequences).
+template <typename T>
+__global__ void __launch_bounds__(256)
+pool_blocks_kernel(const T* __restrict__ kv, T* store, T* __restrict__ flat, const int* __restrict__ page_table, int table_width,
+                   const int* __restrict__ start, const int* __restrict__ kv_len, int G, int d, int e, int block, int rows,
+                   int64_t pool_page, int flat_tiles) {
+    pdl_trigger();
+    pdl_wait();
+    kv = fresh(kv);
+    const int blk = blockIdx.x, b = blockIdx.y, Wk = G * d, W = G * (d + e);
+    const int* table = page_table + (int64_t)b * table_width;
+    const int last = blk * block + block - 1;
+    const bool whole = last < kv_len[b], old = last < start[b];
+    if (!flat && (!whole || old)) return;
+    const int pg = last / kPage;
+    T* dst = whole ? store + table[pg] * pool_page : nullptr;
+    T* out = flat ? flat + (int64_t)(b * flat_tiles + blk / kPage) * W * kPage : nullptr;
+    const int at = block_place(blk, block, pg);
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+        const bool key = c < Wk;
+        const int size = key ? d : e, i = key ? c : c - Wk, g = i / size, x = i - g * size;
+        T* s = whole ? dst + (key ? 0 : (int64_t)G * rows * d) + ((int64_t)g * rows + at) * size + x : nullptr;
+        float v = 0.f;
+        if (whole && !old) {
+            v = block_mean(kv, table, G, d, e, blk * block, block, c);
+            st(s, v);
+        } else if (whole) {
+            v = ld(s);
+        }
+        if (out) st(out + (key ? 0 : (int64_t)G * kPage * d) + ((int64_t)g * kPage + blk % kPage) * size + x, v);
     }
 }
 
@@ -521,7 +656,8 @@ template <typename T>
 int qkv_finish(const float* parts, int splits, int n, const float* bias, int H, int G, int d, int e, const float* q_w,
                int q_span, const float* k_w, int k_span, float eps, const float* cos_t, const float* sin_t, int rot_dims,
                int pairing, int maps, float* v_keep, int v_mode, const float* lambda, void* q_out, void* kv, const int* page_table,
-               int table_width, const int* seq_of_token, const int* positions, int write_kv, int cols, int flags, cudaStream_t s) {
+               int table_width, const int* seq_of_token, const int* positions, int write_kv, int cols, int flags, const FinishExtra<T>& X,
+               cudaStream_t s) {
     WICK_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && e > 0, "qkv_finish: bad head counts or sizes");
     WICK_REQUIRE(!(flags & FINISH_KEYS_ARE_VALUES) || (d == e && v_mode == 0), "qkv_finish: keys that are values have the values' size and are not blended");
     WICK_REQUIRE(cols >= H * d + G * d + ((flags & FINISH_KEYS_ARE_VALUES) ? 0 : G * e), "qkv_finish: rows of %d numbers are too short", cols);
@@ -535,6 +671,13 @@ int qkv_finish(const float* parts, int splits, int n, const float* bias, int H, 
     WICK_REQUIRE((q_span ? Wq / q_span : 0) + (k_span ? Wk / k_span : 0) <= MAX_SPANS, "qkv_finish: too many norm spans");
     WICK_REQUIRE(v_mode == 0 || v_keep, "qkv_finish: the kept values are missing");
     WICK_REQUIRE(v_mode != 2 || lambda, "qkv_finish: the blend factor is missing");
+    WICK_REQUIRE(!X.v_norm || G <= MAX_V_HEADS, "qkv_finish: the values' norm takes up to %d heads", MAX_V_HEADS);
+    WICK_REQUIRE(!X.conv_w || (X.taps >= 1 && X.slots && (X.taps == 1 || X.conv_rec) && !(flags & FINISH_KEYS_ARE_VALUES) &&
+                               X.record >= (int64_t)(X.taps - 1) * (Wq + Wk + G * e)), "qkv_finish: bad filter");
+    WICK_REQUIRE(X.gate_heads == 0 || (X.gate_out && X.gate_parts && X.gate_splits >= 1 && X.gate_col >= 0 && X.gate_col + X.gate_heads <= X.gate_cols),
+                 "qkv_finish: bad gate columns");
+    WICK_REQUIRE(!X.pool || (write_kv && X.block > 0 && X.rows == (kPage + X.block - 1) / X.block && X.pool_page == (int64_t)G * X.rows * (d + e)),
+                 "qkv_finish: bad blocks");
     if (n == 0) return 0;
     const size_t smem = (size_t)(Wq + Wk + G * e) * sizeof(float);
     WICK_REQUIRE(smem <= 200 * 1024, "qkv_finish: a row of %d numbers is beyond one block's shared memory", Wq + Wk + G * e);
@@ -545,7 +688,7 @@ int qkv_finish(const float* parts, int splits, int n, const float* bias, int H, 
     }
     WICK_CUDA(launch(qkv_finish_kernel<T>, dim3(n), dim3(256), smem, s, parts, splits, (int64_t)n * cols, bias, H, G,
                      d, e, q_w, q_span, k_w, k_span, eps, cos_t, sin_t, rot_dims, pairing, maps, v_keep, v_mode, lambda, (T*)q_out,
-                     (T*)kv, page_table, table_width, seq_of_token, positions, write_kv, cols, flags));
+                     (T*)kv, page_table, table_width, seq_of_token, positions, write_kv, cols, flags, X));
     return check_launch("qkv_finish");
 }
 
@@ -595,10 +738,14 @@ typedef __nv_bfloat16 bf16;
                       int q_span, const float* k_w, int k_span, float eps, const float* cos_t, const float* sin_t,               \
                       int rot_dims, int pairing, int maps, float* v_keep, int v_mode, const float* lambda, void* q_out, void* kv, \
                       const int* page_table, int table_width, const int* seq_of_token, const int* positions, int write_kv,       \
-                      int cols, int flags, void* s) {                                                                            \
+                      int cols, int flags, const float* conv_w, float* conv_rec, int64_t record, const int* slots, int taps,     \
+                      int v_norm, float v_eps, float* gate_out, const float* gate_parts, int gate_splits, int gate_cols,         \
+                      int gate_col, int gate_heads, void* pool, int block, int rows, int64_t pool_page, void* s) {                \
+        const FinishExtra<T> X = {conv_w, conv_rec, record, slots, taps, v_norm, v_eps, gate_out, gate_parts, gate_splits, gate_cols, \
+                                  gate_col, gate_heads, (T*)pool, block, rows, pool_page};                                       \
         return qkv_finish<T>(parts, splits, n, bias, H, G, d, e, q_w, q_span, k_w, k_span, eps, cos_t, sin_t, rot_dims, pairing,  \
                              maps, v_keep, v_mode, lambda, q_out, kv, page_table, table_width, seq_of_token, positions, write_kv,      \
-                             cols, flags, (cudaStream_t)s);                                                                      \
+                             cols, flags, X, (cudaStream_t)s);                                                                   \
     }
 WICK_QKV_FINISH(wick_qkv_finish_bf16, bf16)
 WICK_QKV_FINISH(wick_qkv_finish_f32, float)
@@ -612,3 +759,41 @@ WICK_QKV_FINISH(wick_qkv_finish_f32, float)
     }
 WICK_ATTN_MASKED(wick_attn_masked_bf16, bf16)
 WICK_ATTN_MASKED(wick_attn_masked_f32, float)
+
+// parts: float32 [splits, n, cols]; w: float32 [taps, channels]; records: float32 [slots, record], the last taps - 1 inputs, oldest
+// first; out: float32 [n, channels], the filtered first `channels` columns.  The records are brought up to date.
+WICK_API int wick_short_conv(const float* parts, int splits, int n, int cols, int channels, int taps, const float* w, float* records,
+                             int64_t record, const int* slots, int n_seqs, const int* cu_seqlens, const int* start,
+                             const int* seq_of_token, const int* positions, float* out, void* stream) {
+    cudaStream_t s = (cudaStream_t)stream;
+    WICK_REQUIRE(splits >= 1 && channels > 0 && channels <= cols, "short_conv: bad sizes");
+    WICK_REQUIRE(taps >= 1 && taps <= CONV_MAX_TAPS, "short_conv: %d taps (1 .. %d are built)", taps, CONV_MAX_TAPS);
+    WICK_REQUIRE(taps == 1 || (records && record >= (int64_t)(taps - 1) * channels), "short_conv: records of another size");
+    if (n == 0 || n_seqs == 0) return 0;
+    const int64_t stride = (int64_t)n * cols;
+    auto kernel = splits == 1 ? short_conv_kernel<true, false> : short_conv_kernel<false, false>;
+    WICK_CUDA(launch(kernel, dim3(ceil_div(n, CONV_TOKENS), ceil_div(channels, 256)), dim3(256), 0, s, parts, splits, stride, cols, 0, channels,
+                     taps, w, 1, channels, (const float*)nullptr, (const float*)records, record, slots, seq_of_token, positions, start, out, n));
+    if (check_launch("short_conv")) return 1;
+    if (taps > 1) {
+        WICK_CUDA(launch(short_conv_state_kernel, dim3(n_seqs, ceil_div(channels, 256)), dim3(256), 0, s, parts, splits, stride, cols, 0,
+                         channels, taps, records, record, slots, cu_seqlens));
+        if (check_launch("short_conv_state")) return 1;
+    }
+    return 0;
+}
+
+#define WICK_POOL_BLOCKS(NAME, T)                                                                                             \
+    WICK_API int NAME(const void* kv, void* store, void* flat, const int* page_table, int table_width, const int* start,        \
+                      const int* kv_len, int n_seqs, int G, int d, int e, int block, int rows, int64_t pool_page, int blocks,  \
+                      int flat_tiles, void* s) {                                                                               \
+        WICK_REQUIRE(G > 0 && d > 0 && e > 0 && block > 0 && rows == (kPage + block - 1) / block &&                            \
+                     pool_page == (int64_t)G * rows * (d + e), "pool_blocks: bad sizes");                                      \
+        WICK_REQUIRE(n_seqs <= 65535 && (!flat || blocks == flat_tiles * kPage), "pool_blocks: bad numbers of blocks");        \
+        if (n_seqs == 0 || blocks == 0) return 0;                                                                              \
+        WICK_CUDA(launch(pool_blocks_kernel<T>, dim3(blocks, n_seqs), dim3(256), 0, (cudaStream_t)s, (const T*)kv, (T*)store, (T*)flat, \
+                         page_table, table_width, start, kv_len, G, d, e, block, rows, pool_page, flat_tiles));                 \
+        return check_launch("pool_blocks");                                                                                    \
+    }
+WICK_POOL_BLOCKS(wick_pool_blocks_bf16, bf16)
+WICK_POOL_BLOCKS(wick_pool_blocks_f32, float)

@@ -6,6 +6,9 @@
 //              map a scores the a-th dm numbers of the key row, has a softmax of its own, and
 //              weighs the SAME value rows.  Visible keys of the query at position p: with a
 //              window, the keys j <= p with p - j < window or j < keep_first; else every j <= p.
+//              Before these, the blocks of `block` positions that lie wholly before the window may
+//              be seen too, each as one key and one value from a store of its own.  Scores may be
+//              soft-capped, s <- cap tanh(s / cap); a result may be multiplied by a number per head.
 //              A sink per head joins a map's denominator.  MAPS = 2 ends with
 //              y = y_1 - lambda y_2, y / sqrt(mean(y^2) + eps) * factor over the head's values.
 //              Where a key row and a value row lie in a page is given by strides, so the same
@@ -37,6 +40,44 @@ __device__ __forceinline__ void mv_load4(const __nv_bfloat16* p, float* v) {
 
 // The v-th visible key (v counts the kept first keys, then the window).
 __device__ __forceinline__ int visible_key(int v, int n_kept, int lo) { return v < n_kept ? v : lo + (v - n_kept); }
+
+// What some attentions do besides: blocks of positions that are seen as one key and value once they lie before the window
+// (block 0: none; rows: places of a page's blocks, see block_place), a soft cap of the scores (0: none), a factor per
+// (token, head) of the result (null: none).
+template <typename T>
+struct MultiExtra {
+    const T* pool;
+    int block, rows;
+    int64_t page_elems, v_off;
+    float cap;
+    const float* gate;                          // [n, H]
+};
+
+// How many blocks the query at position p sees: those whose last position is at most p - window.
+__device__ __forceinline__ int blocks_seen(int p, int window, int block) {
+    return block > 0 && p + 1 > window ? (p + 1 - window) / block : 0;
+}
+
+// A key's two rows, for the v-th visible key of the query at hand (first the blocks, then the kept keys, then the window).
+template <typename T>
+struct KeyRows {
+    const T *k, *v;
+};
+template <typename T>
+__device__ __forceinline__ KeyRows<T> key_rows(int vi, int n_blocks, int n_kept, int lo, const T* store, const int* table, int64_t page_elems,
+                                               int g, int k_row, int64_t v_off, int v_row, const MultiExtra<T>& X) {
+    if (vi < n_blocks) {
+        const int page = (vi * X.block + X.block - 1) / kPage;
+        const int64_t place = (int64_t)g * X.rows + (vi - (int)((int64_t)page * kPage / X.block));
+        const T* at = X.pool + table[page] * X.page_elems;
+        return {at + place * k_row, at + X.v_off + place * v_row};
+    }
+    const int key = visible_key(vi - n_blocks, n_kept, lo);
+    const int64_t place = (int64_t)g * kPage + (key % kPage);
+    const T* at = store + table[key / kPage] * page_elems;
+    return {at + place * k_row, at + v_off + place * v_row};
+}
+__device__ __forceinline__ float soft_capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
 
 // One block per (token, GROUP query heads, run of the visible keys); its warps share the run's keys, 32 at a
 // time.  A block holds NQ = GROUP * MAPS query vectors of dm numbers ([head][map][dm], as they lie in memory); all
@@ -73,7 +114,7 @@ __device__ __forceinline__ void finish_head(float (&y)[MAPS][4 * MV_CHUNKS], int
 template <typename TO, int MAPS, int GROUP, int MV_CHUNKS>
 __device__ __forceinline__ void fold_warps(float (&m)[MAPS * GROUP], float (&l)[MAPS * GROUP], float (&acc)[MAPS * GROUP][4 * MV_CHUNKS],
                                            float* ms, float* accs, TO* __restrict__ out, float* __restrict__ partial, int t, int h0,
-                                           int H, int e, const float* __restrict__ sink, float lam, float eps, float factor) {
+                                           int H, int e, const float* __restrict__ sink, float lam, float eps, float factor, const float* gate) {
     constexpr int NQ = MAPS * GROUP;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
     const int e_pad = (e + 127) / 128 * 128;
@@ -127,7 +168,8 @@ __device__ __forceinline__ void fold_warps(float (&m)[MAPS * GROUP], float (&l)[
                     if (128 * c < e_pad) *reinterpret_cast<float4*>(rec + 4 + 128 * c + 4 * lane) =
                         make_float4(y[a][4 * c], y[a][4 * c + 1], y[a][4 * c + 2], y[a][4 * c + 3]);
             } else {
-                const float inv = 1.0f / sum;    // (the block holds a visible key: the sum is positive)
+                float inv = 1.0f / sum;          // (the block holds a visible key: the sum is positive)
+                if (gate) inv *= gate[(int64_t)t * H + h];
 #pragma unroll
                 for (int c = 0; c < 4 * MV_CHUNKS; ++c) y[a][c] *= inv;
             }
@@ -151,7 +193,7 @@ attn_multi_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO* __r
                   const int* __restrict__ seq_of_token, const int* __restrict__ positions,
                   const int* __restrict__ page_table, int table_width, int H, int G, int dm, int e, int64_t page_elems,
                   int k_row, int64_t v_off, int v_row, float scale, int window, int keep_first,
-                  const float* __restrict__ sink, float lam, float eps, float factor) {
+                  const float* __restrict__ sink, float lam, float eps, float factor, const MultiExtra<T> X) {
     constexpr int NQ = MAPS * GROUP;
     extern __shared__ __align__(16) float smem[];
     pdl_trigger();
@@ -171,12 +213,13 @@ attn_multi_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO* __r
     for (int x = threadIdx.x; x < dq; x += blockDim.x) qs[x] = ld(q + ((int64_t)t * H + h0) * (MAPS * dm) + x);
     __syncthreads();
     constexpr int VN = Vec16<T>::N;
-    const bool base_ok = (((uintptr_t)store) & 15) == 0;
+    const bool base_ok = (((uintptr_t)store) & 15) == 0 && (X.block == 0 || ((((uintptr_t)X.pool) & 15) == 0 && X.page_elems % VN == 0 && X.v_off % VN == 0));
     const bool k_vec = base_ok && dm % VN == 0 && k_row % VN == 0 && page_elems % VN == 0;
     const bool v_vec = base_ok && e % 4 == 0 && v_row % 4 == 0 && page_elems % 4 == 0 && v_off % 4 == 0;
     const int lo = window > 0 ? max(0, pos - window + 1) : 0;
     const int n_kept = window > 0 ? min(keep_first, lo) : 0;
-    const int total = n_kept + (pos - lo + 1);
+    const int n_blocks = blocks_seen(pos, window, X.block);
+    const int total = n_blocks + n_kept + (pos - lo + 1);
     // this block's run of tiles
     const int tiles = (total + 31) >> 5, per_run = (tiles + (int)gridDim.y - 1) / (int)gridDim.y;
     const int v_begin = 32 * per_run * (int)blockIdx.y, v_end = min(total, 32 * per_run * ((int)blockIdx.y + 1));
@@ -195,11 +238,10 @@ attn_multi_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO* __r
 #pragma unroll
         for (int a = 0; a < NQ; ++a) s[a] = 0.f;
         // where this lane's key row and value row lie (lanes beyond the run's end name its last key and weigh nothing)
-        const int key = visible_key(min(vi, v_end - 1), n_kept, lo);
-        const int64_t in_page = (int64_t)table[key / kPage] * page_elems, place = (int64_t)g * kPage + (key % kPage);
-        const int64_t v_at = in_page + v_off + place * v_row;
+        const KeyRows<T> rows = key_rows(min(vi, v_end - 1), n_blocks, n_kept, lo, store, table, page_elems, g, k_row, v_off, v_row, X);
+        const unsigned long long v_at = (unsigned long long)(uintptr_t)rows.v;
         if (valid) {
-            const T* kp = store + in_page + place * k_row;
+            const T* kp = rows.k;
 #pragma unroll
             for (int a = 0; a < MAPS; ++a) {
                 const T* ka = kp + a * dm;
@@ -240,7 +282,7 @@ attn_multi_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO* __r
         }
 #pragma unroll
         for (int a = 0; a < NQ; ++a) {
-            s[a] = valid ? s[a] * scale : -INFINITY;
+            s[a] = valid ? soft_capped(s[a] * scale, X.cap) : -INFINITY;
             const float m_new = fmaxf(m[a], warp_max(s[a]));         // finite: the tile's first key is visible
             const float corr = expf(m[a] - m_new);                   // (m = -inf at first: 0)
             p[a] = valid ? expf(s[a] - m_new) : 0.f;
@@ -256,7 +298,7 @@ attn_multi_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO* __r
 #pragma unroll 4
         for (int jj = 0; jj < 32; ++jj) {
             if (jj >= n_keys) break;
-            const T* vp = store + __shfl_sync(0xffffffffu, v_at, jj);
+            const T* vp = (const T*)(uintptr_t)__shfl_sync(0xffffffffu, v_at, jj);
             float pj[NQ];
 #pragma unroll
             for (int a = 0; a < NQ; ++a) pj[a] = __shfl_sync(0xffffffffu, p[a], jj);
@@ -279,7 +321,7 @@ attn_multi_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO* __r
             }
         }
     }
-    fold_warps<TO, MAPS, GROUP, MV_CHUNKS>(m, l, acc, ms, accs, out, partial, t, h0, H, e, sink, lam, eps, factor);
+    fold_warps<TO, MAPS, GROUP, MV_CHUNKS>(m, l, acc, ms, accs, out, partial, t, h0, H, e, sink, lam, eps, factor, X.gate);
 }
 
 // The form for steps of few tokens where rows can be copied 16 bytes at a time: one block per (token, GROUP heads, run
@@ -306,7 +348,7 @@ attn_multi_tile_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO
                        const int* __restrict__ seq_of_token, const int* __restrict__ positions,
                        const int* __restrict__ page_table, int table_width, int H, int G, int dm, int e, int64_t page_elems,
                        int k_row, int64_t v_off, int v_row, float scale, int window, int keep_first,
-                       const float* __restrict__ sink, float lam, float eps, float factor) {
+                       const float* __restrict__ sink, float lam, float eps, float factor, const MultiExtra<T> X) {
     constexpr int NQ = MAPS * GROUP;
     constexpr int VN = Vec16<T>::N;
     extern __shared__ __align__(16) float smem[];
@@ -331,7 +373,8 @@ attn_multi_tile_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO
     for (int x = tid; x < dq; x += blockDim.x) qs[x] = ld(q + ((int64_t)t * H + h0) * (MAPS * dm) + x);
     const int lo = window > 0 ? max(0, pos - window + 1) : 0;
     const int n_kept = window > 0 ? min(keep_first, lo) : 0;
-    const int total = n_kept + (pos - lo + 1);
+    const int n_blocks = blocks_seen(pos, window, X.block);
+    const int total = n_blocks + n_kept + (pos - lo + 1);
     const int n_tiles_all = (total + TK - 1) / TK, per_run = (n_tiles_all + (int)gridDim.y - 1) / (int)gridDim.y;
     const int v_begin = TK * per_run * (int)blockIdx.y, v_end = min(total, TK * per_run * ((int)blockIdx.y + 1));
     const int n_tiles = v_end > v_begin ? (v_end - v_begin + TK - 1) / TK : 0;
@@ -345,10 +388,8 @@ attn_multi_tile_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO
         const int v0 = v_begin + it * TK, n_keys = min(TK, v_end - v0);
         const int kk = tid / TPK, c0 = tid % TPK;
         if (kk < n_keys) {
-            const int key = visible_key(v0 + kk, n_kept, lo);
-            const int64_t in_page = (int64_t)table[key / kPage] * page_elems, place = (int64_t)g * kPage + (key % kPage);
-            const T* ksrc = store + in_page + place * k_row;
-            const T* vsrc = store + in_page + v_off + place * v_row;
+            const KeyRows<T> rows = key_rows(v0 + kk, n_blocks, n_kept, lo, store, table, page_elems, g, k_row, v_off, v_row, X);
+            const T *ksrc = rows.k, *vsrc = rows.v;
             T* d = dst + (int64_t)kk * row_elems;
             for (int c = c0; c < kch; c += TPK) cp_async_16(d + c * VN, ksrc + c * VN);
             for (int c = c0; c < vch; c += TPK) cp_async_16(d + kd + c * VN, vsrc + c * VN);
@@ -409,7 +450,7 @@ attn_multi_tile_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO
                 }
             }
 #pragma unroll
-            for (int a = 0; a < NQ; ++a) s[j][a] = kk < n_keys ? warp_sum(s[j][a]) * scale : -INFINITY;
+            for (int a = 0; a < NQ; ++a) s[j][a] = kk < n_keys ? soft_capped(warp_sum(s[j][a]) * scale, X.cap) : -INFINITY;
         }
         // one step of the running maximum and sum for the warp's keys of this tile
         float p[KW][NQ];
@@ -456,7 +497,7 @@ attn_multi_tile_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO
         }
         __syncthreads();                        // everyone is done with this buffer
     }
-    fold_warps<TO, MAPS, GROUP, MV_CHUNKS>(m, l, acc, ms, accs, out, partial, t, h0, H, e, sink, lam, eps, factor);
+    fold_warps<TO, MAPS, GROUP, MV_CHUNKS>(m, l, acc, ms, accs, out, partial, t, h0, H, e, sink, lam, eps, factor, X.gate);
 }
 
 // The records of the runs of keys (a run that held no key has the maximum -inf; at most 64 runs) are folded in run order, map by
@@ -466,7 +507,7 @@ attn_multi_tile_kernel(const TQ* __restrict__ q, const T* __restrict__ store, TO
 template <typename TO, int MAPS, int MV_CHUNKS>
 __global__ void __launch_bounds__(128)
 attn_multi_merge_kernel(const float* __restrict__ partial, TO* __restrict__ out, int n_heads_total, int H, int e, int runs,
-                        const float* __restrict__ sink, float lam, float eps, float factor) {
+                        const float* __restrict__ sink, float lam, float eps, float factor, const float* gate) {
     constexpr unsigned ALL = 0xffffffffu;
     constexpr int CPW = MAPS == 1 ? 1 : MV_CHUNKS;                            // chunks a warp takes
     pdl_trigger();
@@ -516,7 +557,8 @@ attn_multi_merge_kernel(const float* __restrict__ partial, TO* __restrict__ out,
             const float fr = __shfl_sync(ALL, r < 32 ? f[0] : f[1], r & 31);
             if (fr != 0.f) fold(r, fr);               // (a run without a key left no values)
         }
-        const float inv = 1.0f / sum;
+        float inv = 1.0f / sum;
+        if (gate) inv *= gate[th];
 #pragma unroll
         for (int c = 0; c < 4 * CPW; ++c) y[a][c] *= inv;
     }
@@ -992,14 +1034,16 @@ template <typename T, typename TQ, typename TO, int MAPS, int GROUP, int MV_CHUN
 int attn_multi_launch(const void* q, const void* store, void* out, float* partial, const int* seq_of_token, const int* positions,
                       const int* page_table, int table_width, int n, int H, int G, int dm, int e, int64_t page_elems, int k_row,
                       int64_t v_off, int v_row, float scale, int window, int keep_first, const float* sink, float lam, float eps,
-                      float factor, int warps, int runs, cudaStream_t s) {
+                      float factor, int warps, int runs, const MultiExtra<T>& X, cudaStream_t s) {
     constexpr int NQ = MAPS * GROUP;
     constexpr int VN = Vec16<T>::N;
     const int dq_pad = (NQ * dm + 3) & ~3, e_pad = (e + 127) / 128 * 128;
     // rows that can be copied 16 bytes at a time, in a step of few tokens: the form that reads them through shared memory
     const bool v_same = v_off == 0 && v_row == k_row;
     const bool copies = warps > 1 && ((uintptr_t)store & 15) == 0 && dm % VN == 0 && k_row % VN == 0 && page_elems % VN == 0 &&
-                        e % VN == 0 && v_row % VN == 0 && v_off % VN == 0 && e % 4 == 0 && (MAPS * dm == k_row || !v_same);
+                        e % VN == 0 && v_row % VN == 0 && v_off % VN == 0 && e % 4 == 0 && (MAPS * dm == k_row || !v_same) &&
+                        (X.block == 0 || (((uintptr_t)X.pool & 15) == 0 && X.page_elems % VN == 0 && X.v_off % VN == 0));
+    WICK_REQUIRE(X.block == 0 || !v_same, "attn_multi: blocks are seen beside keys with values of their own");
     if (copies) {
         const size_t row_elems = (size_t)MAPS * dm + (v_same ? 0 : e);
         const size_t tile_bytes = (size_t)TS * TK * row_elems * sizeof(T), fold_bytes = (size_t)TW * NQ * e_pad * sizeof(float);
@@ -1013,11 +1057,11 @@ int attn_multi_launch(const void* q, const void* store, void* out, float* partia
             }
             WICK_CUDA(launch(attn_multi_tile_kernel<T, TQ, TO, MAPS, GROUP, MV_CHUNKS>, dim3((unsigned)(n * (H / GROUP)), runs), dim3(32 * TW),
                              smem, s, (const TQ*)q, (const T*)store, (TO*)out, partial, seq_of_token, positions, page_table, table_width,
-                             H, G, dm, e, page_elems, k_row, v_off, v_row, scale, window, keep_first, sink, lam, eps, factor));
+                             H, G, dm, e, page_elems, k_row, v_off, v_row, scale, window, keep_first, sink, lam, eps, factor, X));
             if (int rc = check_launch("attn_multi_tile")) return rc;
             if (partial) {
                 WICK_CUDA(launch(attn_multi_merge_kernel<TO, MAPS, MV_CHUNKS>, dim3(ceil_div((int64_t)n * H * (MAPS == 1 ? e_pad / 128 : 1), 4)), dim3(128), 0, s,
-                                 (const float*)partial, (TO*)out, n * H, H, e, runs, sink, lam, eps, factor));
+                                 (const float*)partial, (TO*)out, n * H, H, e, runs, sink, lam, eps, factor, X.gate));
                 return check_launch("attn_multi_merge");
             }
             return 0;
@@ -1032,11 +1076,11 @@ int attn_multi_launch(const void* q, const void* store, void* out, float* partia
     }
     WICK_CUDA(launch(attn_multi_kernel<T, TQ, TO, MAPS, GROUP, MV_CHUNKS>, dim3((unsigned)(n * (H / GROUP)), runs), dim3(32 * warps), smem, s,
                      (const TQ*)q, (const T*)store, (TO*)out, partial, seq_of_token, positions, page_table, table_width, H, G, dm, e,
-                     page_elems, k_row, v_off, v_row, scale, window, keep_first, sink, lam, eps, factor));
+                     page_elems, k_row, v_off, v_row, scale, window, keep_first, sink, lam, eps, factor, X));
     if (int rc = check_launch("attn_multi")) return rc;
     if (partial) {
         WICK_CUDA(launch(attn_multi_merge_kernel<TO, MAPS, MV_CHUNKS>, dim3(ceil_div((int64_t)n * H * (MAPS == 1 ? e_pad / 128 : 1), 4)), dim3(128), 0, s, (const float*)partial,
-                         (TO*)out, n * H, H, e, runs, sink, lam, eps, factor));
+                         (TO*)out, n * H, H, e, runs, sink, lam, eps, factor, X.gate));
         return check_launch("attn_multi_merge");
     }
     return 0;
@@ -1049,7 +1093,9 @@ template <typename T, typename TQ, typename TO, int MAPS>
 int attn_multi(const void* q, const void* store, void* out, float* partial, const int* seq_of_token, const int* positions,
                const int* page_table, int table_width, int n, int H, int G, int dm, int e, int64_t page_elems, int k_row,
                int64_t v_off, int v_row, float scale, int window, int keep_first, const float* sink, float lam, float eps,
-               float factor, int few, int runs, cudaStream_t s) {
+               float factor, int few, int runs, const MultiExtra<T>& X, cudaStream_t s) {
+    WICK_REQUIRE(X.block >= 0 && (X.block == 0 || (window > 0 && X.pool && X.rows == (kPage + X.block - 1) / X.block)), "attn_multi: bad blocks");
+    WICK_REQUIRE(!X.gate || MAPS == 1, "attn_multi: the factor per head belongs to one map");
     WICK_REQUIRE(H > 0 && G > 0 && H % G == 0 && dm > 0 && e > 0, "attn_multi: bad head counts or sizes");
     WICK_REQUIRE(e <= 128 * MV_MAX_CHUNKS, "attn_multi: a value size of %d is beyond %d", e, 128 * MV_MAX_CHUNKS);
     WICK_REQUIRE(window >= 0 && keep_first >= 0, "attn_multi: bad window");
@@ -1063,7 +1109,7 @@ int attn_multi(const void* q, const void* store, void* out, float* partial, cons
 #define WICK_AM(GROUP, CH)                                                                                                       \
     return attn_multi_launch<T, TQ, TO, MAPS, GROUP, CH>(q, store, out, partial, seq_of_token, positions, page_table, table_width, n, H, \
                                                          G, dm, e, page_elems, k_row, v_off, v_row, scale, window, keep_first, sink, \
-                                                         lam, eps, factor, few ? (GROUP * CH > 4 && (int64_t)n * (H / GROUP) * runs > 2 * sm_count() ? 4 : 8) : 1, runs, s)
+                                                         lam, eps, factor, few ? (GROUP * CH > 4 && (int64_t)n * (H / GROUP) * runs > 2 * sm_count() ? 4 : 8) : 1, runs, X, s)
     if (e <= 128) {
         if (MAPS == 1 && few && per_kv % 4 == 0) WICK_AM(4, 1);
         if (MAPS == 1 && few && per_kv % 2 == 0) WICK_AM(2, 1);
@@ -1149,20 +1195,25 @@ typedef __nv_bfloat16 bf16;
 
 // q: [n, H, maps * dm] (maps = 2: the activation type; maps = 1: float32, a query carried into the rows' space);
 // store: pages of page_elems elements; key row of (page, kv head g, place c): store + page * page_elems + (g * 64 + c) * k_row,
-// value row: ... + v_off + (g * 64 + c) * v_row; out: [n, H, e] (maps = 2: activation type; maps = 1: float32).
+// value row: ... + v_off + (g * 64 + c) * v_row; out: [n, H, e] (maps = 2: activation type; maps = 1: float32).  pool, block, rows: see
+// MultiExtra; its pages hold pool_page elements, the rows lie k_row and v_row apart, a page's values pool_v_off behind its keys.
+// (multi1_act: one map whose queries and results have the activation type.)
 #define WICK_ATTN_MULTI(NAME, T, TQ, TO, MAPS)                                                                                   \
     WICK_API int NAME(const void* q, const void* store, void* out, const int* seq_of_token, const int* positions,               \
                       const int* page_table, int table_width, int n, int H, int G, int dm, int e, int64_t page_elems, int k_row, \
                       int64_t v_off, int v_row, float scale, int window, int keep_first, const float* sink, float lam, float eps, \
-                      float factor, int few, int runs, float* partial, void* s) {                                                \
+                      float factor, int few, int runs, float* partial, const void* pool, int block, int rows,                    \
+                      int64_t pool_page, int64_t pool_v_off, float cap, const float* gate, void* s) {                            \
+        const MultiExtra<T> X = {(const T*)pool, block, rows, pool_page, pool_v_off, cap, gate};                                 \
         return attn_multi<T, TQ, TO, MAPS>(q, store, out, partial, seq_of_token, positions, page_table, table_width, n, H, G, dm, \
                                            e, page_elems, k_row, v_off, v_row, scale, window, keep_first, sink, lam, eps,        \
-                                           factor, few, runs, (cudaStream_t)s);                                                  \
+                                           factor, few, runs, X, (cudaStream_t)s);                                               \
     }
 WICK_ATTN_MULTI(wick_attn_multi2_bf16, bf16, bf16, bf16, 2)
 WICK_ATTN_MULTI(wick_attn_multi2_f32, float, float, float, 2)
 WICK_ATTN_MULTI(wick_attn_multi1_bf16, bf16, float, float, 1)
 WICK_ATTN_MULTI(wick_attn_multi1_f32, float, float, float, 1)
+WICK_ATTN_MULTI(wick_attn_multi1_act_bf16, bf16, bf16, bf16, 1)
 
 #define WICK_LATENT(T, SUFFIX)                                                                                                   \
     WICK_API int wick_latent_finish_##SUFFIX(const float* parts, int splits, int n, int cols, int qr, int r, int dr, int Hg,  \

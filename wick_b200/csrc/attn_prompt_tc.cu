@@ -24,6 +24,10 @@
 // float32 hold without loss of relative precision.
 // Value rows beyond the cached length are zeroed in shared memory before they
 // are multiplied (their weight is zero, but the row may hold anything).
+// The EXTRA form also sees the blocks of `block` positions that lie wholly before a row's
+// window, each as one key and value (tiles of 64 blocks a sequence, laid out like cache
+// pages; their key blocks come before the window's), soft-caps the scores and multiplies
+// the result by a number per token and head.
 // Every wait is bounded and reports through the status word.
 // Formulas: wick src/model.rs:520-553.  The plain forms of this computation are
 // attn_prompt_mma_kernel (attn_prompt_mma.cu) and attn_prompt_kernel (attn.cu).
@@ -174,12 +178,27 @@ __device__ __forceinline__ int first_visible_key(int p, int mask, int size) {
     return mask == 1 ? p / size * size : (mask == 2 ? max(0, p - size + 1) : 0);
 }
 
+// What the EXTRA form does besides.
+struct TcExtra {
+    int pool_tiles, block;         // tile i of sequence b is page b * pool_tiles + i of the blocks' array; block 0: there are none
+    float cap;                     // of the scores; 0: none
+    const float* gate;             // float32 [n, heads] or null: a factor of the result
+};
+__device__ __forceinline__ int blocks_seen(int p, int window, int block) { return block > 0 && p + 1 > window ? (p + 1 - window) / block : 0; }
+__device__ __forceinline__ float rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+template <bool EXTRA>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_prompt_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map,
                       bf16* __restrict__ out, const int* __restrict__ cu_seqlens, int n_seqs,
                       const int* __restrict__ start_arr,
                       const int* __restrict__ page_table, int table_width, int n_tiles, int n_heads, int n_kv,
-                      float scale, int* status, int mask, int mask_size, const float* __restrict__ sink) {
+                      float scale, int* status, int mask, int mask_size, const float* __restrict__ sink,
+                      const __grid_constant__ CUtensorMap pool_map, const TcExtra X) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ uint64_t q_full, full[NSLOT];
     __shared__ uint64_t s_full[NBUF], p_full[NBUF], pv_done[2], v_free[NBUF], x_bar[4];   // pv_done: even blocks, odd blocks
@@ -201,7 +220,10 @@ attn_prompt_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
     // With a mask the first block of keys is the one that holds the first row's first visible key (the first
     // visible key grows with the position); blocks are counted from there, j = 0 .. n_blk - 1, everywhere below.
     const int jb0 = first_visible_key(start + q0, mask, mask_size) / BK;
-    const int n_blk = last_key / BK + 1 - jb0;
+    // (EXTRA: the first n_pool key blocks hold blocks of positions; block j >= n_pool holds the keys from (j + jw) BK on)
+    const int n_pool = EXTRA ? (blocks_seen(last_key, mask_size, X.block) + BK - 1) / BK : 0;
+    const int jw = jb0 - n_pool;
+    const int n_blk = last_key / BK + 1 - jw;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     uint8_t* base = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -253,8 +275,17 @@ attn_prompt_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
                     if (!mbar_wait(is_v ? &v_free[jp % NBUF] : &s_full[jp % NBUF], (jp / NBUF) & 1, &abort_flag, status, 7)) break;
                 }
                 mbar_expect_tx(&full[slot], TILE_BYTES);
+                if (EXTRA && j < n_pool) {
+                    for (int w = 0; w < 2; ++w) {
+                        const int page = b * X.pool_tiles + min(2 * j + w, X.pool_tiles - 1);
+                        for (int pn = 0; pn < PANELS; ++pn)
+                            tma_load_2d(&pool_map, &full[slot], kv_s + slot * TILE_BYTES + pn * PANEL_BYTES + w * (kPage * 128), pn * 64,
+                                        ((page * 2 + is_v) * n_kv + kvh) * kPage);
+                    }
+                    continue;
+                }
                 for (int w = 0; w < 2; ++w) {
-                    const int idx = 2 * (j + jb0) + w;
+                    const int idx = 2 * (j + jw) + w;
                     const int page = idx < table_width ? page_table[(int64_t)b * table_width + idx] : 0;
                     for (int pn = 0; pn < PANELS; ++pn)
                         tma_load_2d(&kv_map, &full[slot], kv_s + slot * TILE_BYTES + pn * PANEL_BYTES + w * (kPage * 128), pn * 64,
@@ -314,7 +345,10 @@ attn_prompt_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
         const int q_pos = start + q0 + r;
         const int limit = min(q_pos, kv_len - 1);                   // last visible key position
         const int vis = first_visible_key(limit, mask, mask_size);  // first visible key position
-        const float sl2 = scale * 1.4426950408889634f;
+        const bool capped = EXTRA && X.cap > 0.f;
+        const float sl2 = capped ? 1.0f : scale * 1.4426950408889634f;   // (a capped score comes in units of log2 e)
+        const float cap2 = EXTRA ? X.cap * 1.4426950408889634f : 0.f, two_s = capped ? 2.0f * scale * 1.4426950408889634f / X.cap : 0.f;
+        const int n_seen = EXTRA ? blocks_seen(limit, mask_size, X.block) : 0;
         const float sink2 = sink ? sink[head] * 1.4426950408889634f : -INFINITY;   // a score without a value
         const uint32_t lane_base = tmem + ((uint32_t)(quad * 32) << 16);
         constexpr int OW = HD / 2;                                  // columns of O this thread rescales and stores
@@ -330,15 +364,21 @@ attn_prompt_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
             ok = __all_sync(0xffffffffu, mbar_wait(&s_full[buf], (j / NBUF) & 1, &abort_flag, status, 7));
             if (!ok) break;
             tc_fence_after();
-            const int key0 = (j + jb0) * BK + c_lo;
+            const bool pooled = EXTRA && j < n_pool;
+            const int key0 = (pooled ? j : j + jw) * BK + c_lo;
+            const int last = pooled ? n_seen - 1 : limit, first_key = pooled ? 0 : vis;
             float s[HALF_K];
             tc_ld32_nowait(s_addr + c_lo, reinterpret_cast<uint32_t*>(s));
             tc_ld32_nowait(s_addr + c_lo + 32, reinterpret_cast<uint32_t*>(s + 32));
             tc_ld_wait();
-            if (key0 + HALF_K - 1 > limit || key0 < vis) {
+            if (capped) {                                           // cap tanh(s / cap) = cap (1 - 2 / (1 + exp(2 s / cap)))
+#pragma unroll
+                for (int i = 0; i < HALF_K; ++i) s[i] = fmaf(-2.0f * cap2, rcp(1.0f + ex2(s[i] * two_s)), cap2);
+            }
+            if (key0 + HALF_K - 1 > last || key0 < first_key) {
 #pragma unroll
                 for (int i = 0; i < HALF_K; ++i)
-                    if (key0 + i > limit || key0 + i < vis) s[i] = -INFINITY;
+                    if (key0 + i > last || key0 + i < first_key) s[i] = -INFINITY;
             }
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -403,7 +443,7 @@ attn_prompt_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
             tc_st_wait();
             l = l * alpha + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
             // value rows that hold no token yet are made zero before they are multiplied
-            const int valid = kv_len - (j + jb0) * BK;
+            const int valid = pooled ? BK : kv_len - (j + jw) * BK;  // (places without a block hold zeros)
             if (valid < BK) {
                 ok = __all_sync(0xffffffffu, mbar_wait(&full[v_slot], (v_item / NSLOT) & 1, &abort_flag, status, 7));
                 if (!ok) break;
@@ -435,7 +475,8 @@ attn_prompt_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
             // every lane takes part in the loads from tensor memory; only rows that exist are stored
             const float l_row = l_x[r] + l_x[BQ + r] + (sink ? ex2(sink2 - m) : 0.f);   // (both halves scale by the same m)
             const bool store = r < rows && l_row > 0.f;
-            const float inv = store ? 1.0f / l_row : 0.f;
+            float inv = store ? 1.0f / l_row : 0.f;
+            if (EXTRA && X.gate && store) inv *= X.gate[(int64_t)(tok0 + q0 + r) * n_heads + head];
             bf16* dst = out + ((int64_t)(tok0 + q0 + r) * n_heads + head) * HD + half * OW;
 #pragma unroll
             for (int c = 0; c < OW; c += 32) {
@@ -482,29 +523,58 @@ WICK_API int wick_attn_prompt_tc_supported() { return prompttc::SUPPORTED ? 1 : 
 // [kv_pages, 2, n_kv, 64, HD] (it already holds the new tokens' keys and values);
 // n_tiles: the step's 64-row work items (one per 64 new tokens of a sequence, numbered
 // sequence by sequence); status: device int (code 7 if a block gave up waiting).
-// ... then the mask (0, or 1 / 2 with its size) and the sinks (float32 [n_heads] or null).
-WICK_API int wick_attn_prompt_tc_masked_bf16(const void* q, long long n_tokens, const void* kv, long long kv_pages, void* out,
-                                             int n_tiles, const int* cu_seqlens, int n_seqs,
-                                             const int* start, const int* page_table, int table_width, int n_heads, int n_kv,
-                                             float scale, int* status, int mask, int mask_size, const float* sink, void* s) {
+static int attn_prompt_tc(const void* q, long long n_tokens, const void* kv, long long kv_pages, void* out, int n_tiles, const int* cu_seqlens,
+                          int n_seqs, const int* start, const int* page_table, int table_width, int n_heads, int n_kv, float scale,
+                          int* status, int mask, int mask_size, const float* sink, const void* pool, const prompttc::TcExtra* extra, void* s) {
     using namespace prompttc;
     WICK_REQUIRE(mask == 0 || ((mask == 1 || mask == 2) && mask_size > 0), "attention: mask %d of size %d", mask, mask_size);
     WICK_REQUIRE(SUPPORTED, "attention (tcgen05): head_dim %d is not 64 or 128", (int)WICK_HD);
     WICK_REQUIRE(n_heads > 0 && n_kv > 0 && n_heads % n_kv == 0, "attention: %d heads over %d kv heads", n_heads, n_kv);
     WICK_REQUIRE(n_heads <= 65535, "attention: %d heads is beyond the grid limit", n_heads);
     if (n_tiles == 0) return 0;
-    CUtensorMap q_map, kv_map;
+    CUtensorMap q_map, kv_map, pool_map;
     if (int e = make_bf16_map(&q_map, q, n_tokens, (long long)n_heads * HD, BQ, "attention (tcgen05)")) return e;
     if (int e = make_bf16_map(&kv_map, kv, kv_pages * 2 * n_kv * kPage, HD, kPage, "attention (tcgen05)")) return e;
-    static bool raised = false;
-    if (!raised) {
-        WICK_CUDA(cudaFuncSetAttribute(attn_prompt_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
-        raised = true;
+    pool_map = kv_map;
+    TcExtra X = {0, 0, 0.f, nullptr};
+    if (extra) X = *extra;
+    if (pool) {
+        WICK_REQUIRE(mask == 2 && X.block > 0 && X.pool_tiles > 0, "attention (tcgen05): blocks are seen beside a window");
+        if (int e = make_bf16_map(&pool_map, pool, (long long)n_seqs * X.pool_tiles * 2 * n_kv * kPage, HD, kPage, "attention (tcgen05)")) return e;
+    } else {
+        X.block = 0;
     }
-    WICK_CUDA(launch(attn_prompt_tc_kernel, dim3(n_tiles, n_heads), dim3(THREADS), (size_t)SMEM_BYTES, (cudaStream_t)s, q_map,
+    auto kernel = extra ? attn_prompt_tc_kernel<true> : attn_prompt_tc_kernel<false>;
+    static bool raised[2] = {false, false};
+    if (!raised[extra ? 1 : 0]) {
+        WICK_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES));
+        raised[extra ? 1 : 0] = true;
+    }
+    WICK_CUDA(launch(kernel, dim3(n_tiles, n_heads), dim3(THREADS), (size_t)SMEM_BYTES, (cudaStream_t)s, q_map,
                      kv_map, (bf16*)out, cu_seqlens, n_seqs, start, page_table, table_width, n_tiles, n_heads,
-                     n_kv, scale, status, mask, mask_size, sink));
+                     n_kv, scale, status, mask, mask_size, sink, pool_map, X));
     return check_launch("attn_prompt_tc");
+}
+
+// ... then the mask (0, or 1 / 2 with its size) and the sinks (float32 [n_heads] or null).
+WICK_API int wick_attn_prompt_tc_masked_bf16(const void* q, long long n_tokens, const void* kv, long long kv_pages, void* out,
+                                             int n_tiles, const int* cu_seqlens, int n_seqs,
+                                             const int* start, const int* page_table, int table_width, int n_heads, int n_kv,
+                                             float scale, int* status, int mask, int mask_size, const float* sink, void* s) {
+    return attn_prompt_tc(q, n_tokens, kv, kv_pages, out, n_tiles, cu_seqlens, n_seqs, start, page_table, table_width, n_heads, n_kv, scale,
+                          status, mask, mask_size, sink, nullptr, nullptr, s);
+}
+
+// ... then the blocks' array (bfloat16 [n_seqs * pool_tiles, 2, n_kv, 64, HD], or null), its tiles a sequence and positions a block, the cap
+// of the scores (0: none) and the factors of the result (float32 [n_tokens, n_heads] or null).
+WICK_API int wick_attn_prompt_tc_pooled_bf16(const void* q, long long n_tokens, const void* kv, long long kv_pages, void* out,
+                                             int n_tiles, const int* cu_seqlens, int n_seqs,
+                                             const int* start, const int* page_table, int table_width, int n_heads, int n_kv,
+                                             float scale, int* status, int mask, int mask_size, const float* sink, const void* pool,
+                                             int pool_tiles, int block, float cap, const float* gate, void* s) {
+    const prompttc::TcExtra X = {pool_tiles, block, cap, gate};
+    return attn_prompt_tc(q, n_tokens, kv, kv_pages, out, n_tiles, cu_seqlens, n_seqs, start, page_table, table_width, n_heads, n_kv, scale,
+                          status, mask, mask_size, sink, pool, &X, s);
 }
 
 WICK_API int wick_attn_prompt_tc_bf16(const void* q, long long n_tokens, const void* kv, long long kv_pages, void* out,

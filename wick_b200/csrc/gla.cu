@@ -13,6 +13,10 @@
 // A second preparation (hgrn2) makes the same rows from [q: H dk | z: H dk | v: H dv]: q <- silu(q), with a learned lower
 // bound l per channel a = l + (1 - l) sigmoid(z + b) and k = 1 - a = (1 - l) sigmoid(-(z + b)); scan and norm follow (no gate).
 //
+// A third one (retention) makes them from [q: H dk | k: H dk | v: H dv | g: H dv]: pairs (i, i + dims / 2) of the first `dims` elements of
+// every q and k head turn by the angles of the step's tables, k is multiplied by dk^(-1/2); the decay is one given number per
+// head, so the rows hold no decays, [q | k | v].  The norm that follows has no weight.
+//
 // A sequence's record (float32) is the state as [H][dv][dk] (a column of S, the dk numbers that meet one element of v,
 // lies together).  Everything here is float32 arithmetic; a token's numbers depend on its own sequence alone.  A step of
 // few tokens adds them in the same order whatever its shape; a long prompt step scanned in chunks (below) rounds the
@@ -189,6 +193,84 @@ hgrn2_prepare_kernel(const float* __restrict__ parts, int splits, int64_t split_
     store(2 * HK + c, a);
 }
 
+// grid (tokens, ceil(items / 256)), an item VEC neighbours: first the turning pairs of every head (of q and k together), then the key
+// channels that pass, then the value elements.  out row: [q | k | v], 2 H dk + H dv numbers.
+template <int VEC, bool ONE>
+__global__ void __launch_bounds__(256)
+retention_prepare_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, int cols, int H, int dk, int HV, int half,
+                         float k_scale, const float* __restrict__ cos_t, const float* __restrict__ sin_t, float* __restrict__ out) {
+    pdl_trigger();
+    pdl_wait();
+    parts = fresh(parts);
+    cos_t = fresh(cos_t);
+    sin_t = fresh(sin_t);
+    const int64_t t = blockIdx.x;
+    int c = ((int)blockIdx.y * (int)blockDim.x + (int)threadIdx.x) * VEC;
+    const int HK = H * dk, pass = dk - 2 * half;
+    const float* row = parts + t * cols;
+    float* o = out + t * (2 * HK + HV);
+    auto load = [&](const float* src, float (&v)[VEC]) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+        for (int s = 0; s < (ONE ? 1 : splits); ++s) {
+            const float* p = src + s * split_stride;
+            if (VEC == 4) {
+                const float4 d = *reinterpret_cast<const float4*>(p);
+                v[0] += d.x; v[VEC > 1 ? 1 : 0] += d.y; v[VEC > 2 ? 2 : 0] += d.z; v[VEC > 3 ? 3 : 0] += d.w;
+            } else {
+                v[0] += *p;
+            }
+        }
+    };
+    auto store = [&](float* dst, const float (&v)[VEC]) {
+        if (VEC == 4) *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[VEC > 1 ? 1 : 0], v[VEC > 2 ? 2 : 0], v[VEC > 3 ? 3 : 0]);
+        else *dst = v[0];
+    };
+    if (c < H * half) {                                                  // (VEC divides half, what passes and dv: an item is of one kind)
+        const int h = c / half, i = c - h * half;
+        float u[2][VEC], v[2][VEC];
+#pragma unroll
+        for (int a = 0; a < 2; ++a) {
+            load(row + a * HK + h * dk + i, u[a]);
+            load(row + a * HK + h * dk + half + i, v[a]);
+        }
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+            const float cs = cos_t[t * half + i + j], sn = sin_t[t * half + i + j];
+#pragma unroll
+            for (int a = 0; a < 2; ++a) {
+                const float ru = u[a][j] * cs - v[a][j] * sn, rv = v[a][j] * cs + u[a][j] * sn;
+                u[a][j] = a ? ru * k_scale : ru;
+                v[a][j] = a ? rv * k_scale : rv;
+            }
+        }
+#pragma unroll
+        for (int a = 0; a < 2; ++a) {
+            store(o + a * HK + h * dk + i, u[a]);
+            store(o + a * HK + h * dk + half + i, v[a]);
+        }
+        return;
+    }
+    c -= H * half;
+    if (c < H * pass) {
+        const int h = c / pass, at = h * dk + 2 * half + (c - h * pass);
+        float q[VEC], k[VEC];
+        load(row + at, q);
+        load(row + HK + at, k);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) k[j] *= k_scale;
+        store(o + at, q);
+        store(o + HK + at, k);
+        return;
+    }
+    c -= H * pass;
+    if (c < HV) {
+        float v[VEC];
+        load(row + 2 * HK + c, v);
+        store(o + 2 * HK + c, v);
+    }
+}
+
 // The sums of four columns over the LN threads that share them (see the state-space scan: the same exchange).
 template <int LN>
 __device__ __forceinline__ float gla_sum_columns(float (&a)[4], int sub, int& col, bool& writes) {
@@ -225,11 +307,12 @@ __device__ __forceinline__ float gla_sum_columns(float (&a)[4], int sub, int& co
 //           the products of its decays to `chunk_decay` [chunks][H][dk].  gla_chunk_join_kernel then walks a sequence's chunks
 //           and leaves in `chunk_state` the state each chunk starts from, and the last one in the record.
 //   MODE 2, the same grid: a chunk from the state it starts from, o out.
-template <int LN, int MODE>
+// FIXED: the decay is one number per head, head_decay[h], and the tokens' rows hold none ([q | k | v]).
+template <int LN, int MODE, bool FIXED>
 __global__ void __launch_bounds__(128)
 gla_scan_kernel(const float* __restrict__ qkav, int channels, int H, int P, int N, float* __restrict__ state, int64_t record,
                 const int* __restrict__ slots, const int* __restrict__ cu_seqlens, float* __restrict__ y, int run, int n_seqs,
-                int chunk, float* __restrict__ chunk_state, float* __restrict__ chunk_decay) {
+                int chunk, float* __restrict__ chunk_state, float* __restrict__ chunk_decay, const float* __restrict__ head_decay) {
     extern __shared__ float4 gla_smem4[];
     float* smem = reinterpret_cast<float*>(gla_smem4);
     pdl_trigger();
@@ -249,8 +332,10 @@ gla_scan_kernel(const float* __restrict__ qkav, int channels, int H, int P, int 
         return;
     }
     const int tid = threadIdx.x, sub = tid % LN, lc = tid / LN, pc0 = blockIdx.y * CPB, col0 = pc0 + lc * CT;
+    constexpr int VECS = FIXED ? 2 : 3;                                  // vectors of key channels a token brings
+    const float fixed = FIXED ? head_decay[h] : 0.f;
     const int per4 = (N + 4 * LN - 1) / (4 * LN), NP = per4 * 4 * LN, HK = H * N, inner = H * P;
-    const int stage = (run * (CPB + 3 * NP) + 3) & ~3;
+    const int stage = (run * (CPB + VECS * NP) + 3) & ~3;
     float* ys = smem + 2 * stage;                                        // [run][CPB]
     float* sp = MODE == 0 ? state + (int64_t)slots[b] * record + ((int64_t)h * P + col0) * N
                           : chunk_state + (((int64_t)unit * H + h) * P + col0) * N;
@@ -290,7 +375,7 @@ gla_scan_kernel(const float* __restrict__ qkav, int channels, int H, int P, int 
             const int c4 = CPB / 4, n4 = NP / 4;
             for (int idx = tid; idx < len * c4; idx += blockDim.x) {
                 const int i = idx / c4, c = (idx - i * c4) * 4;
-                if (pc0 + c < P) gla_cp_async<16>(vs + i * CPB + c, src + (int64_t)i * channels + 3 * HK + h * P + pc0 + c);
+                if (pc0 + c < P) gla_cp_async<16>(vs + i * CPB + c, src + (int64_t)i * channels + VECS * HK + h * P + pc0 + c);
             }
             for (int idx = tid; idx < len * n4; idx += blockDim.x) {
                 const int i = idx / n4, n = (idx - i * n4) * 4;
@@ -298,13 +383,13 @@ gla_scan_kernel(const float* __restrict__ qkav, int channels, int H, int P, int 
                     const float* rowp = src + (int64_t)i * channels + h * N + n;
                     if (MODE != 1) gla_cp_async<16>(qs + i * NP + n, rowp);
                     gla_cp_async<16>(ks + i * NP + n, rowp + HK);
-                    gla_cp_async<16>(as + i * NP + n, rowp + 2 * HK);
+                    if (!FIXED) gla_cp_async<16>(as + i * NP + n, rowp + 2 * HK);
                 }
             }
         } else {
             for (int idx = tid; idx < len * CPB; idx += blockDim.x) {
                 const int i = idx / CPB, c = idx - i * CPB;
-                if (pc0 + c < P) gla_cp_async<4>(vs + idx, src + (int64_t)i * channels + 3 * HK + h * P + pc0 + c);
+                if (pc0 + c < P) gla_cp_async<4>(vs + idx, src + (int64_t)i * channels + VECS * HK + h * P + pc0 + c);
             }
             for (int idx = tid; idx < len * NP; idx += blockDim.x) {
                 const int i = idx / NP, n = idx - i * NP;
@@ -312,7 +397,7 @@ gla_scan_kernel(const float* __restrict__ qkav, int channels, int H, int P, int 
                     const float* rowp = src + (int64_t)i * channels + h * N + n;
                     if (MODE != 1) gla_cp_async<4>(qs + idx, rowp);
                     gla_cp_async<4>(ks + idx, rowp + HK);
-                    gla_cp_async<4>(as + idx, rowp + 2 * HK);
+                    if (!FIXED) gla_cp_async<4>(as + idx, rowp + 2 * HK);
                 }
             }
         }
@@ -342,7 +427,7 @@ gla_scan_kernel(const float* __restrict__ qkav, int channels, int H, int P, int 
 #pragma unroll
             for (int r = 0; r < R4; ++r) {
                 if (r < per4) {
-                    const float4 kv = ki[r * LN], av = ai[r * LN];
+                    const float4 kv = ki[r * LN], av = FIXED ? make_float4(fixed, fixed, fixed, fixed) : ai[r * LN];
                     const float kk[4] = {kv.x, kv.y, kv.z, kv.w}, aa[4] = {av.x, av.y, av.z, av.w};
 #pragma unroll
                     for (int j = 0; j < 4; ++j) {
@@ -453,8 +538,8 @@ gla_chunk_join_kernel(float* __restrict__ chunk_state, const float* __restrict__
     *rec = S;
 }
 
-// grid (tokens, groups of heads), a warp per head: o / sqrt(mean(o^2) + eps) * w * silu(g), g from the projection's sums (no
-// gate where there are none).
+// grid (tokens, groups of heads), a warp per head: o / sqrt(mean(o^2) + eps) * w * silu(g) (no factor w where it is null), g from the projection's
+// sums (no gate where there are none).
 template <typename T, bool ONE>
 __global__ void __launch_bounds__(256)
 gla_norm_gate_kernel(const float* __restrict__ y, const float* __restrict__ parts, int splits, int64_t split_stride, int cols,
@@ -471,7 +556,7 @@ gla_norm_gate_kernel(const float* __restrict__ y, const float* __restrict__ part
         ss = warp_sum(ss);
         const float f = 1.0f / sqrtf(ss / (float)P + eps);
         for (int j = lane; j < P; j += 32) {
-            float v = (row[j] * f) * w[j];
+            float v = w ? (row[j] * f) * w[j] : row[j] * f;
             if (parts) {
                 const int64_t at = (int64_t)t * cols + g_col + h * P + j;
                 const float g = ONE ? parts[at] : gla_sum_parts(parts, splits, split_stride, at);
@@ -484,59 +569,61 @@ gla_norm_gate_kernel(const float* __restrict__ y, const float* __restrict__ part
 
 struct GlaArgs {
     const float* qkav; int channels, H, P, N; float* state; int64_t record; const int *slots, *cu_seqlens; float* y;
-    int run, n_seqs, chunk; float *chunk_state, *chunk_decay; int threads;
+    int run, n_seqs, chunk; float *chunk_state, *chunk_decay; int threads; const float* head_decay;
 };
 
-template <int LN, int MODE>
+template <int LN, int MODE, bool FIXED>
 int gla_launch_mode(const GlaArgs& a, int units, size_t smem, cudaStream_t s) {
     static bool raised = false;
     if (smem > 48 * 1024 && !raised) {
-        WICK_CUDA(cudaFuncSetAttribute(gla_scan_kernel<LN, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+        WICK_CUDA(cudaFuncSetAttribute(gla_scan_kernel<LN, MODE, FIXED>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
         raised = true;
     }
-    WICK_CUDA(launch(gla_scan_kernel<LN, MODE>, dim3(units * a.H, ceil_div(a.P, a.threads / LN * GLA_COLS)), dim3(a.threads), smem, s,
+    WICK_CUDA(launch(gla_scan_kernel<LN, MODE, FIXED>, dim3(units * a.H, ceil_div(a.P, a.threads / LN * GLA_COLS)), dim3(a.threads), smem, s,
                      a.qkav, a.channels, a.H, a.P, a.N, a.state, a.record, a.slots, a.cu_seqlens, a.y, a.run, a.n_seqs, a.chunk,
-                     a.chunk_state, a.chunk_decay));
+                     a.chunk_state, a.chunk_decay, a.head_decay));
     return check_launch("gla_scan");
 }
 
-template <int LN>
+template <int LN, bool FIXED>
 int gla_launch(const GlaArgs& a, int chunks, size_t smem, cudaStream_t s) {
-    if (chunks == 0) return gla_launch_mode<LN, 0>(a, a.n_seqs, smem, s);
-    if (gla_launch_mode<LN, 1>(a, chunks, smem, s)) return 1;
+    if (chunks == 0) return gla_launch_mode<LN, 0, FIXED>(a, a.n_seqs, smem, s);
+    if (gla_launch_mode<LN, 1, FIXED>(a, chunks, smem, s)) return 1;
     const int64_t all = (int64_t)a.H * a.P * a.N;
     WICK_CUDA(launch(gla_chunk_join_kernel, dim3(a.n_seqs, (unsigned)ceil_div(all, (int64_t)256)), dim3(256), 0, s, a.chunk_state,
                      (const float*)a.chunk_decay, a.H, a.P, a.N, a.state, a.record, a.slots, a.cu_seqlens, a.chunk));
     if (check_launch("gla_chunk_join")) return 1;
-    return gla_launch_mode<LN, 2>(a, chunks, smem, s);
+    return gla_launch_mode<LN, 2, FIXED>(a, chunks, smem, s);
 }
 
 // The scan of prepared rows, by whichever form the step's shape asks for.
+template <bool FIXED>
 int gla_scan(float* qkav, int H, int dk, int dv, float* state, int64_t record, const int* slots, int n_seqs, const int* cu_seqlens,
-             float* y, int max_q, int chunk, int chunks, float* chunk_state, float* chunk_decay, cudaStream_t s) {
-    const int N = dk, P = dv, channels = 3 * H * dk + H * dv;
+             float* y, int max_q, int chunk, int chunks, float* chunk_state, float* chunk_decay, const float* head_decay, cudaStream_t s) {
+    constexpr int VECS = FIXED ? 2 : 3;
+    const int N = dk, P = dv, channels = VECS * H * dk + H * dv;
     int ln = 1;
     while (ln < 32 && (N + ln - 1) / ln > GLA_ROWS) ln *= 2;
     if (ln < 4 && N >= 16) ln = 4;                                       // (a thread keeps a few numbers, not a whole column)
     int threads = ceil_div(P, GLA_COLS) * ln;
     threads = threads > 128 ? 128 : (threads + 31) / 32 * 32;
     const int cpb = threads / ln * GLA_COLS, np = ceil_div(N, 4 * ln) * 4 * ln;
-    const int per_token = 2 * (cpb + 3 * np) + cpb;                       // (two stages of inputs, one of results)
+    const int per_token = 2 * (cpb + VECS * np) + cpb;                       // (two stages of inputs, one of results)
     int run = (52 * 1024 / 4) / per_token;                                // (four blocks of this size share an SM)
     run = run < 1 ? 1 : (run > 64 ? 64 : run);
     if (run > max_q && max_q >= 1) run = max_q;
     if (chunks > 0 && run > chunk) run = chunk;
     if (chunks > 0 && run < chunk) run = ceil_div(chunk, ceil_div(chunk, run));   // (equal runs)
-    const size_t smem = (size_t)(2 * ((run * (cpb + 3 * np) + 3) & ~3) + run * cpb) * sizeof(float);
+    const size_t smem = (size_t)(2 * ((run * (cpb + VECS * np) + 3) & ~3) + run * cpb) * sizeof(float);
     const GlaArgs a = {qkav, channels, H, P, N, state, record, slots, cu_seqlens, y, run, n_seqs, chunk, chunk_state, chunk_decay,
-                       threads};
+                       threads, head_decay};
     switch (ln) {
-        case 1: return gla_launch<1>(a, chunks, smem, s);
-        case 2: return gla_launch<2>(a, chunks, smem, s);
-        case 4: return gla_launch<4>(a, chunks, smem, s);
-        case 8: return gla_launch<8>(a, chunks, smem, s);
-        case 16: return gla_launch<16>(a, chunks, smem, s);
-        default: return gla_launch<32>(a, chunks, smem, s);
+        case 1: return gla_launch<1, FIXED>(a, chunks, smem, s);
+        case 2: return gla_launch<2, FIXED>(a, chunks, smem, s);
+        case 4: return gla_launch<4, FIXED>(a, chunks, smem, s);
+        case 8: return gla_launch<8, FIXED>(a, chunks, smem, s);
+        case 16: return gla_launch<16, FIXED>(a, chunks, smem, s);
+        default: return gla_launch<32, FIXED>(a, chunks, smem, s);
     }
 }
 
@@ -582,7 +669,7 @@ WICK_API int wick_gla_mix(const float* parts, int splits, int n, int cols, int H
     WICK_CUDA(launch(prepare, dim3(ceil_div(n, pb), prep_tiles), dim3(GLA_PREP_THREADS), prep_smem, s, parts, splits, stride, cols, HK, HV,
                      rank, w2, b2, q_scale, 1.0f / tau, qkav, n, stage));
     if (check_launch("gla_prepare")) return 1;
-    return gla_scan(qkav, H, dk, dv, state, record, slots, n_seqs, cu_seqlens, y, max_q, chunk, chunks, chunk_state, chunk_decay, s);
+    return gla_scan<false>(qkav, H, dk, dv, state, record, slots, n_seqs, cu_seqlens, y, max_q, chunk, chunks, chunk_state, chunk_decay, nullptr, s);
 }
 
 // parts: float32 [splits, n, 2 H dk + H dv] laid out [q | z | v]; bias, lower: float32 [H dk]; the rest as above.
@@ -601,10 +688,34 @@ WICK_API int wick_hgrn2_mix(const float* parts, int splits, int n, int H, int dk
     WICK_CUDA(launch(prepare, dim3(n, ceil_div(HK + HV, vec ? 1024 : 256)), dim3(256), 0, s, parts, splits, stride, HK, HV, bias, lower,
                      qkav));
     if (check_launch("hgrn2_prepare")) return 1;
-    return gla_scan(qkav, H, dk, dv, state, record, slots, n_seqs, cu_seqlens, y, max_q, chunk, chunks, chunk_state, chunk_decay, s);
+    return gla_scan<false>(qkav, H, dk, dv, state, record, slots, n_seqs, cu_seqlens, y, max_q, chunk, chunks, chunk_state, chunk_decay, nullptr, s);
 }
 
-// y: float32 [n, H dv]; parts as above (g from column g_col on) or null (no gate); w: float32 [dv]; out: [n, H dv].
+// parts: float32 [splits, n, cols] laid out [q | k | v] and whatever follows; cos_t, sin_t: float32 [n, dims / 2]; decay: float32 [H];
+// qkv: float32 [n, 2 H dk + H dv], written here; the rest as above.
+WICK_API int wick_retention_mix(const float* parts, int splits, int n, int cols, int H, int dk, int dv, const float* cos_t, const float* sin_t,
+                                int dims, float k_scale, const float* decay, float* state, int64_t record, const int* slots, int n_seqs,
+                                const int* cu_seqlens, float* qkv, float* y, int max_q, int chunk, int chunks, float* chunk_state,
+                                float* chunk_decay, void* stream) {
+    cudaStream_t s = (cudaStream_t)stream;
+    WICK_REQUIRE(H > 0 && dk > 0 && dv > 0 && decay, "retention_mix: bad sizes");
+    WICK_REQUIRE(dims >= 0 && dims % 2 == 0 && dims <= dk && (dims == 0 || (cos_t && sin_t)), "retention_mix: %d rotated elements of %d", dims, dk);
+    WICK_GLA_CHECKS("retention_mix");
+    const int HK = H * dk, HV = H * dv, half = dims / 2;
+    WICK_REQUIRE(cols >= 2 * HK + HV, "retention_mix: rows of %d numbers, %d expected", cols, 2 * HK + HV);
+    if (n == 0 || n_seqs == 0) return 0;
+    const int64_t stride = (int64_t)n * cols;
+    const bool vec = ((half | (dk - dims) | dk | HV | cols) & 3) == 0 && (((uintptr_t)parts | (uintptr_t)qkv) & 15) == 0;
+    auto prepare = vec ? (splits == 1 ? retention_prepare_kernel<4, true> : retention_prepare_kernel<4, false>)
+                       : (splits == 1 ? retention_prepare_kernel<1, true> : retention_prepare_kernel<1, false>);
+    const int items = H * half + H * (dk - dims) + HV;
+    WICK_CUDA(launch(prepare, dim3(n, ceil_div(items, vec ? 1024 : 256)), dim3(256), 0, s, parts, splits, stride, cols, H, dk, HV, half, k_scale,
+                     cos_t, sin_t, qkv));
+    if (check_launch("retention_prepare")) return 1;
+    return gla_scan<true>(qkv, H, dk, dv, state, record, slots, n_seqs, cu_seqlens, y, max_q, chunk, chunks, chunk_state, chunk_decay, decay, s);
+}
+
+// y: float32 [n, H dv]; parts as above (g from column g_col on) or null (no gate); w: float32 [dv] or null; out: [n, H dv].
 #define WICK_GLA_NORM_GATE(NAME, T)                                                                                            \
     WICK_API int NAME(const float* y, const float* parts, int splits, int n, int cols, int g_col, int H, int dv, const float* w, \
                       float eps, void* out, void* s) {                                                                         \

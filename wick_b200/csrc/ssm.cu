@@ -17,10 +17,11 @@
 // arithmetic; a token's numbers depend on its own sequence alone.  A step of few tokens adds them in the same order whatever
 // its shape; a long prompt step scanned in chunks (below) rounds the state differently, and no more than that.
 #include "common.cuh"
+#include "short_conv.cuh"
 
 namespace wick {
 
-constexpr int SSM_MAX_TAPS = 16;
+constexpr int SSM_MAX_TAPS = CONV_MAX_TAPS;
 constexpr int SSM_ROWS = 16;                    // state numbers a thread keeps of one column, at most
 constexpr int SSM_COLS = 4;                     // columns of the state a thread keeps
 
@@ -52,93 +53,7 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int LEFT>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(LEFT) : "memory"); }
 
-__device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
 __device__ __forceinline__ float softplus_f(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
-
-__device__ __forceinline__ float sum_parts(const float* __restrict__ parts, int splits, int64_t split_stride, int64_t at) {
-    float v = 0.f;
-    for (int s = 0; s < splits; ++s) v += parts[s * split_stride + at];
-    return v;
-}
-
-constexpr int SSM_CONV_TOKENS = 4;              // tokens a thread of the convolution takes (their loads are in flight together)
-
-// grid (ceil(tokens / SSM_CONV_TOKENS), ceil(channels / 256)).  ONE: the projection came as a single set of sums (its loads
-// need no loop and go out together).
-template <bool ONE>
-__global__ void __launch_bounds__(256)
-ssm_conv_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, int cols, int first_col, int channels, int taps,
-                const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ state, int64_t record,
-                const int* __restrict__ slots, const int* __restrict__ seq_of_token, const int* __restrict__ positions,
-                const int* __restrict__ start, float* __restrict__ out, int n) {
-    pdl_trigger();
-    pdl_wait();
-    parts = fresh(parts);
-    state = fresh(state);
-    const int c = blockIdx.y * blockDim.x + threadIdx.x;
-    if (c >= channels) return;
-    const float b0 = bias ? bias[c] : 0.f;
-    float acc[SSM_CONV_TOKENS];
-    int pos[SSM_CONV_TOKENS], first[SSM_CONV_TOKENS];
-    const float* rec[SSM_CONV_TOKENS];
-#pragma unroll
-    for (int j = 0; j < SSM_CONV_TOKENS; ++j) {
-        const int t = min(blockIdx.x * SSM_CONV_TOKENS + j, n - 1), b = seq_of_token[t];
-        pos[j] = positions[t];
-        first[j] = start[b];
-        rec[j] = state + (int64_t)slots[b] * record;
-        acc[j] = b0;
-    }
-#pragma unroll 4
-    for (int k = 0; k < taps; ++k) {
-        const float wk = w[(int64_t)c * taps + k];
-        float u[SSM_CONV_TOKENS];
-#pragma unroll
-        for (int j = 0; j < SSM_CONV_TOKENS; ++j) {
-            const int t = min(blockIdx.x * SSM_CONV_TOKENS + j, n - 1), sp = pos[j] - (taps - 1) + k;
-            u[j] = 0.f;
-            const int64_t at = (int64_t)(t - (pos[j] - sp)) * cols + first_col + c;
-            if (sp >= first[j]) u[j] = ONE ? parts[at] : sum_parts(parts, splits, split_stride, at);
-            else if (sp >= 0) u[j] = rec[j][(int64_t)(sp - (first[j] - (taps - 1))) * channels + c];
-        }
-#pragma unroll
-        for (int j = 0; j < SSM_CONV_TOKENS; ++j) acc[j] = fmaf(wk, u[j], acc[j]);
-    }
-#pragma unroll
-    for (int j = 0; j < SSM_CONV_TOKENS; ++j) {
-        const int t = blockIdx.x * SSM_CONV_TOKENS + j;
-        if (t < n) out[(int64_t)t * channels + c] = silu_f(acc[j]);
-    }
-}
-
-// grid (sequences, ceil(channels / 256)).  Runs after the convolution has read the old inputs.
-__global__ void __launch_bounds__(256)
-ssm_conv_state_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, int cols, int first_col, int channels,
-                      int taps, float* __restrict__ state, int64_t record, const int* __restrict__ slots,
-                      const int* __restrict__ cu_seqlens) {
-    pdl_trigger();
-    pdl_wait();
-    parts = fresh(parts);
-    state = fresh(state);
-    const int b = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
-    if (c >= channels) return;
-    const int t0 = cu_seqlens[b], q = cu_seqlens[b + 1] - t0;
-    if (q <= 0) return;
-    float* rec = state + (int64_t)slots[b] * record;
-    float keep[SSM_MAX_TAPS];
-#pragma unroll
-    for (int j = 0; j < SSM_MAX_TAPS; ++j) {
-        if (j >= taps - 1) break;
-        const int from = j + q;                                          // where the input of new place j lies now
-        keep[j] = from >= taps - 1 ? sum_parts(parts, splits, split_stride, (int64_t)(t0 + from - (taps - 1)) * cols + first_col + c)
-                                   : rec[(int64_t)from * channels + c];
-    }
-#pragma unroll
-    for (int j = 0; j < SSM_MAX_TAPS; ++j) {
-        if (j >= taps - 1) break;
-        rec[(int64_t)j * channels + c] = keep[j];
-    }
-}
 
 // The sums of four columns over the LN threads that share them.  Two exchanges halve what a thread carries (it keeps two
 // columns, then one), the rest is a butterfly over one number; `col` is the column a thread ends with and `writes` whether
@@ -512,17 +427,17 @@ WICK_API int wick_ssm_mix(const float* parts, int splits, int n, int cols, int H
                  "ssm_mix: the chunked scan needs room for %d chunks", chunk > 0 ? n / chunk + n_seqs : 0);
     if (n == 0 || n_seqs == 0) return 0;
     const int64_t stride = (int64_t)n * cols;
-    const dim3 conv_grid(ceil_div(n, SSM_CONV_TOKENS), ceil_div(channels, 256));
+    const dim3 conv_grid(ceil_div(n, CONV_TOKENS), ceil_div(channels, 256));
     if (splits == 1) {
-        WICK_CUDA(launch(ssm_conv_kernel<true>, conv_grid, dim3(256), 0, s, parts, splits, stride, cols, inner, channels, taps, conv_w,
-                         conv_b, (const float*)state, record, slots, seq_of_token, positions, start, xbc, n));
+        WICK_CUDA(launch(short_conv_kernel<true, true>, conv_grid, dim3(256), 0, s, parts, splits, stride, cols, inner, channels, taps, conv_w,
+                         taps, 1, conv_b, (const float*)state, record, slots, seq_of_token, positions, start, xbc, n));
     } else {
-        WICK_CUDA(launch(ssm_conv_kernel<false>, conv_grid, dim3(256), 0, s, parts, splits, stride, cols, inner, channels, taps, conv_w,
-                         conv_b, (const float*)state, record, slots, seq_of_token, positions, start, xbc, n));
+        WICK_CUDA(launch(short_conv_kernel<false, true>, conv_grid, dim3(256), 0, s, parts, splits, stride, cols, inner, channels, taps, conv_w,
+                         taps, 1, conv_b, (const float*)state, record, slots, seq_of_token, positions, start, xbc, n));
     }
     if (check_launch("ssm_conv")) return 1;
     if (taps > 1) {
-        WICK_CUDA(launch(ssm_conv_state_kernel, dim3(n_seqs, ceil_div(channels, 256)), dim3(256), 0, s, parts, splits, stride, cols,
+        WICK_CUDA(launch(short_conv_state_kernel, dim3(n_seqs, ceil_div(channels, 256)), dim3(256), 0, s, parts, splits, stride, cols,
                          inner, channels, taps, state, record, slots, cu_seqlens));
         if (check_launch("ssm_conv_state")) return 1;
     }

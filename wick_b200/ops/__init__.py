@@ -587,6 +587,62 @@ def _kv_pages(name: str, kv: torch.Tensor, dtype, n_kv: int, d: int, e: int) -> 
           f"{name} must hold pages of {n_kv} x {PAGE} x ({d} + {e}) elements, is {tuple(kv.shape)}")
 
 
+def block_rows(block: int) -> int:
+    """The most blocks of ``block`` positions that end on one page."""
+    return (PAGE + block - 1) // block
+
+
+def _block_pages(name: str, store: torch.Tensor, dtype, n_kv: int, d: int, e: int, block: int) -> Tuple[int, int]:
+    """(blocks a page holds, elements of a page) of a store of blocks' keys and values."""
+    _cuda(name, store, dtype)
+    _need(block > 0, "a block has a positive number of positions")
+    rows = block_rows(block)
+    page = n_kv * rows * (d + e)
+    _need(store.dim() >= 2 and store[0].numel() == page,
+          f"{name} must hold pages of {n_kv} x {rows} x ({d} + {e}) elements, is {tuple(store.shape)}")
+    return rows, page
+
+
+def pool_blocks(kv: torch.Tensor, store: torch.Tensor, batch, *, n_kv: int, d: int, e: int, block: int, flat: bool = False
+                ) -> Optional[Tuple[torch.Tensor, int]]:
+    """The step's keys and values are in ``kv`` (pages of [n_kv][64][d] keys, then [n_kv][64][e] values): the blocks of ``block``
+    positions that the step completes leave the means of their keys and of their values in ``store``, pages of
+    [n_kv][rows][d], then [n_kv][rows][e], a block on the page of its last position (rows: :func:`block_rows`).  With
+    ``flat`` also returns (array, tiles): all whole blocks of the step's sequences, tile i of sequence b being page b * tiles + i
+    of an array laid out like ``kv``, 64 blocks a page, zeros behind a sequence's last block."""
+    _kv_pages("kv", kv, kv.dtype, n_kv, d, e)
+    rows, page = _block_pages("store", store, kv.dtype, n_kv, d, e, block)
+    blocks, tiles, out = batch.table_width * PAGE // block, 0, None
+    if flat:
+        tiles = max(2, (blocks + 2 * PAGE - 1) // (2 * PAGE) * 2)          # (whole pairs of tiles)
+        blocks = tiles * PAGE
+        out = torch.empty((batch.n_seqs * tiles, n_kv * PAGE * (d + e)), dtype=kv.dtype, device=kv.device)
+    _layer().call(f"wick_pool_blocks_{_dt(kv)}", "ppppippiiiiiiliip", _p(kv), _p(store), _p(out), _p(batch.page_table), batch.table_width,
+                  _p(batch.start), _p(batch.kv_len), batch.n_seqs, n_kv, d, e, int(block), rows, page, blocks, tiles, _stream())
+    return (out, tiles) if flat else None
+
+
+def short_conv(parts: torch.Tensor, w: torch.Tensor, records: Optional[torch.Tensor], batch) -> torch.Tensor:
+    """A causal filter over time, channel by channel, of the first columns of the float32 partial sums ``parts`` [splits, n, cols]:
+    y_t = sum_k w[k] u_(t - taps + 1 + k), zeros before a sequence's start.  ``w``: float32 [taps, channels].  ``records``: float32
+    [slots, (taps - 1) * channels], the inputs of earlier steps, oldest first; brought up to date.  Returns float32 [n, channels]."""
+    _cuda("parts", parts, torch.float32)
+    _cuda("w", w, torch.float32)
+    taps, channels = w.shape
+    _need(parts.dim() == 3 and parts.shape[2] >= channels, f"parts must be [splits, n, {channels} or more], is {tuple(parts.shape)}")
+    splits, n, cols = parts.shape
+    _need(n == batch.n_tokens, f"{n} rows, the batch has {batch.n_tokens} tokens")
+    record = (taps - 1) * channels
+    if record:
+        _cuda("records", records, torch.float32)
+        _need(records.dim() == 2 and records.shape[1] == record, f"records must be [slots, {record}], are {tuple(records.shape)}")
+    out = torch.empty((n, channels), dtype=torch.float32, device=parts.device)
+    _layer().call("wick_short_conv", "piiiiipplpippppp" + "p", _p(parts), splits, n, cols, channels, taps, _p(w), _p(records) if record else None,
+                  record, _p(batch.slots), batch.n_seqs, _p(batch.cu_seqlens), _p(batch.start), _p(batch.seq_of_token), _p(batch.positions),
+                  _p(out), _stream(), kernels=2 if taps > 1 else 1)
+    return out
+
+
 def stream_update(x: torch.Tensor, delta: Optional[torch.Tensor], *, scale: Optional[torch.Tensor] = None,
                   rms: Optional[Tuple[torch.Tensor, float]] = None, norm: Optional[tuple] = None,
                   out_dtype: Optional[torch.dtype] = None, rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
@@ -657,7 +713,8 @@ ATTN_MULTI_MAX_V = 512      # the most numbers of a value row that attention_mul
 def attention_multi(q: torch.Tensor, store: torch.Tensor, batch, scale: float, *, maps: int, kv_heads: int, v_dim: int,
                     window: int = 0, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
                     combine: Optional[Tuple[float, float, float]] = None, rows_of: Optional[int] = None,
-                    out_dtype: torch.dtype) -> torch.Tensor:
+                    out_dtype: torch.dtype, blocks: Optional[Tuple[torch.Tensor, int]] = None, soft_cap: Optional[float] = None,
+                    gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of the step's tokens over the cache (which already holds their own rows) with ``maps`` score maps
     a head.  q: [n, H, maps * dm]; map a scores the a-th dm numbers of a key row and has a softmax of its own; all
     maps weigh the same values.  Visible to the query at position p: with ``window`` > 0 the keys j <= p with
@@ -669,7 +726,10 @@ def attention_multi(q: torch.Tensor, store: torch.Tensor, batch, scale: float, *
 
     maps = 2 with ``combine`` = (lambda, eps, factor): the result is y = y_1 - lambda y_2, then
     y / sqrt(mean(y^2) + eps) * factor over a head's values; q in the activation type.  maps = 1: q is float32 and
-    so is the result.  Returns [n, H, v_dim] in ``out_dtype``."""
+    so is the result, or both have the store's type.  ``blocks`` = (their store, P): beside a window the query also sees the
+    block b of P positions if (b + 1) P <= p + 1 - window, as the one key and value the store holds for it (see
+    :func:`pool_blocks`).  ``soft_cap``: scores s become cap * tanh(s / cap).  ``gate`` (float32 [n, H], one map): a factor of
+    the result.  Returns [n, H, v_dim] in ``out_dtype``."""
     _cuda("q", q)
     n, H, d = q.shape
     _need(maps in (1, 2) and d % maps == 0, f"a head of {d} numbers is not {maps} maps")
@@ -692,9 +752,18 @@ def attention_multi(q: torch.Tensor, store: torch.Tensor, batch, scale: float, *
         name = f"wick_attn_multi2_{_dt(q)}"
         lam, eps, factor = combine
     else:
-        _need(q.dtype == torch.float32 and out_dtype == torch.float32, "one map takes and gives float32")
-        name = f"wick_attn_multi1_{'bf16' if T == torch.bfloat16 else 'f32'}"
+        _need(q.dtype == out_dtype and q.dtype in (torch.float32, T), "one map takes and gives float32, or the store's type")
+        name = f"wick_attn_multi1_{'bf16' if T == torch.bfloat16 else 'f32'}" if q.dtype == torch.float32 else "wick_attn_multi1_act_bf16"
         lam, eps, factor = 0.0, 0.0, 1.0
+    pool, block, pool_rows, pool_page, pool_v = None, 0, 0, 0, 0
+    if blocks is not None:
+        pool, block = blocks
+        pool_rows, pool_page = _block_pages("blocks", pool, T, kv_heads, d, v_dim, block)
+        pool_v = kv_heads * pool_rows * d
+        _need(window > 0 and rows_of is None, "blocks are seen beside a window of keys with values of their own")
+    if gate is not None:
+        _cuda("gate", gate, torch.float32, (n, H))
+        _need(maps == 1, "the factor per head belongs to one map")
     out = torch.empty((n, H, v_dim), dtype=out_dtype, device=q.device)
     # A step of few tokens: eight warps a block, heads that read the same rows together, and the visible keys cut into
     # runs (a block each, records merged by a second kernel) until the step fills the device about twice.  How many keys
@@ -704,7 +773,7 @@ def attention_multi(q: torch.Tensor, store: torch.Tensor, batch, scale: float, *
     if few:
         group = 1 if maps == 2 else (4 if (H // kv_heads) % 4 == 0 else (2 if (H // kv_heads) % 2 == 0 else 1))
         bound = getattr(batch, "kv_bound", None) or batch.max_kv_len
-        keys = min(bound, window + keep_first) if window > 0 else bound
+        keys = min(bound, window + keep_first + (bound // block if block else 0)) if window > 0 else bound
         tiles = (max(1, keys) + 31) // 32
         runs = max(1, min(-(-2 * 148 // (n * (H // group))), tiles // 2, 16))        # (a run is two tiles of 32 keys at least)
         if runs > 1:
@@ -712,9 +781,10 @@ def attention_multi(q: torch.Tensor, store: torch.Tensor, batch, scale: float, *
             ws = getattr(batch, "workspace", None)
             partial = ws.get("attention_multi", need, torch.float32) if ws is not None else \
                 torch.empty(need, dtype=torch.float32, device=q.device)
-    _layer().call(name, "ppppppiiiiiililifiipfffiipp", _p(q), _p(store), _p(out), _p(batch.seq_of_token), _p(batch.positions),
+    _layer().call(name, "ppppppiiiiiililifiipfffiippiillfpp", _p(q), _p(store), _p(out), _p(batch.seq_of_token), _p(batch.positions),
                   _p(batch.page_table), batch.table_width, n, H, kv_heads, dm, v_dim, page_elems, k_row, v_off, v_row, float(scale),
-                  int(window), int(keep_first), _p(sink), float(lam), float(eps), float(factor), few, runs, _p(partial), _stream(),
+                  int(window), int(keep_first), _p(sink), float(lam), float(eps), float(factor), few, runs, _p(partial), _p(pool), int(block),
+                  pool_rows, pool_page, pool_v, float(soft_cap or 0.0), _p(gate), _stream(),
                   kernels=2 if partial is not None else 1)
     return out
 
@@ -816,13 +886,16 @@ def flex_source(t: Optional[torch.Tensor] = None, *, tile_elems: int = 0, const_
 
 def attention_flex(q: torch.Tensor, k0: List[int], k1: List[int], v: List[int], batch, scale: float, *, dv: int, window: int = 0,
                    keep_first: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                   gate_parts: Optional[Tuple[torch.Tensor, int]] = None, out_dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
+                   gate_parts: Optional[Tuple[torch.Tensor, int]] = None, out_dtype: torch.dtype = torch.bfloat16,
+                   blocks: Optional[Tuple[torch.Tensor, int, int]] = None, soft_cap: Optional[float] = None) -> torch.Tensor:
     """Attention of a prompt's tokens on the tensor cores.  q: bfloat16 [n, heads, dk]; a key row is ``k0``'s numbers
     followed by ``k1``'s (sources as :func:`flex_source` makes them; flat sources need sequences that start at position
     0), a value row ``v``'s.  Visible to the query at position p: the keys j <= p with p - j < window or j < keep_first
     (window 0: every j <= p).  ``sink`` float32 [heads]; ``gate`` float32 [n, heads], a factor of the bfloat16 result;
     ``gate_parts`` = (float32 partial sums [splits, n, cols], first column): the bfloat16 result is multiplied element by
-    element by the sigmoid of the heads * dv columns' sums.
+    element by the sigmoid of the heads * dv columns' sums.  ``blocks`` = (array, tiles, P) as :func:`pool_blocks` makes them, laid out
+    like the (one, paged) source: beside the window the query sees the blocks of P positions that lie wholly before it.
+    ``soft_cap``: scores s become cap * tanh(s / cap).
     Returns [n, heads, dv] in ``out_dtype`` (float32 or bfloat16)."""
     import numpy as np
     _cuda("q", q, torch.bfloat16)
@@ -838,10 +911,15 @@ def attention_flex(q: torch.Tensor, k0: List[int], k1: List[int], v: List[int], 
     _need(gp is None or (gate is None and out_dtype == torch.bfloat16), "one gate, a factor of the bfloat16 result")
     out = torch.empty((n, heads, dv), dtype=out_dtype, device=q.device)
     src = np.asarray(k0 + k1 + v, dtype=np.int64)
-    _flex(dk, dv).call("wick_attn_flex_bf16", "pppppppippiiiiifpiliip", _p(q), src.ctypes.data, _p(out) if out_dtype == torch.float32 else None,
+    pool, pool_tiles, block = blocks if blocks is not None else (None, 0, 0)
+    if pool is not None:
+        _cuda("blocks", pool, torch.bfloat16)
+        _need(pool.dim() == 2 and pool.shape[0] >= batch.n_seqs * pool_tiles and pool.shape[1] == k0[1], "the blocks' array is laid out like the source")
+    _flex(dk, dv).call("wick_attn_flex_bf16", "pppppppippiiiiifpiliipiifp", _p(q), src.ctypes.data, _p(out) if out_dtype == torch.float32 else None,
                        _p(out) if out_dtype == torch.bfloat16 else None, _p(gate), _p(sink), _p(batch.cu_seqlens), batch.n_seqs,
                        _p(batch.start), _p(batch.page_table), batch.table_width, attention_tiles(batch), heads, int(window),
-                       int(keep_first), float(scale), _p(gp), g_splits, n * g_cols, g_cols, g_col, _stream())
+                       int(keep_first), float(scale), _p(gp), g_splits, n * g_cols, g_cols, g_col, _p(pool), int(pool_tiles), int(block),
+                       float(soft_cap or 0.0), _stream())
     return out
 
 
@@ -905,7 +983,9 @@ def qkv_finish(parts: torch.Tensor, n_heads: int, n_kv: int, d: int, e: int, *, 
                blend: Optional[torch.Tensor] = None, kv: Optional[torch.Tensor], page_table: torch.Tensor,
                seq_of_token: torch.Tensor, positions: torch.Tensor, write_kv: bool = True,
                q_span: Optional[int] = None, k_span: Optional[int] = None, norm_after_rotation: bool = False,
-               keys_are_values: bool = False) -> torch.Tensor:
+               keys_are_values: bool = False, conv: Optional[Tuple[torch.Tensor, Optional[torch.Tensor], torch.Tensor]] = None,
+               v_eps: Optional[float] = None, gate: Optional[Tuple[torch.Tensor, int, torch.Tensor]] = None,
+               blocks: Optional[Tuple[torch.Tensor, int]] = None) -> torch.Tensor:
     """From the q/k/v projection's float32 partial sums ``parts`` [splits, n, H d + G d + G e (+ more)]:
     biases, RMS norms of q and k over spans the length of their weight vectors (a head, or the
     whole projection; ``q_span`` / ``k_span`` without a weight vector: the span is divided by its root
@@ -916,7 +996,11 @@ def qkv_finish(parts: torch.Tensor, n_heads: int, n_kv: int, d: int, e: int, *, 
     (``v_mode`` 1: the values are also kept in ``v_keep`` [n, G e]; 2: v <- (1 - blend) v + blend
     v_keep), then q -> the result [n, H, d] in ``dtype`` and k, v -> the token's place in ``kv``.
     ``keys_are_values``: the rows hold no values; a head's value is its key as projected, before norm
-    and rotation.  Columns behind q, k and v (an output gate's) are left alone."""
+    and rotation.  Columns behind q, k and v (an output gate's) are left alone.
+    ``v_eps``: every head's values are divided by their root mean square.  ``gate`` = (float32 partial sums [splits, n, cols], first
+    column, float32 [n, heads] to write): the sigmoids of the columns' sums.  For steps of one token per sequence only:
+    ``conv`` = (w, records, slots), the filter of :func:`short_conv` over q, k and v before everything else; ``blocks`` = (store, P):
+    the token that completes a block of P positions leaves the block's means (see :func:`pool_blocks`)."""
     _cuda("parts", parts, torch.float32)
     W = (n_heads + n_kv) * d + (0 if keys_are_values else n_kv * e)
     _need(parts.dim() == 3 and parts.shape[2] >= W, f"parts must be [splits, n, {W} or more], is {tuple(parts.shape)}")
@@ -945,11 +1029,38 @@ def qkv_finish(parts: torch.Tensor, n_heads: int, n_kv: int, d: int, e: int, *, 
     q_out = torch.empty((n, n_heads, d), dtype=dtype, device=parts.device)
     _need(maps >= 1 and d % maps == 0, f"a head of {d} numbers is not {maps} vectors")
     flags = (1 if keys_are_values else 0) | (2 if norm_after_rotation else 0)
-    _layer().call(f"wick_qkv_finish_{_dt(q_out)}", "piipiiiipipifppiiipippppippiiip", _p(parts), parts.shape[0], n, _p(bias),
+    conv_w = conv_rec = slots = None
+    taps = record = 0
+    if conv is not None:
+        conv_w, conv_rec, slots = conv
+        _cuda("conv's w", conv_w, torch.float32)
+        taps = conv_w.shape[0]
+        record = (taps - 1) * W
+        _need(conv_w.dim() == 2 and conv_w.shape[1] == W, f"the filters must be [taps, {W}], are {tuple(conv_w.shape)}")
+        if record:
+            _cuda("conv's records", conv_rec, torch.float32)
+            _need(conv_rec.dim() == 2 and conv_rec.shape[1] == record, f"records must be [slots, {record}], are {tuple(conv_rec.shape)}")
+        _cuda("slots", slots, torch.int32, (n,))
+    gp = g_out = None
+    g_splits = g_cols = g_col = g_heads = 0
+    if gate is not None:
+        gp, g_col, g_out = gate
+        _cuda("gate's sums", gp, torch.float32)
+        g_heads = g_out.shape[1]
+        _cuda("gate's result", g_out, torch.float32, (n, g_heads))
+        _need(gp.dim() == 3 and gp.shape[1] == n and g_col + g_heads <= gp.shape[2], "the gate's columns lie beyond its rows")
+        g_splits, g_cols = gp.shape[0], gp.shape[2]
+    pool, block, pool_rows, pool_page = None, 0, 0, 0
+    if blocks is not None:
+        pool, block = blocks
+        pool_rows, pool_page = _block_pages("blocks", pool, dtype, n_kv, d, e, block)
+    _layer().call(f"wick_qkv_finish_{_dt(q_out)}", "piipiiiipipifppiiipippppippiii" + "pplpiifppiiiipiil" + "p", _p(parts), parts.shape[0], n, _p(bias),
                   n_heads, n_kv, d, e, _p(q_weight), int(q_span or 0), _p(k_weight), int(k_span or 0), float(eps), _p(cos), _p(sin),
                   rot_dims if cos is not None else 0, PAIRINGS[pairing], int(maps), _p(v_keep), v_mode, _p(blend), _p(q_out),
                   _p(kv) if write_kv else None, _p(page_table), page_table.shape[-1], _p(seq_of_token), _p(positions),
-                  1 if write_kv else 0, int(cols), flags, _stream())
+                  1 if write_kv else 0, int(cols), flags, _p(conv_w), _p(conv_rec) if record else None, record, _p(slots), taps,
+                  1 if v_eps is not None else 0, float(v_eps or 0.0), _p(g_out), _p(gp), g_splits, g_cols, int(g_col), g_heads,
+                  _p(pool), int(block), pool_rows, pool_page, _stream())
     return q_out
 
 
@@ -1059,6 +1170,56 @@ def attention_masked(q: torch.Tensor, kv: torch.Tensor, batch, scale: float, *, 
                   _p(batch.positions), _p(batch.page_table), batch.table_width, n, n_heads, n_kv, d, v_dim, float(scale),
                   MASKS[mask], int(mask_size), _p(sink), _stream())
     return out
+
+
+def attention_pooled_kind(d: int, v_dim: int, dtype: torch.dtype, is_decode: bool, plain: bool = False) -> str:
+    """Which kernel :func:`attention_pooled` runs: for a prompt's tokens in bfloat16 ``tc`` (tcgen05: keys and values of one size, 64
+    or 128) or ``mma`` (mma.sync: other multiples of 16 that :func:`attention_flex` takes); else, and as the twin the former are
+    checked against, ``rows`` (:func:`attention_multi`: CUDA cores, row by row)."""
+    if plain or PLAIN_KERNELS or is_decode or dtype != torch.bfloat16:
+        return "rows"
+    if d == v_dim and d in (64, 128):
+        return "tc"
+    return "mma" if attention_flex_supported(d, v_dim, dtype) else "rows"
+
+
+def attention_pooled(q: torch.Tensor, kv: torch.Tensor, batch, scale: float, *, n_kv: int, v_dim: int, window: int = 0,
+                     store: Optional[torch.Tensor] = None, block: int = 0, pooled: bool = False, soft_cap: Optional[float] = None,
+                     gate: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, kind: Optional[str] = None) -> torch.Tensor:
+    """Attention of the step's tokens over the cache, which already holds their keys and values, with a window (0: every earlier
+    key) beside which the blocks of ``block`` positions before it are seen by their mean keys and values (``store``; 0: they are
+    not seen), scores soft-capped by ``soft_cap`` and results times ``gate`` (float32 [n, H]), each where given.  The blocks that the
+    step completes are brought into the store first, unless that is done (``pooled``).  q [n, H, d] -> [n, H, v_dim]."""
+    _cuda("q", q)
+    n, H, d = q.shape
+    kind = kind or attention_pooled_kind(d, v_dim, q.dtype, batch.is_decode)
+    _need(kind == "rows" or q.dtype == torch.bfloat16, "the tensor-core attention kernels take bfloat16")
+    _need(not (block and pooled) or kind == "rows", "the tensor-core attention kernels read the blocks from an array of this step")
+    flat, tiles = None, 0
+    if block and not pooled:
+        res = pool_blocks(kv, store, batch, n_kv=n_kv, d=d, e=v_dim, block=block, flat=kind != "rows")
+        flat, tiles = res if res is not None else (None, 0)
+    if kind == "rows":
+        return attention_multi(q, kv, batch, scale, maps=1, kv_heads=n_kv, v_dim=v_dim, window=window, sink=sink, out_dtype=q.dtype,
+                               blocks=(store, block) if block else None, soft_cap=soft_cap, gate=gate)
+    _kv_pages("kv", kv, q.dtype, n_kv, d, v_dim)
+    _need(n == batch.n_tokens, f"q has {n} rows, the batch {batch.n_tokens} tokens")
+    if sink is not None:
+        _cuda("sink", sink, torch.float32, (H,))
+    if gate is not None:
+        _cuda("gate", gate, torch.float32, (n, H))
+    if kind == "tc":
+        out = torch.empty((n, H, v_dim), dtype=q.dtype, device=q.device)
+        _attn(d).call("wick_attn_prompt_tc_pooled_bf16", "plplpipippiiifpiippiifpp", _p(q), n, _p(kv), kv.shape[0], _p(out), attention_tiles(batch),
+                      _p(batch.cu_seqlens), batch.n_seqs, _p(batch.start), _p(batch.page_table), batch.table_width, H, n_kv, float(scale),
+                      _p(status_tensor(q.device)), MASKS["window" if window else "causal"], int(window), _p(sink), _p(flat), tiles, int(block),
+                      float(soft_cap or 0.0), _p(gate), _stream())
+        return out
+    page = n_kv * PAGE * (d + v_dim)
+    k0 = flex_source(kv, tile_elems=page, hdiv=H // n_kv, hmul=PAGE * d, row_stride=d, length=d, paged=True)
+    v = flex_source(kv, tile_elems=page, const_off=n_kv * PAGE * d, hdiv=H // n_kv, hmul=PAGE * v_dim, row_stride=v_dim, length=v_dim, paged=True)
+    return attention_flex(q, k0, flex_source(), v, batch, scale, dv=v_dim, window=window, sink=sink, gate=gate,
+                          blocks=(flat, tiles, block) if block else None, soft_cap=soft_cap)
 
 
 def moe_table_up(x: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, gate_up: torch.Tensor) -> torch.Tensor:
@@ -1290,10 +1451,35 @@ def hgrn2_mix(parts: torch.Tensor, *, heads: int, key_dim: int, v_dim: int, bias
     return y
 
 
-def _gla_scratch(n: int, hk: int, hv: int, key_dim: int, batch, device):
-    """What a linear attention's kernels write on the way: the tokens' rows [q | k | a | v], o, and (steps of many tokens) the
-    chunks' states and decays."""
-    qkav = torch.empty((n, 3 * hk + hv), dtype=torch.float32, device=device)
+def retention_mix(parts: torch.Tensor, *, heads: int, key_dim: int, v_dim: int, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor],
+                  rot_dims: int, k_scale: float, decay: torch.Tensor, records: torch.Tensor, batch) -> torch.Tensor:
+    """The recurrence with a fixed decay per head.  ``parts``: the input projection's float32 partial sums [splits, n, cols], a row laid out
+    [q: H dk | k: H dk | v: H dv] and whatever follows.  Pairs (i, i + rot_dims / 2) of the first ``rot_dims`` elements of every q and k
+    head turn by the angles of ``cos`` / ``sin`` [n, rot_dims / 2], k is multiplied by ``k_scale``; per head S <- decay S + k v^T
+    (``decay`` float32 [H]) and o = S^T q.  ``records`` as for :func:`gla_mix`.  Returns o float32 [n, H dv]."""
+    _cuda("parts", parts, torch.float32)
+    hk, hv = heads * key_dim, heads * v_dim
+    _need(parts.dim() == 3 and parts.shape[2] >= 2 * hk + hv, f"parts must be [splits, n, {2 * hk + hv} or more], are {tuple(parts.shape)}")
+    splits, n, cols = parts.shape
+    if rot_dims:
+        _cuda("cos", cos, torch.float32, (n, rot_dims // 2))
+        _cuda("sin", sin, torch.float32, (n, rot_dims // 2))
+    _cuda("decay", decay, torch.float32, (heads,))
+    _cuda("records", records, torch.float32)
+    _need(records.dim() == 2 and records.shape[1] == hv * key_dim, f"records must be [slots, {hv * key_dim}], are {tuple(records.shape)}")
+    _need(n == batch.n_tokens, f"{n} rows, the batch has {batch.n_tokens} tokens")
+    qkv, y, max_q, chunk, chunks, chunk_state, chunk_decay = _gla_scratch(n, hk, hv, key_dim, batch, parts.device, vectors=2)
+    _layer().call("wick_retention_mix", "piiiiiippifpplpipppiiippp", _p(parts), splits, n, cols, heads, key_dim, v_dim, _p(cos) if rot_dims else None,
+                  _p(sin) if rot_dims else None, int(rot_dims), float(k_scale), _p(decay), _p(records), hv * key_dim, _p(batch.slots), batch.n_seqs,
+                  _p(batch.cu_seqlens), _p(qkv), _p(y), max_q, chunk, chunks, _p(chunk_state), _p(chunk_decay), _stream(),
+                  kernels=1 + (3 if chunks else 1))
+    return y
+
+
+def _gla_scratch(n: int, hk: int, hv: int, key_dim: int, batch, device, vectors: int = 3):
+    """What a linear attention's kernels write on the way: the tokens' rows [q | k | a | v] (``vectors`` 2: [q | k | v]), o, and (steps of
+    many tokens) the chunks' states and decays."""
+    qkav = torch.empty((n, vectors * hk + hv), dtype=torch.float32, device=device)
     y = torch.empty((n, hv), dtype=torch.float32, device=device)
     max_q = 1 if batch.is_decode else 0          # (0: unknown to the host, as in a captured prompt step)
     chunk, chunks, chunk_state, chunk_decay = GLA_CHUNK, 0, None, None
@@ -1304,10 +1490,10 @@ def _gla_scratch(n: int, hk: int, hv: int, key_dim: int, batch, device):
     return qkav, y, max_q, chunk, chunks, chunk_state, chunk_decay
 
 
-def gla_norm_gate(y: torch.Tensor, parts: Optional[torch.Tensor], g_col: int, heads: int, v_dim: int, weight: torch.Tensor, eps: float,
-                  dtype: torch.dtype) -> torch.Tensor:
+def gla_norm_gate(y: torch.Tensor, parts: Optional[torch.Tensor], g_col: int, heads: int, v_dim: int, weight: Optional[torch.Tensor],
+                  eps: float, dtype: torch.dtype) -> torch.Tensor:
     """Every head's ``v_dim`` numbers of y (float32 [n, H dv]) divided by their root mean square and multiplied by ``weight``
-    (float32 [dv], shared by the heads), then by silu(g), g the columns from ``g_col`` on of the float32 partial sums
+    (float32 [dv], shared by the heads; None: no factor), then by silu(g), g the columns from ``g_col`` on of the float32 partial sums
     ``parts`` [splits, n, cols] (``parts`` None: no gate); [n, H dv] in ``dtype``."""
     _cuda("y", y, torch.float32)
     n = y.shape[0]
@@ -1315,7 +1501,8 @@ def gla_norm_gate(y: torch.Tensor, parts: Optional[torch.Tensor], g_col: int, he
     if parts is not None:
         _cuda("parts", parts, torch.float32)
         _need(parts.dim() == 3 and parts.shape[1] == n and parts.shape[2] >= g_col + heads * v_dim, "parts must hold the gate's columns")
-    _cuda("weight", weight, torch.float32, (v_dim,))
+    if weight is not None:
+        _cuda("weight", weight, torch.float32, (v_dim,))
     out = torch.empty((n, heads * v_dim), dtype=dtype, device=y.device)
     _layer().call(f"wick_gla_norm_gate_{_dt(out)}", "ppiiiiiipfpp", _p(y), _p(parts), 1 if parts is None else parts.shape[0], n,
                   0 if parts is None else parts.shape[2], int(g_col), heads,

@@ -115,7 +115,8 @@ def compile_library(name: str, sources: Sequence[str], defines: Sequence[str] = 
                 return out
             nvcc = find_nvcc()
             tmp = f"{out}.{os.getpid()}.tmp"
-            cmd = [nvcc] + flags + ["-I", CSRC, "-o", tmp] + srcs
+            # (a library's sources are compiled side by side)
+            cmd = [nvcc, "--threads", str(max(1, min(len(srcs), os.cpu_count() or 1)))] + flags + ["-I", CSRC, "-o", tmp] + srcs
             if verbose:
                 _note(f"compiling {name} for sm_100a ({', '.join(os.path.basename(s) for s in srcs)}) ...")
             t0 = time.time()

@@ -88,7 +88,8 @@ class CacheNeed:
 
     kind ``paged_kv``: keys and values of every position, ``kv_heads`` x
     ``head_dim`` each, in pages (values ``v_head_dim`` each, if that is given and
-    differs); ``window`` (tokens) if only the last ones are ever read.  kind ``paged_rows``:
+    differs); ``window`` (tokens) if only the last ones are ever read.  kind ``paged_blocks``: a key and a value for every
+    whole block of ``block`` positions, on the page of the block's last position.  kind ``paged_rows``:
     one row of ``shape`` per position, in the same pages.  kind ``state``: one record of fixed
     ``shape`` and ``dtype`` per sequence, zeroed when the sequence starts.  kind ``several``:
     a mixer made of several keeps what each of ``parts`` asks for; its cache view's ``parts``
@@ -102,6 +103,7 @@ class CacheNeed:
     dtype: Optional[torch.dtype] = None   # None: the compute dtype
     v_head_dim: Optional[int] = None      # None: as head_dim
     parts: Tuple["CacheNeed", ...] = ()
+    block: int = 0
 
 
 class Part:
@@ -219,7 +221,10 @@ class FeedForward(Part):
     category = "ffn"
 
     def forward(self, x: torch.Tensor, batch: "Any") -> torch.Tensor:
-        """x: [tokens, width], compute dtype.  Returns float32 [splits, tokens, width]."""
+        """x: [tokens, width], compute dtype.  Returns float32 [splits, tokens, width].
+
+        A feed-forward whose class sets ``JOINS_BESIDE = True`` can also be given ``beside=`` (float32 [splits, tokens,
+        width], what another sublayer made of the same input): its last kernel then adds that to its result."""
         raise NotImplementedError
 
 

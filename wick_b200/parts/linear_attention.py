@@ -1,4 +1,4 @@
-"""Linear attentions with a decay per key channel as mixers.
+"""Linear attentions with a decay, per key channel or fixed per head, as mixers.
 
 =============  ===========================  ==========================================
 category       kind                         params
@@ -14,6 +14,12 @@ mixer          ``hgrn2``                    width, heads, head_dim (key channels
                                             head), v_dim, eps, names (q, forget,
                                             forget_bias, lower, v, norm, o -> local
                                             names)
+mixer          ``retention``                width, heads, head_dim (key channels of a
+                                            head), v_dim, decay (a number per head),
+                                            eps, k_scale (default head_dim^(-1/2)),
+                                            position (PartSpec ``rotary_pairs`` of
+                                            pairing ``halves``, or None), names (q, k,
+                                            v, gate, o -> local names)
 =============  ===========================  ==========================================
 
 ``gated_linear_attention``, with h the mixer's input, H heads of dk key channels and dv value numbers:
@@ -34,6 +40,14 @@ mixer          ``hgrn2``                    width, heads, head_dim (key channels
   (1 - l) sigmoid(-z)) where it has a key;
 * the per-head norm above, no gate, Wo.
 
+``retention``, with the same letters:
+
+* q = Wq h, k = Wk h (H x dk each), v = Wv h (H x dv), g = Wg h (H x dv): one matrix product; the position encoding turns q
+  and k, k is multiplied by ``k_scale`` afterwards;
+* per head S <- a S + k v^T with the head's fixed number a, o = S^T q;
+* every head's o is divided by its root mean square (no weight); the heads side by side are multiplied by silu(g) and go
+  through Wo.
+
 The state is one float32 record per sequence (kind ``state`` of the cache: zero when a sequence starts), read and brought
 up to date by every step whatever its shape.  Everything between the two matrix products is float32, W2's product
 included (W2 is held in float32; its rank is small).
@@ -43,8 +57,11 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from .base import CacheNeed, Mixer, TensorSpec, register_part
+from ..models.spec import PartSpec
+from .attention import RotaryPairs
+from .base import CacheNeed, Mixer, TensorSpec, build_part, register_part
 from .linear import Linear
+from .standard import NoPosition
 
 
 class GatedLinearAttention(Mixer):
@@ -186,4 +203,68 @@ class Hgrn2(Mixer):
 
 
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
+class Retention(Mixer):
+    PROMPT_CAPTURABLE = True
+
+    def __init__(self, params, ctx):
+        super().__init__(params, ctx)
+        p = params
+        self.width, self.heads = int(p["width"]), int(p["heads"])
+        self.key_dim, self.v_dim, self.eps = int(p["head_dim"]), int(p["v_dim"]), float(p["eps"])
+        decay = [float(a) for a in p["decay"]]
+        if self.heads <= 0 or self.key_dim <= 0 or self.v_dim <= 0 or len(decay) != self.heads:
+            raise ValueError("heads, head_dim and v_dim must be positive, and every head has a decay")
+        self.decay = torch.tensor(decay, dtype=torch.float32, device=ctx.device)
+        self.k_scale = float(p["k_scale"]) if p.get("k_scale") is not None else self.key_dim ** -0.5
+        self.position = build_part("position", p.get("position") or PartSpec("none"), ctx)
+        if not isinstance(self.position, NoPosition) and not (
+                isinstance(self.position, RotaryPairs) and self.position.pairing == "halves" and self.position.head_dim == self.key_dim):
+            raise ValueError("this mixer's kernel turns half-split pairs (rotary_pairs) of its heads or nothing")
+        self.hk, self.hv = self.heads * self.key_dim, self.heads * self.v_dim
+        names = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", gate="g_proj.weight", o="o_proj.weight")
+        names.update(p.get("names") or {})
+        self.names = names
+        self.input = Linear(2 * self.hk + 2 * self.hv, self.width, ctx)      # rows: q, k, v, gate
+        self.o = Linear(self.width, self.hv, ctx)
+
+    def tensor_specs(self):
+        nm = self.names
+        return [TensorSpec(nm["q"], (self.hk, self.width)), TensorSpec(nm["k"], (self.hk, self.width)),
+                TensorSpec(nm["v"], (self.hv, self.width)), TensorSpec(nm["gate"], (self.hv, self.width)),
+                TensorSpec(nm["o"], (self.width, self.hv))]
+
+    def load(self, fetch):
+        nm = self.names
+        self.input.load_rows([fetch(nm[k]) for k in ("q", "k", "v", "gate")])
+        self.o.load_rows([fetch(nm["o"])])
+
+    def tensor(self, name):
+        nm, hk, hv = self.names, self.hk, self.hv
+        spans = {nm["q"]: (0, hk), nm["k"]: (hk, 2 * hk), nm["v"]: (2 * hk, 2 * hk + hv), nm["gate"]: (2 * hk + hv, 2 * hk + 2 * hv)}
+        if name in spans:
+            return self.input.rows(*spans[name])
+        return self.o.rows(0, self.width) if name == nm["o"] else None
+
+    def record_floats(self) -> int:
+        return self.hv * self.key_dim
+
+    def cache_need(self):
+        return CacheNeed("state", shape=(self.record_floats(),), dtype=torch.float32)
+
+    def weight_bytes(self):
+        return self.input.weight_bytes() + self.o.weight_bytes()
+
+    def forward(self, x, batch, cache, write_cache):
+        if not write_cache:
+            raise RuntimeError("a linear-attention mixer keeps its own record; it cannot read another entry's")
+        parts = self.input.forward_delta(x)                         # float32 [splits, n, 2 H dk + 2 H dv]
+        rot = self.position if isinstance(self.position, RotaryPairs) else None
+        cos, sin = rot.tables(batch) if rot else (None, None)
+        y = ops.retention_mix(parts, heads=self.heads, key_dim=self.key_dim, v_dim=self.v_dim, cos=cos, sin=sin, rot_dims=rot.dims if rot else 0,
+                              k_scale=self.k_scale, decay=self.decay, records=cache.state, batch=batch)
+        g = ops.gla_norm_gate(y, parts, 2 * self.hk + self.hv, self.heads, self.v_dim, None, self.eps, self.ctx.dtype)
+        return self.o.forward_delta(g)
+
+
 register_part("mixer", "hgrn2", Hgrn2)
+register_part("mixer", "retention", Retention)

@@ -30,7 +30,8 @@ outputs of s_i r_i (the chosen scores divided by their sum + ``norm_eps`` first,
 matrix) for an expert with matrices and r_i = h for one of the last ``identity`` outputs.  ``groups``: the
 experts form ``count`` equal groups of neighbours; a group's score is the sum of its two largest s + correction,
 and only experts of the ``keep`` best groups can be chosen.  ``shared``: a feed-forward that runs for every
-token; its result is added, with ``shared_gate`` times sigmoid(w_sg . h), one number per token (float32).
+token; its result is added, with ``shared_gate`` times sigmoid(w_sg . h), one number per token (float32).  What another
+sublayer made of the same input (``beside``) joins the sum in the kernel that adds up the experts' results.
 
 The experts' products reuse the kernels of the experts chosen by a table: the router's choice,
 [tokens, top], is such a table with the token's number as its row.  From ``SORTED_FROM`` tokens on
@@ -51,6 +52,7 @@ from .linear import Linear
 
 class RoutedMoE(FeedForward):
     PROMPT_CAPTURABLE = True
+    JOINS_BESIDE = True
     SORTED_FROM = 16
     ROW_TILE = 256
 
@@ -159,14 +161,16 @@ class RoutedMoE(FeedForward):
             n += self.shared.weight_bytes()
         return n
 
-    def forward(self, x, batch):
+    def forward(self, x, batch, beside=None):
+        if beside is not None and self.shared is not None:           # (the kernel takes one term beside the experts)
+            return ops.weighted_sum([(beside, 1.0), (self.forward(x, batch), 1.0)])
         n = x.shape[0]
         logits = self.router.forward_delta(x)                        # float32 [splits, n, outputs (+ 1: the shared expert's gate)]
         choice, weight, ident = ops.moe_router(logits, self.correction, self.top, renormalize=self.renormalize, scores=self.scores,
                                                groups=self.group_count, keep=self.group_keep, scale=self.route_scale,
                                                norm_eps=self.norm_eps, outputs=self.outputs)
         own = x if self.identity else None
-        base = base_gate = None
+        base, base_gate = beside, None
         if self.shared is not None:
             base = as_splits(self.shared.forward(x, batch))
             if self.has_shared_gate:

@@ -26,6 +26,8 @@ block          ``prenorm_residual``    width and layer_scale (mixer, ffn -> loca
                                        they are normed before the sum
 block          ``postnorm_residual``   alpha
 block          ``normed_sum_residual`` —
+block          ``parallel_residual``   width, factor (of the layer's sum, default 1)
+norm           ``none``                —
 embedding      ``table``               vocab, width, tensor, scale (a factor of
                                        the rows, default 1), position (None or
                                        {"kind": "sinusoid", "base": b}: a vector
@@ -117,6 +119,14 @@ class RMSNorm(Norm):
 
     def weight_bytes(self):
         return self.width * 4
+
+
+class NoNorm(Norm):
+    """No norm: what stands where a block reads one norm only."""
+    PROMPT_CAPTURABLE = True
+
+    def forward(self, x, out_dtype, rows=None):
+        raise RuntimeError("a norm of kind 'none' is never run")
 
 
 class TanhNorm(Norm):
@@ -541,6 +551,43 @@ class NormedSumResidual(Block):
         return h
 
 
+class ParallelResidual(Block):
+    """x <- x + factor (mixer(h) + ffn(h)) with h = norm1(x): both sublayers read the output of the layer's one norm (its
+    second norm is of kind ``none``).  The mixer's partial sums join the feed-forward's last kernel where it takes them, and
+    the layer's sum stays pending with its factor for the next norm.  A layer whose feed-forward is of kind ``none`` adds its
+    mixer's result alone."""
+
+    PROMPT_CAPTURABLE = True
+
+    def __init__(self, params, ctx, mixer, mixer_norm, ffn, ffn_norm):
+        super().__init__(params, ctx, mixer, mixer_norm, ffn, ffn_norm)
+        if not isinstance(ffn_norm, NoNorm):
+            raise ValueError("sublayers side by side share one norm: the second one is of kind 'none'")
+        factor = float(params.get("factor", 1.0))
+        self.scale = None if factor == 1.0 else torch.full((int(params["width"]),), factor, dtype=torch.float32, device=ctx.device)
+
+    def forward(self, h, batch, cache, write_cache):
+        dt = self.ctx.dtype
+        h.act = None
+        if h.pending is None:
+            xn = self.mixer_norm.forward(h.x, dt)
+        elif h.scale is not None or h.rms is not None:
+            xn = self.mixer_norm.add_forward(h.x, h.pending, dt, scale=h.scale, rms=h.rms)
+        else:
+            xn = self.mixer_norm.add_forward(h.x, h.pending, dt)
+        h.defer(None)
+        d = as_splits(self.mixer.forward(xn, batch, cache, write_cache))
+        if not getattr(self.ffn, "IS_NONE", False):
+            if getattr(self.ffn, "JOINS_BESIDE", False):
+                d = as_splits(self.ffn.forward(xn, batch, beside=d))
+            else:
+                d = ops.weighted_sum([(d, 1.0), (as_splits(self.ffn.forward(xn, batch)), 1.0)])
+        h.defer(d, self.scale)
+        if self.side is not None:
+            self.side.forward(h, batch)
+        return h
+
+
 # ---------------------------------------------------------------------------
 class TableEmbedding(Embedding):
     """x = table[token] * scale (+ the position's vector) (+ the pair's row).  ``position`` of kind ``sinusoid``: element 2 i of position p's
@@ -660,6 +707,7 @@ class LinearHead(Head):
 
 register_part("norm", "rms", RMSNorm)
 register_part("norm", "tanh", TanhNorm)
+register_part("norm", "none", NoNorm)
 register_part("position", "rotary_half_split", RotaryHalfSplit)
 register_part("position", "none", NoPosition)
 register_part("mixer", "gqa_attention", GQAttention)
@@ -667,5 +715,6 @@ register_part("ffn", "gated_mlp", GatedMLP)
 register_part("block", "prenorm_residual", PreNormResidual)
 register_part("block", "postnorm_residual", PostNormResidual)
 register_part("block", "normed_sum_residual", NormedSumResidual)
+register_part("block", "parallel_residual", ParallelResidual)
 register_part("embedding", "table", TableEmbedding)
 register_part("head", "linear", LinearHead)
