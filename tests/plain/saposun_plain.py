@@ -141,20 +141,23 @@ def projected(h, t, pre: str, m: dict, eps: float):
     return turn(make("q", H, d), base, dims, True), turn(make("k", G, d), base, dims, True), rms(make("v", G, e), eps)
 
 
-def window_attention(h, t, pre: str, m: dict, eps: float) -> torch.Tensor:
-    n = h.shape[0]
-    H, G, e = m["heads"], m["kv_heads"], m["vdim"]
-    q, k, v = projected(h, t, pre, m, eps)
-    size = m["mask"]["size"] if m.get("mask") else None
+def attend(q, k, v, scale: float, size: Optional[int], P: Optional[int], cap: Optional[float]) -> torch.Tensor:
+    """q [n, H, d], k [n, G, d], v [n, G, e] -> [n, H, e]: tokens of the window and blocks before it in one softmax."""
+    n, H, G = q.shape[0], q.shape[1], k.shape[1]
     vis = in_window(n, size)
-    P = (m.get("mask") or {}).get("pool")
     if P:
         k, v = torch.cat([k, pooled(k, P)]), torch.cat([v, pooled(v, P)])
         vis = torch.cat([vis, sees_block(n, size, P)], 1)
     kk, vv = k.repeat_interleave(H // G, dim=1), v.repeat_interleave(H // G, dim=1)
-    s = capped(torch.einsum("ihd,jhd->hij", q, kk) * m["scale"], m.get("softcap"))
-    out = torch.einsum("hij,jhe->ihe", softmax_over(s, vis), vv)
-    return (out * torch.sigmoid(h @ t[pre + "g"].T)[:, :, None]).reshape(n, H * e) @ t[pre + "o"].T
+    s = capped(torch.einsum("ihd,jhd->hij", q, kk) * scale, cap)
+    return torch.einsum("hij,jhe->ihe", softmax_over(s, vis), vv)
+
+
+def window_attention(h, t, pre: str, m: dict, eps: float) -> torch.Tensor:
+    q, k, v = projected(h, t, pre, m, eps)
+    mask = m.get("mask") or {}
+    out = attend(q, k, v, m["scale"], mask.get("size"), mask.get("pool"), m.get("softcap"))
+    return (out * torch.sigmoid(h @ t[pre + "g"].T)[:, :, None]).reshape(h.shape[0], -1) @ t[pre + "o"].T
 
 
 # ---- feed-forward -----------------------------------------------------------------------------------------------------------

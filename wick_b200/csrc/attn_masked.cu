@@ -109,7 +109,8 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
     const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n_warps = blockDim.x >> 5;
     const bool keys_are_values = flags & FINISH_KEYS_ARE_VALUES, norm_after = flags & FINISH_NORM_AFTER;
     const int Wq = H * d, Wk = G * d, Wv = G * e, W = Wq + Wk + (keys_are_values ? 0 : Wv);
-    float* rec = X.conv_w ? X.conv_rec + (int64_t)X.slots[seq_of_token[t]] * X.record : nullptr;
+    const bool filtered = X.conv_w != nullptr;
+    float* rec = filtered && X.taps > 1 ? X.conv_rec + (int64_t)X.slots[seq_of_token[t]] * X.record : nullptr;
     if ((W & 3) == 0 && (cols & 3) == 0 && (split_stride & 3) == 0 && (X.record & 3) == 0) {
         // four neighbours a load, the loads of four partial sums issued together (a chain of dependent trips to
         // the L2 cache is what a step of few tokens would otherwise wait for); the sums in index order
@@ -129,7 +130,7 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
             if (bias) {
                 v.x += bias[j]; v.y += bias[j + 1]; v.z += bias[j + 2]; v.w += bias[j + 3];
             }
-            if (rec) {                           // (a place's old input moves one place down: read before it is written over)
+            if (filtered) {                      // (a place's old input moves one place down: read before it is written over)
                 float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 3
                 for (int k = 0; k < X.taps; ++k) {
@@ -147,7 +148,7 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
             float v = parts[(int64_t)t * cols + j];
             for (int s = 1; s < splits; ++s) v += parts[s * split_stride + (int64_t)t * cols + j];
             if (bias) v += bias[j];
-            if (rec) {
+            if (filtered) {
                 float y = 0.f;
                 for (int k = 0; k < X.taps; ++k) {
                     const float u = k < X.taps - 1 ? rec[(int64_t)k * W + j] : v;
