@@ -2,7 +2,7 @@
 """Decode and prefill throughput of wick_b200 on one B200, as one JSON line.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--model 8b|14b|32b]
-    python bench.py --design nibotar|tuguvik|fasunex|sunosun|kikopel [--design-size 2k|4k]      (a line of its own, see below)
+    python bench.py --design nibotar|tuguvik|fasunex|sunosun|kikopel|saposun [--design-size 2k|4k]      (a line of its own, see below)
 
 The default run has the layer sizes of Qwen3-8B (36 layers, hidden 4096, 32
 heads over 8 kv heads of 128, intermediate 12288, vocabulary 151936) with random
@@ -47,6 +47,10 @@ cores, since that, not memory, bounds them in a prompt.
 a linear attention whose forget factor says what is written; normed results, PolyNorm feed-forwards, a pair embedding) beside
 the two designs whose layers are the closest: Tuguvik (latent attention) and Sunosun (a linear attention of the same state),
 at equal size, with the same kind of ``parts``.
+``--design saposun`` prints the line of the Saposun design (latent attention with and without latents of its own, retention, and
+an attention with short filters, capped scores and pooled blocks beside its window, each in parallel with routed experts)
+beside the three designs that have the like kernels: Tuguvik (latent attention), Fasunex (a masked attention, a recurrence
+with a short filter, gated routed experts) and Sunosun (a linear attention of the same state), at equal size.
 """
 import argparse
 import json
@@ -280,6 +284,8 @@ def design_step_bytes(eng, z, name, batch, kv_tokens):
         kv_tokens = min(kv_tokens, batch * (z["window"] + z["keep_first"]))
     if name == "kikopel":
         return kikopel_step_bytes(eng, z, batch, kv_tokens)
+    if name == "saposun":
+        return saposun_step_bytes(eng, z, batch, kv_tokens)
     if name == "fasunex":
         return fasunex_step_bytes(eng, z, batch, kv_tokens)
     if name == "sunosun":
@@ -487,6 +493,8 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
 
     def timed(kind, fn, work):
         def run(*a, **kw):
+            if callable(kind) and kind(*a, **kw) is None:            # (part of a call that is timed as a whole)
+                return fn(*a, **kw)
             e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             e0.record(torch.cuda.current_stream())
             r = fn(*a, **kw)
@@ -550,12 +558,41 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
     def norm_gate_work(r, y, parts, *a, **k):
         return 0.0, nbytes(y, r) + (parts.shape[0] * nbytes(y) if parts is not None else 0)
 
-    latent_multi = lambda *a, **k: "attention over latent rows" if k.get("rows_of") else "attention"
+    def attn_pooled_work(r, q, kv, batch, scale, **k):       # (a step's pairs and rows, the blocks' among them)
+        n, H, d = q.shape
+        row = k["n_kv"] * (d + k["v_dim"]) * 2
+        return 2.0 * ctx["pairs_pooled"] * H * (d + k["v_dim"]), nbytes(q, r) + ctx["rows_pooled"] * row
+
+    def retention_work(r, parts, **k):
+        n, H, dk, dv = parts.shape[1], k["heads"], k["key_dim"], k["v_dim"]
+        return 4.0 * n * H * dk * dv, nbytes(parts, r) + 2 * 4 * n * (2 * H * dk + H * dv) + 2 * 4 * k["batch"].n_seqs * H * dk * dv
+
+    def conv_work(r, parts, w, records, batch):
+        return 0.0, nbytes(parts, r) + batch.n_seqs * 2 * 4 * (w.shape[0] - 1) * w.shape[1]
+
+    def qkv_work(r, parts, *a, **k):
+        if name != "saposun":
+            return rows_work(r, parts, *a, **k)
+        n, H, G, d, e = r.shape[0], a[0], a[1], a[2], a[3]
+        rec = n * 2 * 4 * (k["conv"][0].shape[0] - 1) * k["conv"][0].shape[1] if k.get("conv") else 0
+        return 0.0, 4 * parts.shape[0] * n * ((H + G) * d + G * e) + nbytes(r) + 2 * n * G * (d + e) + rec
+
+    def moe_work(blk):
+        f, W = blk.ffn, z["width"]
+        def work(r, x, batch, beside=None):
+            n = x.shape[0]
+            one = 3 * W * f.intermediate
+            return 2.0 * n * f.top * one, nbytes(x, r, beside) + f.experts * (1.0 - (1.0 - f.top / f.experts) ** n) * one * 2
+        return work
+
+    latent_multi = lambda *a, **k: "attention over latent rows" if k.get("rows_of") else (None if name == "saposun" else "attention")
     latent_flex = lambda q, k0, k1, *a, **k: "attention with keys from the latent" if k1[8] else "attention"
     for fname, kind, work in (("attention_multi", latent_multi, attn_multi_work), ("attention_flex", latent_flex, attn_flex_work),
                               ("combine_maps", "attention", rows_work), ("latent_query", "finish", rows_work),
                               ("attention_prompt", "attention", attn_std_work),
-                              ("attention_decode", "attention", attn_std_work), ("qkv_finish", "finish", rows_work),
+                              ("attention_decode", "attention", attn_std_work), ("qkv_finish", "finish", qkv_work),
+                              ("attention_pooled", "attention", attn_pooled_work), ("short_conv", "short filters", conv_work),
+                              ("retention_mix", "recurrence (rotation, scan)", retention_work),
                               ("latent_finish", "finish", finish_work), ("qk_norm_rope_append", "finish", rows_work),
                               ("embed_pairs", "embedding", pairs_work), ("poly_norm", "activation", rows_work),
                               ("hgrn2_mix", "recurrence (forget factors, scan)", hgrn2_work),
@@ -577,6 +614,8 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
         for attr in ("gate_up", "up", "down"):
             if isinstance(getattr(blk.ffn, attr, None), Linear):
                 product("feed-forward", getattr(blk.ffn, attr))
+        if type(blk.ffn).__name__ == "RoutedMoE":
+            blk.ffn.forward = timed("feed-forward RoutedMoE", blk.ffn.forward, moe_work(blk))
         if blk.side is not None:
             product("side input", blk.side.gate)
             product("side input", blk.side.proj)
@@ -600,10 +639,12 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
         return res
 
     out = {}
-    win, keep = {"tuguvik": (z["window"], z["keep_first"]), "kikopel": (z["window"], 0)}.get(name, (None, 0))
+    win, keep = {"tuguvik": (z["window"], z["keep_first"]), "kikopel": (z["window"], 0), "saposun": (z["window"], 0)}.get(name, (None, 0))
     seen = lambda p: p + 1 if win is None else min(p + 1, win + (keep if name == "tuguvik" else 0))   # (an upper bound for kept keys)
     ptoks = random_prompts(torch, z["vocab"], [PREFILL], 3)[0]
     ctx["pairs"], ctx["kv_rows"] = sum(seen(p) for p in range(PREFILL)), PREFILL
+    pooled = lambda p: min(p + 1, z["window"]) + max(0, p + 1 - z["window"]) // SAPOSUN_POOL
+    ctx["pairs_pooled"], ctx["rows_pooled"] = sum(pooled(p) for p in range(PREFILL)), PREFILL + PREFILL // SAPOSUN_POOL
     for i in range(3):
         s = eng.open_seq()
         acc.clear()
@@ -613,6 +654,7 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
     slots = [eng.open_seq() for _ in range(8)]
     eng.step(slots, random_prompts(torch, z["vocab"], [1500] * 8, 4))
     ctx["pairs"] = ctx["kv_rows"] = 8 * seen(1503)
+    ctx["pairs_pooled"] = ctx["rows_pooled"] = 8 * pooled(1503)
     for i in range(4):
         acc.clear()
         eng.step(slots, [[1 + i]] * 8)
@@ -970,6 +1012,81 @@ def kikopel_compare(args) -> int:
     return 0 if all(m["finite"] for m in models.values()) else 1
 
 
+# ---- --design saposun ----------------------------------------------------------
+# Saposun beside the designs that have the like kernels: the latent attention of Tuguvik (the same latent, window, heads), the
+# experts of Fasunex (as many, as large, as many chosen) and its masked attention with as many heads, and a linear attention
+# with as large a state as Sunosun's.  Every fourth layer is of one kind: latent attention, retention, the attention with
+# pooled blocks, latent attention over the first one's rows.
+SAPOSUN_POOL = 16
+
+
+def saposun_sizes(size):
+    return {**TUGUVIK_SIZES[size], **DESIGN_SIZES[size]}
+
+
+def saposun_configs(z):
+    d = z["dim"]
+    latent = dict(heads=z["heads"], dim=d, rot_dim=z["rot_dim"], vdim=d, q_rank=z["q_rank"], kv_rank=z["kv_rank"],
+                  scale=(d + z["rot_dim"]) ** -0.5, mask={"size": z["window"]}, rot={"dims": z["rot_dim"], "base": 10000.0})
+    heads = z["width"] // 128
+    retention = dict(heads=heads, dim=128, vdim=128, decay=[1.0 - 2.0 ** (-5.0 - 4.0 * i / heads) for i in range(heads)],
+                     rot={"dims": 128, "base": 1000000.0})
+    att = dict(heads=z["heads"], kv_heads=z["kv"], dim=d, vdim=d, scale=d ** -0.5, conv=4, softcap=30.0, rot={"dims": d, "base": 50000.0},
+               mask={"size": z["window"], "pool": SAPOSUN_POOL})
+    mlp = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    kinds = (("latent_attention", latent), ("retention", retention), ("attention", att), ("latent_attention", latent))
+    layers = []
+    for i in range(z["layers"]):
+        kind, mixer = kinds[i % 4]
+        layers.append(dict(type=kind, mixer=dict(mixer, kv_from=i - 3) if i % 4 == 3 else mixer, mlp=mlp))
+    return dict(architecture="Saposun", vocab=z["vocab"], width=z["width"], norm={"eps": 1e-5}, residual_mult=0.5, layers=layers)
+
+
+def saposun_step_bytes(eng, z, batch, kv_tokens):
+    """Bytes a decode step of Saposun has to read: the weights (of a layer's experts a batch uses E (1 - (1 - top / E)^batch) on
+    average), the windows' rows and blocks, and the records (read and written back)."""
+    n = eng.model.weight_bytes_per_step()
+    e, top = z["experts"], z["top"]
+    n += z["layers"] * (e * (1.0 - (1.0 - top / e) ** batch) - min(top, e)) * 3 * z["expert_ff"] * z["width"] * 2
+    windows = int(min(kv_tokens, batch * z["window"]))
+    for g in eng.cache.groups:
+        n += 2 * g.store.read_bytes(0, batch) if g.need.kind == "state" else \
+            g.store.read_bytes(int(kv_tokens) - windows if g.need.kind == "paged_blocks" else windows, batch)
+    return n + z["layers"] // 4 * windows * (z["kv_rank"] + z["rot_dim"]) * 2      # (the rows that a second layer reads)
+
+
+def saposun_compare(args) -> int:
+    import torch
+    import wick_b200 as wick
+    pk = peaks()
+    z, zt, zd = saposun_sizes(args.design_size), TUGUVIK_SIZES[args.design_size], DESIGN_SIZES[args.design_size]
+    cfgs = {"saposun": (z, saposun_configs(z), tuguvik_parts), "tuguvik": (zt, tuguvik_configs(zt)["tuguvik"], tuguvik_parts),
+            "fasunex": (zd, fasunex_configs(zd)["fasunex"], fasunex_parts), "sunosun": (zd, sunosun_configs(zd)["sunosun"], fasunex_parts)}
+    if args.design_parts:
+        z, cfg, parts_of = cfgs[args.design_parts]
+        print(json.dumps({args.design_parts: parts_of(torch, wick, pk, z, args.design_parts, cfg)}))
+        return 0
+    steps, warmup = min(args.steps, 64), max(args.warmup, 3)
+    with Clocks() as clk:
+        models = {name: design_model(torch, wick, pk, z, name, cfg, steps, warmup) for name, (z, cfg, _) in cfgs.items()}
+    env = dict(os.environ, WICK_B200_NO_PDL="1")
+    parts, errors = {}, {}
+    for name in cfgs:                                  # (a process each: the timing wrappers replace the module's functions)
+        r = subprocess.run([sys.executable, os.path.abspath(__file__), "--design", "saposun", "--design-size", args.design_size,
+                            "--design-parts", name], env=env, capture_output=True, text=True)
+        for ln in r.stdout.splitlines():
+            if ln.startswith("{"):
+                parts.update(json.loads(ln))
+        if name not in parts:
+            errors[name] = r.stderr[-600:]
+    line = {"metric": f"Saposun beside Tuguvik, Fasunex and Sunosun at equal size ({args.design_size}): prefill and decode tok/s, bf16",
+            "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": warmup, "dtype": "bf16", "sizes": saposun_sizes(args.design_size),
+            "data": "synthetic: seeded random weights, seeded uniform random token ids", "models": models, "parts": parts,
+            "parts_error": errors or None, "clocks": clk.result, "peaks": pk, "fp32_tflops_nominal": FP32_TFLOPS_NOMINAL}
+    print(json.dumps(line))
+    return 0 if all(m["finite"] for m in models.values()) else 1
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -990,8 +1107,9 @@ def main() -> int:
     ap.add_argument("--skip-prefill", action="store_true")
     ap.add_argument("--skip-decode", action="store_true", help="prefill only (for profiling)")
     ap.add_argument("--eager", action="store_true", help="no CUDA graphs (every kernel is a launch of its own)")
-    ap.add_argument("--design", default=None, choices=["nibotar", "tuguvik", "fasunex", "sunosun", "kikopel"],
-                    help="another line: this design beside Qwen3 (fasunex: beside Nibotar; sunosun: beside Fasunex; kikopel: beside Tuguvik and Sunosun) at equal size")
+    ap.add_argument("--design", default=None, choices=["nibotar", "tuguvik", "fasunex", "sunosun", "kikopel", "saposun"],
+                    help="another line: this design beside Qwen3 (fasunex: beside Nibotar; sunosun: beside Fasunex; kikopel: beside Tuguvik and "
+                         "Sunosun; saposun: beside Tuguvik, Fasunex and Sunosun) at equal size")
     ap.add_argument("--design-size", default="2k", choices=sorted(DESIGN_SIZES))
     ap.add_argument("--design-parts", nargs="?", const="both", default=None,
                     help="only the per-kernel times of --design (run by --design itself; tuguvik: of the model named)")
@@ -1006,6 +1124,8 @@ def main() -> int:
         return sunosun_compare(args)
     if args.design == "kikopel":
         return kikopel_compare(args)
+    if args.design == "saposun":
+        return saposun_compare(args)
     if args.design:
         return design_compare(args)
     if args.gpus != 1:
