@@ -567,14 +567,14 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
         n, H, dk, dv = parts.shape[1], k["heads"], k["key_dim"], k["v_dim"]
         return 4.0 * n * H * dk * dv, nbytes(parts, r) + 2 * 4 * n * (2 * H * dk + H * dv) + 2 * 4 * k["batch"].n_seqs * H * dk * dv
 
-    def conv_work(r, parts, w, records, batch):
-        return 0.0, nbytes(parts, r) + batch.n_seqs * 2 * 4 * (w.shape[0] - 1) * w.shape[1]
+    def experts_norm_work(r, x, d, *a, **k):
+        return 0.0, 4 * d.choice.numel() * x.shape[1] + nbytes(d.base, x, r) + (nbytes(x) if k.get("rows") is None else 0)
 
     def qkv_work(r, parts, *a, **k):
         if name != "saposun":
             return rows_work(r, parts, *a, **k)
         n, H, G, d, e = r.shape[0], a[0], a[1], a[2], a[3]
-        rec = n * 2 * 4 * (k["conv"][0].shape[0] - 1) * k["conv"][0].shape[1] if k.get("conv") else 0
+        rec = k["conv"][2].n_seqs * 2 * 4 * (k["conv"][0].shape[0] - 1) * k["conv"][0].shape[1] if k.get("conv") else 0
         return 0.0, 4 * parts.shape[0] * n * ((H + G) * d + G * e) + nbytes(r) + 2 * n * G * (d + e) + rec
 
     def moe_work(blk):
@@ -582,7 +582,7 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
         def work(r, x, batch, beside=None):
             n = x.shape[0]
             one = 3 * W * f.intermediate
-            return 2.0 * n * f.top * one, nbytes(x, r, beside) + f.experts * (1.0 - (1.0 - f.top / f.experts) ** n) * one * 2
+            return 2.0 * n * f.top * one, nbytes(x) + 4 * n * f.top * W + f.experts * (1.0 - (1.0 - f.top / f.experts) ** n) * one * 2
         return work
 
     latent_multi = lambda *a, **k: "attention over latent rows" if k.get("rows_of") else (None if name == "saposun" else "attention")
@@ -591,10 +591,10 @@ def tuguvik_parts(torch, wick, pk, z, name, cfg_json):
                               ("combine_maps", "attention", rows_work), ("latent_query", "finish", rows_work),
                               ("attention_prompt", "attention", attn_std_work),
                               ("attention_decode", "attention", attn_std_work), ("qkv_finish", "finish", qkv_work),
-                              ("attention_pooled", "attention", attn_pooled_work), ("short_conv", "short filters", conv_work),
+                              ("attention_pooled", "attention", attn_pooled_work), 
                               ("retention_mix", "recurrence (rotation, scan)", retention_work),
                               ("latent_finish", "finish", finish_work), ("qk_norm_rope_append", "finish", rows_work),
-                              ("embed_pairs", "embedding", pairs_work), ("poly_norm", "activation", rows_work),
+                              ("moe_experts_norm", "experts' sum and norm", experts_norm_work), ("embed_pairs", "embedding", pairs_work), ("poly_norm", "activation", rows_work),
                               ("hgrn2_mix", "recurrence (forget factors, scan)", hgrn2_work),
                               ("gla_norm_gate", "recurrence's norm", norm_gate_work),
                               ("latent_absorb", "query into the rows' space", absorb_work),

@@ -350,7 +350,8 @@ def test_experts_chosen_by_corrected_scores_weighted_by_the_scores_themselves(dt
         x = h.to(DEV, TORCH[dtype]).contiguous()
         tight(part.forward(x, seq_batch(n)).sum(0), ref, dtype, f"{n} tokens")
         beside = rnd(g, 3, n, width)
-        tight(part.forward(x, seq_batch(n), beside=beside.to(DEV)).sum(0), ref + beside.double().sum(0), dtype, f"{n} tokens beside")
+        got = part.forward(x, seq_batch(n), beside=beside.to(DEV))
+        tight(got.sums()[0], ref + beside.double().sum(0), dtype, f"{n} tokens beside")
 
 
 LATS = [lat(3, 12, 8, 20, 28, 24, 0.3, 1000.0, 17), lat(2, 16, 16, 16, 32, 40, 0.2, 20000.0, 64), lat(5, 7, 6, 9, 11, 13, 0.3, 50.0, 1),
@@ -445,26 +446,61 @@ def test_the_state_remembers_a_token_hundreds_of_positions_back():
             tight(run_mixer(part, h2, "float32", cuts, record_view(part)), ref2, "float32", f"changed, cuts {cuts[:3]}", tol=2e-4)
 
 
-@pytest.mark.parametrize("channels,taps,extra", [(40, 4, 3), (37, 2, 0), (300, 7, 5), (8, 1, 2), (64, 16, 0)])
-def test_the_short_filter_and_its_record(channels, taps, extra):
-    g = torch.Generator().manual_seed(channels)
-    n = 90
-    u = rnd(g, n, channels + extra)
-    a = rnd(g, n, channels + extra)
-    parts, w = torch.stack([u - a, a]).to(DEV), rnd(g, taps, channels)
-    ref = P.causal_filter(u[:, :channels].double(), w.T.double())
+@pytest.mark.parametrize("H,G,d,e,taps,extra,splits", [(3, 1, 8, 4, 4, 3, 2), (2, 2, 7, 5, 2, 0, 1), (4, 2, 32, 16, 7, 4, 3), (1, 1, 4, 4, 1, 2, 1), (2, 1, 16, 16, 16, 0, 2)])
+def test_the_short_filters_and_their_record(H, G, d, e, taps, extra, splits):
+    """The finish kernel on given partial sums: q comes out filtered, k and v lie filtered in the cache, and the record holds the
+    last inputs, oldest first, zeros before the start."""
+    g = torch.Generator().manual_seed(d)
+    n, W = 90, (H + G) * d + G * e
+    u = rnd(g, n, W + extra)
+    a = rnd(g, splits - 1, n, W + extra)
+    parts, w = torch.cat([(u - a.sum(0))[None], a]).to(DEV), rnd(g, taps, W)
+    ref = P.causal_filter(u[:, :W].double(), w.T.double())
     for cuts in ([n], [1] * 9 + [2, 2, 3, 64, 10], [1, 2, 87]):
-        rec = torch.full((3, (taps - 1) * channels), float("nan"), device=DEV)
+        rec = torch.full((3, (taps - 1) * W), float("nan"), device=DEV)
         rec[1].zero_()
+        kv = torch.full((4, G * PAGE * (d + e)), float("nan"), device=DEV)
         outs, at = [], 0
         for c in cuts:
-            outs.append(ops.short_conv(parts[:, at:at + c].contiguous(), w.to(DEV), rec if taps > 1 else None, seq_batch(c, at)))
+            b = seq_batch(c, at)
+            outs.append(ops.qkv_finish(parts[:, at:at + c].contiguous(), H, G, d, e, dtype=torch.float32, kv=kv, page_table=b.page_table,
+                                       seq_of_token=b.seq_of_token, positions=b.positions, conv=(w.to(DEV), rec if taps > 1 else None, b)))
             at += c
-            if taps > 1:                                    # the last inputs, oldest first, zeros before the start
-                want = torch.cat([torch.zeros(taps - 1, channels), u[:at, :channels]])[-(taps - 1):]
-                tight(rec[1].view(taps - 1, channels), want, "float32", f"record after {at}")
-        tight(torch.cat(outs), ref, "float32", f"cuts {cuts[:3]}")
+            if taps > 1:
+                want = torch.cat([torch.zeros(taps - 1, W), u[:at, :W]])[-(taps - 1):]
+                tight(rec[1].view(taps - 1, W), want, "float32", f"record after {at}")
+        tight(torch.cat(outs).view(n, -1), ref[:, :H * d], "float32", f"q, cuts {cuts[:3]}")
+        keys = kv[1:3, :G * PAGE * d].view(2, G, PAGE, d).transpose(1, 2).reshape(2 * PAGE, G * d)[:n]
+        vals = kv[1:3, G * PAGE * d:].view(2, G, PAGE, e).transpose(1, 2).reshape(2 * PAGE, G * e)[:n]
+        tight(torch.cat([keys, vals], 1), ref[:, H * d:], "float32", f"k and v, cuts {cuts[:3]}")
         assert torch.isnan(rec[0]).all() and torch.isnan(rec[2]).all()
+
+
+@pytest.mark.parametrize("width,top,splits,factor,sorted_rows", [(64, 2, 3, 0.4, False), (2048, 4, 1, 1.0, True), (4100, 1, 2, -0.7, True), (12, 33, 1, 0.5, False)])
+def test_experts_sums_join_the_stream_and_its_norm_in_one_kernel(width, top, splits, factor, sorted_rows):
+    g = torch.Generator().manual_seed(width)
+    n, E, eps = 9, top + 2, 1e-4
+    choice = torch.stack([torch.randperm(E, generator=g)[:top] for _ in range(n)]).int()
+    choice[0, 0] = -1                                       # (names no expert)
+    row_of = torch.randperm(3 * n * top, generator=g)[:n * top].view(n, top).int() if sorted_rows else None
+    y, weight = rnd(g, 3 * n * top if sorted_rows else n * top, width), torch.rand(n, top, generator=g)
+    base, x, w = rnd(g, splits, n, width), 3 * rnd(g, n, width), 1 + 0.3 * rnd(g, width)
+    rows = row_of.long() if sorted_rows else torch.arange(n * top).view(n, top)
+    d = (weight * (choice >= 0)).double()[:, :, None] * y.double()[rows]
+    dev = lambda t: None if t is None else t.to(DEV)
+    for b in (base, None):
+        want = x.double() + factor * (d.sum(1) + (0 if b is None else b.double().sum(0)))
+        s = ops.ExpertSum(dev(y), dev(row_of), dev(choice), dev(weight), E, dev(b))
+        assert s.joins_norm()
+        tight(s.sums()[0], (want - x.double()) / factor, "float32", "sums", 1e-5)
+        xd = x.to(DEV)
+        got = ops.moe_experts_norm(xd, s, factor, w.to(DEV), eps, torch.float32, torch.tensor([3, 3, 8, 0], dtype=torch.int32, device=DEV))
+        tight(got, P.norm(want, w.double(), eps)[[3, 3, 8, 0]], "float32", "chosen rows", 3e-6)
+        assert torch.equal(xd.cpu(), x)
+        for dt in DTYPES:
+            xd = x.to(DEV)
+            tight(ops.moe_experts_norm(xd, s, factor, w.to(DEV), eps, TORCH[dt]), P.norm(want, w.double(), eps), dt, "normed", 3e-6 if dt == "float32" else 5e-3)
+            tight(xd, want, "float32", "the stream", 3e-6)
 
 
 ATTS = [att(4, 2, 16, 12, 0.3, 20, 3, 4, 12.0, 700.0, 8), att(2, 1, 8, 8, 0.4, 64, 10, 2, 30.0), att(5, 5, 7, 9, 0.3, 1, 1, 1, 8.0, 50.0, 6),

@@ -47,8 +47,9 @@ constexpr int MAX_V_HEADS = 256;                // value heads that the values' 
 
 // What some attentions do besides.
 //   conv_w  : [taps][W] or null: the row is a causal filter over time of what was projected, channel by channel, the inputs
-//             before this token from the sequence's record ([taps - 1][W], oldest first), which moves on by this token (steps
-//             of one token per sequence only; a longer step runs the filter as a kernel of its own)
+//             before this step from the sequence's record ([taps - 1][W], oldest first), zeros before position 0.  In a step of
+//             one token per sequence (start null) the record moves on by the token; a longer step reads its own earlier rows of
+//             `parts`, from position start[b] on, and a kernel behind this one brings the records up to date
 //   v_norm  : every head's values are divided by their root mean square (v_eps inside the root)
 //   gate_out: [n, gate_heads], the sigmoids of the columns from gate_col on of gate_parts (sums laid out like parts, gate_cols a row)
 //   pool    : (steps of one token per sequence only) the token that completes a block of `block` positions leaves the block's mean key
@@ -59,7 +60,7 @@ struct FinishExtra {
     const float* conv_w;
     float* conv_rec;
     int64_t record;
-    const int* slots;
+    const int *slots, *start;
     int taps, v_norm;
     float v_eps;
     float* gate_out;
@@ -110,7 +111,9 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
     const bool keys_are_values = flags & FINISH_KEYS_ARE_VALUES, norm_after = flags & FINISH_NORM_AFTER;
     const int Wq = H * d, Wk = G * d, Wv = G * e, W = Wq + Wk + (keys_are_values ? 0 : Wv);
     const bool filtered = X.conv_w != nullptr;
+    const int pos = positions[t];
     float* rec = filtered && X.taps > 1 ? X.conv_rec + (int64_t)X.slots[seq_of_token[t]] * X.record : nullptr;
+    const int earlier = filtered && X.start ? pos - X.start[seq_of_token[t]] : 0;    // the step's own rows before this one
     if ((W & 3) == 0 && (cols & 3) == 0 && (split_stride & 3) == 0 && (X.record & 3) == 0) {
         // four neighbours a load, the loads of four partial sums issued together (a chain of dependent trips to
         // the L2 cache is what a step of few tokens would otherwise wait for); the sums in index order
@@ -132,12 +135,37 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
             }
             if (filtered) {                      // (a place's old input moves one place down: read before it is written over)
                 float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 3
-                for (int k = 0; k < X.taps; ++k) {
-                    const float4 u = k < X.taps - 1 ? *reinterpret_cast<const float4*>(rec + (int64_t)k * W + j) : v;
-                    const float4 w = *reinterpret_cast<const float4*>(X.conv_w + (int64_t)k * W + j);
-                    if (k > 0) *reinterpret_cast<float4*>(rec + (int64_t)(k - 1) * W + j) = u;
-                    y.x = fmaf(w.x, u.x, y.x); y.y = fmaf(w.y, u.y, y.y); y.z = fmaf(w.z, u.z, y.z); y.w = fmaf(w.w, u.w, y.w);
+                for (int k0 = 0; k0 < X.taps; k0 += 4) {            // (the loads of four taps go out together)
+                    float4 u[4], w[4];
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const int k = k0 + i, back = X.taps - 1 - k;
+                        u[i] = w[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                        if (back < 0) continue;
+                        w[i] = *reinterpret_cast<const float4*>(X.conv_w + (int64_t)k * W + j);
+                        if (back == 0) u[i] = v;
+                        else if (back > earlier) u[i] = *reinterpret_cast<const float4*>(rec + (int64_t)(k + earlier) * W + j);
+                        else u[i] = *reinterpret_cast<const float4*>(parts + (int64_t)(t - back) * cols + j);
+                    }
+                    if (splits > 1) {
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            const int back = X.taps - 1 - (k0 + i);
+                            if (back <= 0 || back > earlier) continue;
+                            for (int s = 1; s < splits; ++s) {
+                                const float4 d = *reinterpret_cast<const float4*>(parts + s * split_stride + (int64_t)(t - back) * cols + j);
+                                u[i].x += d.x; u[i].y += d.y; u[i].z += d.z; u[i].w += d.w;
+                            }
+                        }
+                    }
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const int k = k0 + i;
+                        if (k >= X.taps) continue;
+                        if (k > 0 && !X.start) *reinterpret_cast<float4*>(rec + (int64_t)(k - 1) * W + j) = u[i];
+                        y.x = fmaf(w[i].x, u[i].x, y.x); y.y = fmaf(w[i].y, u[i].y, y.y);
+                        y.z = fmaf(w[i].z, u[i].z, y.z); y.w = fmaf(w[i].w, u[i].w, y.w);
+                    }
                 }
                 v = y;
             }
@@ -151,8 +179,14 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
             if (filtered) {
                 float y = 0.f;
                 for (int k = 0; k < X.taps; ++k) {
-                    const float u = k < X.taps - 1 ? rec[(int64_t)k * W + j] : v;
-                    if (k > 0) rec[(int64_t)(k - 1) * W + j] = u;
+                    const int back = X.taps - 1 - k;
+                    float u = v;
+                    if (back > earlier) u = rec[(int64_t)(k + earlier) * W + j];
+                    else if (back > 0) {
+                        u = parts[(int64_t)(t - back) * cols + j];
+                        for (int s = 1; s < splits; ++s) u += parts[s * split_stride + (int64_t)(t - back) * cols + j];
+                    }
+                    if (k > 0 && !X.start) rec[(int64_t)(k - 1) * W + j] = u;
                     y = fmaf(X.conv_w[(int64_t)k * W + j], u, y);
                 }
                 v = y;
@@ -177,7 +211,6 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
         }
         __syncthreads();
     }
-    const int pos = positions[t];
     const float lam = v_mode == 2 ? *lambda : 0.f;
     T* page = nullptr;
     if (write_kv) {
@@ -658,7 +691,7 @@ int qkv_finish(const float* parts, int splits, int n, const float* bias, int H, 
                int q_span, const float* k_w, int k_span, float eps, const float* cos_t, const float* sin_t, int rot_dims,
                int pairing, int maps, float* v_keep, int v_mode, const float* lambda, void* q_out, void* kv, const int* page_table,
                int table_width, const int* seq_of_token, const int* positions, int write_kv, int cols, int flags, const FinishExtra<T>& X,
-               cudaStream_t s) {
+               int n_seqs, const int* cu_seqlens, cudaStream_t s) {
     WICK_REQUIRE(H > 0 && G > 0 && H % G == 0 && d > 0 && e > 0, "qkv_finish: bad head counts or sizes");
     WICK_REQUIRE(!(flags & FINISH_KEYS_ARE_VALUES) || (d == e && v_mode == 0), "qkv_finish: keys that are values have the values' size and are not blended");
     WICK_REQUIRE(cols >= H * d + G * d + ((flags & FINISH_KEYS_ARE_VALUES) ? 0 : G * e), "qkv_finish: rows of %d numbers are too short", cols);
@@ -673,7 +706,7 @@ int qkv_finish(const float* parts, int splits, int n, const float* bias, int H, 
     WICK_REQUIRE(v_mode == 0 || v_keep, "qkv_finish: the kept values are missing");
     WICK_REQUIRE(v_mode != 2 || lambda, "qkv_finish: the blend factor is missing");
     WICK_REQUIRE(!X.v_norm || G <= MAX_V_HEADS, "qkv_finish: the values' norm takes up to %d heads", MAX_V_HEADS);
-    WICK_REQUIRE(!X.conv_w || (X.taps >= 1 && X.slots && (X.taps == 1 || X.conv_rec) && !(flags & FINISH_KEYS_ARE_VALUES) &&
+    WICK_REQUIRE(!X.conv_w || (X.taps >= 1 && X.taps <= CONV_MAX_TAPS && (!X.start || (cu_seqlens && n_seqs <= n)) && X.slots && (X.taps == 1 || X.conv_rec) && !(flags & FINISH_KEYS_ARE_VALUES) &&
                                X.record >= (int64_t)(X.taps - 1) * (Wq + Wk + G * e)), "qkv_finish: bad filter");
     WICK_REQUIRE(X.gate_heads == 0 || (X.gate_out && X.gate_parts && X.gate_splits >= 1 && X.gate_col >= 0 && X.gate_col + X.gate_heads <= X.gate_cols),
                  "qkv_finish: bad gate columns");
@@ -690,7 +723,13 @@ int qkv_finish(const float* parts, int splits, int n, const float* bias, int H, 
     WICK_CUDA(launch(qkv_finish_kernel<T>, dim3(n), dim3(256), smem, s, parts, splits, (int64_t)n * cols, bias, H, G,
                      d, e, q_w, q_span, k_w, k_span, eps, cos_t, sin_t, rot_dims, pairing, maps, v_keep, v_mode, lambda, (T*)q_out,
                      (T*)kv, page_table, table_width, seq_of_token, positions, write_kv, cols, flags, X));
-    return check_launch("qkv_finish");
+    if (int rc = check_launch("qkv_finish")) return rc;
+    if (X.conv_w && X.start && X.taps > 1) {
+        WICK_CUDA(launch(short_conv_state_kernel, dim3(n_seqs, ceil_div(Wq + Wk + G * e, 256)), dim3(256), 0, s, parts, splits, (int64_t)n * cols,
+                         cols, 0, Wq + Wk + G * e, X.taps, X.conv_rec, X.record, X.slots, cu_seqlens));
+        return check_launch("short_conv_state");
+    }
+    return 0;
 }
 
 template <typename T>
@@ -740,13 +779,13 @@ typedef __nv_bfloat16 bf16;
                       int rot_dims, int pairing, int maps, float* v_keep, int v_mode, const float* lambda, void* q_out, void* kv, \
                       const int* page_table, int table_width, const int* seq_of_token, const int* positions, int write_kv,       \
                       int cols, int flags, const float* conv_w, float* conv_rec, int64_t record, const int* slots, int taps,     \
-                      int v_norm, float v_eps, float* gate_out, const float* gate_parts, int gate_splits, int gate_cols,         \
+                      const int* start, const int* cu_seqlens, int n_seqs, int v_norm, float v_eps, float* gate_out, const float* gate_parts, int gate_splits, int gate_cols,         \
                       int gate_col, int gate_heads, void* pool, int block, int rows, int64_t pool_page, void* s) {                \
-        const FinishExtra<T> X = {conv_w, conv_rec, record, slots, taps, v_norm, v_eps, gate_out, gate_parts, gate_splits, gate_cols, \
+        const FinishExtra<T> X = {conv_w, conv_rec, record, slots, start, taps, v_norm, v_eps, gate_out, gate_parts, gate_splits, gate_cols, \
                                   gate_col, gate_heads, (T*)pool, block, rows, pool_page};                                       \
         return qkv_finish<T>(parts, splits, n, bias, H, G, d, e, q_w, q_span, k_w, k_span, eps, cos_t, sin_t, rot_dims, pairing,  \
                              maps, v_keep, v_mode, lambda, q_out, kv, page_table, table_width, seq_of_token, positions, write_kv,      \
-                             cols, flags, X, (cudaStream_t)s);                                                                   \
+                             cols, flags, X, n_seqs, cu_seqlens, (cudaStream_t)s);                                                                   \
     }
 WICK_QKV_FINISH(wick_qkv_finish_bf16, bf16)
 WICK_QKV_FINISH(wick_qkv_finish_f32, float)
@@ -760,29 +799,6 @@ WICK_QKV_FINISH(wick_qkv_finish_f32, float)
     }
 WICK_ATTN_MASKED(wick_attn_masked_bf16, bf16)
 WICK_ATTN_MASKED(wick_attn_masked_f32, float)
-
-// parts: float32 [splits, n, cols]; w: float32 [taps, channels]; records: float32 [slots, record], the last taps - 1 inputs, oldest
-// first; out: float32 [n, channels], the filtered first `channels` columns.  The records are brought up to date.
-WICK_API int wick_short_conv(const float* parts, int splits, int n, int cols, int channels, int taps, const float* w, float* records,
-                             int64_t record, const int* slots, int n_seqs, const int* cu_seqlens, const int* start,
-                             const int* seq_of_token, const int* positions, float* out, void* stream) {
-    cudaStream_t s = (cudaStream_t)stream;
-    WICK_REQUIRE(splits >= 1 && channels > 0 && channels <= cols, "short_conv: bad sizes");
-    WICK_REQUIRE(taps >= 1 && taps <= CONV_MAX_TAPS, "short_conv: %d taps (1 .. %d are built)", taps, CONV_MAX_TAPS);
-    WICK_REQUIRE(taps == 1 || (records && record >= (int64_t)(taps - 1) * channels), "short_conv: records of another size");
-    if (n == 0 || n_seqs == 0) return 0;
-    const int64_t stride = (int64_t)n * cols;
-    auto kernel = splits == 1 ? short_conv_kernel<true, false> : short_conv_kernel<false, false>;
-    WICK_CUDA(launch(kernel, dim3(ceil_div(n, CONV_TOKENS), ceil_div(channels, 256)), dim3(256), 0, s, parts, splits, stride, cols, 0, channels,
-                     taps, w, 1, channels, (const float*)nullptr, (const float*)records, record, slots, seq_of_token, positions, start, out, n));
-    if (check_launch("short_conv")) return 1;
-    if (taps > 1) {
-        WICK_CUDA(launch(short_conv_state_kernel, dim3(n_seqs, ceil_div(channels, 256)), dim3(256), 0, s, parts, splits, stride, cols, 0,
-                         channels, taps, records, record, slots, cu_seqlens));
-        if (check_launch("short_conv_state")) return 1;
-    }
-    return 0;
-}
 
 #define WICK_POOL_BLOCKS(NAME, T)                                                                                             \
     WICK_API int NAME(const void* kv, void* store, void* flat, const int* page_table, int table_width, const int* start,        \

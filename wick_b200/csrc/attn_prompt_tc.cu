@@ -167,6 +167,20 @@ __device__ __forceinline__ float2 add2(float2 a, float2 b) {
     return d;
 }
 
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    uint64_t ra, rb, rd;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(ra) : "f"(a.x), "f"(a.y));
+    asm("mov.b64 %0, {%1, %2};" : "=l"(rb) : "f"(b.x), "f"(b.y));
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(rd) : "l"(ra), "l"(rb));
+    float2 d;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(d.x), "=f"(d.y) : "l"(rd));
+    return d;
+}
+// tanh(z) = z (c0 + c1 z^2 + c2 z^4 + c3 z^6 + c4 z^8) for |z| <= 0.75, off by at most 4.2e-7 (the interpolant of tanh(z) / z, as a
+// function of z^2, at the Chebyshev points of the interval, fitted by least squares).
+constexpr float TANH_SMALL = 0.75f, TANH_C0 = 0.99999945f, TANH_C1 = -0.33328349f, TANH_C2 = 0.13259838f, TANH_C3 = -0.050080256f,
+                TANH_C4 = 0.012950745f;
+
 // Descriptors.  A k-major operand (Q, K): rows of 128 bytes, eight-row groups 1024
 // bytes apart, the leading offset unused (1).  The MN-major operand (V): rows are
 // keys, a row holds 64 consecutive dims in 128 bytes, eight rows make a 1024-byte
@@ -347,7 +361,8 @@ attn_prompt_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
         const int vis = first_visible_key(limit, mask, mask_size);  // first visible key position
         const bool capped = EXTRA && X.cap > 0.f;
         const float sl2 = capped ? 1.0f : scale * 1.4426950408889634f;   // (a capped score comes in units of log2 e)
-        const float cap2 = EXTRA ? X.cap * 1.4426950408889634f : 0.f, two_s = capped ? 2.0f * scale * 1.4426950408889634f / X.cap : 0.f;
+        const float cap2 = EXTRA ? X.cap * 1.4426950408889634f : 0.f, z_of_s = capped ? scale / X.cap : 0.f,
+                    two_s = 2.0f * 1.4426950408889634f * z_of_s;
         const int n_seen = EXTRA ? blocks_seen(limit, mask_size, X.block) : 0;
         const float sink2 = sink ? sink[head] * 1.4426950408889634f : -INFINITY;   // a score without a value
         const uint32_t lane_base = tmem + ((uint32_t)(quad * 32) << 16);
@@ -371,9 +386,30 @@ attn_prompt_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
             tc_ld32_nowait(s_addr + c_lo, reinterpret_cast<uint32_t*>(s));
             tc_ld32_nowait(s_addr + c_lo + 32, reinterpret_cast<uint32_t*>(s + 32));
             tc_ld_wait();
-            if (capped) {                                           // cap tanh(s / cap) = cap (1 - 2 / (1 + exp(2 s / cap)))
+            if (capped) {
+                // cap tanh(z), z = s / cap: by a polynomial where all of the warp's |z| are small (two products and sums an
+                // instruction), else as cap (1 - 2 / (1 + exp(2 z))), whose two special functions a score would bound the block.
+                float big = 0.f;
 #pragma unroll
-                for (int i = 0; i < HALF_K; ++i) s[i] = fmaf(-2.0f * cap2, rcp(1.0f + ex2(s[i] * two_s)), cap2);
+                for (int i = 0; i < HALF_K; i += 2) big = max3(big, fabsf(s[i]), fabsf(s[i + 1]));
+                if (__all_sync(0xffffffffu, big * z_of_s <= TANH_SMALL)) {
+                    const float2 zs = make_float2(z_of_s, z_of_s), c2 = make_float2(cap2, cap2);
+#pragma unroll
+                    for (int i = 0; i < HALF_K; i += 2) {
+                        const float2 z = mul2(make_float2(s[i], s[i + 1]), zs), q = mul2(z, z);
+                        float2 p = make_float2(TANH_C4, TANH_C4);
+                        p = fma2(p, q, make_float2(TANH_C3, TANH_C3));
+                        p = fma2(p, q, make_float2(TANH_C2, TANH_C2));
+                        p = fma2(p, q, make_float2(TANH_C1, TANH_C1));
+                        p = fma2(p, q, make_float2(TANH_C0, TANH_C0));
+                        const float2 r2 = mul2(mul2(p, z), c2);
+                        s[i] = r2.x;
+                        s[i + 1] = r2.y;
+                    }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < HALF_K; ++i) s[i] = fmaf(-2.0f * cap2, rcp(1.0f + ex2(s[i] * two_s)), cap2);
+                }
             }
             if (key0 + HALF_K - 1 > last || key0 < first_key) {
 #pragma unroll

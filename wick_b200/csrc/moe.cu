@@ -516,6 +516,107 @@ __global__ void moe_combine_weighted_kernel(const float* __restrict__ y, const i
     }
 }
 
+// The experts' results straight into the residual stream and through the norm that reads it next: with d = sum over c of
+// weight[t][c] * y[row(t, c)] (as above) + the partial sums of `base`, x[t] <- x[t] + factor d, and
+// out = x / sqrt(mean(x^2) + eps) * w in the output type.  With `rows` only those rows go out and x stays as it is.  A thread
+// keeps VPT groups of four of the row; everything it adds up is on its way before the first sum.
+constexpr int EXPERTS_TOP = 64;                // choices a token can have in this form
+template <typename TOut, int VPT>
+__global__ void __launch_bounds__(512)
+moe_experts_norm_kernel(const float* __restrict__ y, const int* __restrict__ row_of, const int* __restrict__ choice,
+                        const float* __restrict__ weight, int n_experts, int top, const float* __restrict__ base, int base_splits,
+                        int64_t base_stride, float* __restrict__ x, float factor, const float* __restrict__ w, float eps,
+                        const int* __restrict__ rows, TOut* __restrict__ out, int width) {
+    __shared__ int64_t at[EXPERTS_TOP];
+    __shared__ float wt[EXPERTS_TOP], red[32];
+    pdl_trigger();
+    pdl_wait();
+    y = fresh(y);
+    row_of = fresh(row_of);
+    choice = fresh(choice);
+    weight = fresh(weight);
+    base = fresh(base);
+    x = fresh(x);
+    const int i = blockIdx.x, t = rows ? rows[i] : i, tid = threadIdx.x;
+    if (tid < top) {
+        const int64_t p = (int64_t)t * top + tid;
+        const int ex = choice[p];
+        const int64_t row = row_of ? (int64_t)row_of[p] : p;
+        const bool in = ex >= 0 && ex < n_experts && row >= 0;
+        at[tid] = in ? row * width : -1;
+        wt[tid] = in ? weight[p] : 0.f;
+    }
+    float4 xv[VPT], d[VPT], b[VPT];
+    float* xr = x + (int64_t)t * width;
+#pragma unroll
+    for (int u = 0; u < VPT; ++u) {
+        const int j = (u * (int)blockDim.x + tid) * 4;
+        d[u] = b[u] = xv[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < width) xv[u] = ld4(xr + j);
+    }
+    for (int s = 0; s < base_splits; ++s) {
+#pragma unroll
+        for (int u = 0; u < VPT; ++u) {
+            const int j = (u * (int)blockDim.x + tid) * 4;
+            if (j >= width) continue;
+            const float4 v = ld4(base + s * base_stride + (int64_t)t * width + j);
+            b[u].x += v.x; b[u].y += v.y; b[u].z += v.z; b[u].w += v.w;
+        }
+    }
+    __syncthreads();
+#pragma unroll 2
+    for (int c = 0; c < top; ++c) {
+        if (at[c] < 0) continue;
+        const float f = wt[c];
+#pragma unroll
+        for (int u = 0; u < VPT; ++u) {
+            const int j = (u * (int)blockDim.x + tid) * 4;
+            if (j >= width) continue;
+            const float4 v = ld4(y + at[c] + j);
+            d[u].x = fmaf(f, v.x, d[u].x); d[u].y = fmaf(f, v.y, d[u].y); d[u].z = fmaf(f, v.z, d[u].z); d[u].w = fmaf(f, v.w, d[u].w);
+        }
+    }
+    float ss[1] = {0.f};
+#pragma unroll
+    for (int u = 0; u < VPT; ++u) {
+        const int j = (u * (int)blockDim.x + tid) * 4;
+        if (j >= width) continue;
+        float4& v = xv[u];
+        v.x += factor * (d[u].x + b[u].x); v.y += factor * (d[u].y + b[u].y);
+        v.z += factor * (d[u].z + b[u].z); v.w += factor * (d[u].w + b[u].w);
+        if (!rows) st4(xr + j, v.x, v.y, v.z, v.w);
+        ss[0] = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss[0]))));
+    }
+    block_sums(ss, red);
+    const float g = 1.0f / sqrtf(ss[0] / (float)width + eps);
+#pragma unroll
+    for (int u = 0; u < VPT; ++u) {
+        const int j = (u * (int)blockDim.x + tid) * 4;
+        if (j >= width) continue;
+        const float4 k = ld4(w + j), v = xv[u];
+        st4(out + (int64_t)i * width + j, (v.x * g) * k.x, (v.y * g) * k.y, (v.z * g) * k.z, (v.w * g) * k.w);
+    }
+}
+
+template <typename TOut>
+int moe_experts_norm(const float* y, const int* row_of, const int* choice, const float* weight, int n_experts, int top, const float* base,
+                     int base_splits, float* x, float factor, const float* w, float eps, const int* rows, void* out, int n, int n_out,
+                     int width, cudaStream_t s) {
+    WICK_REQUIRE(n_experts > 0 && top > 0 && top <= EXPERTS_TOP, "moe_experts_norm: %d choices (up to %d are built)", top, EXPERTS_TOP);
+    WICK_REQUIRE(width > 0 && width % 4 == 0 && width <= 4 * 512 * 8, "moe_experts_norm: rows of %d numbers", width);
+    WICK_REQUIRE((((uintptr_t)y | (uintptr_t)base | (uintptr_t)x | (uintptr_t)w) & 15) == 0 && ((uintptr_t)out & 7) == 0,
+                 "moe_experts_norm: rows must start at multiples of 16 bytes");
+    if (n_out == 0) return 0;
+    const int groups = width / 4, vpt = groups <= 512 ? 1 : (groups <= 1024 ? 2 : (groups <= 2048 ? 4 : 8));
+    int threads = (ceil_div(groups, vpt) + 31) / 32 * 32;
+    if (threads < (top + 31) / 32 * 32) threads = (top + 31) / 32 * 32;
+    auto kernel = vpt == 1 ? moe_experts_norm_kernel<TOut, 1> : (vpt == 2 ? moe_experts_norm_kernel<TOut, 2>
+                                                                         : (vpt == 4 ? moe_experts_norm_kernel<TOut, 4> : moe_experts_norm_kernel<TOut, 8>));
+    WICK_CUDA(launch(kernel, dim3(n_out), dim3(threads), 0, s, y, row_of, choice, weight, n_experts, top, base, base ? base_splits : 0,
+                     (int64_t)n * width, x, factor, w, eps, rows, (TOut*)out, width));
+    return check_launch("moe_experts_norm");
+}
+
 template <typename T>
 int moe_up(const void* x, const int* tokens, const int* table, int top, int n_experts, const void* gate_up, void* hidden, int n,
            int width, int ff, int gated, cudaStream_t s) {
@@ -686,3 +787,15 @@ WICK_API int wick_moe_expert_down_f32(const void* hidden, const int* tokens, con
     }
 WICK_MOE_COMBINE_WEIGHTED(wick_moe_combine_weighted_bf16, bf16)
 WICK_MOE_COMBINE_WEIGHTED(wick_moe_combine_weighted_f32, float)
+
+// y, row_of, choice, weight: as for wick_moe_combine_weighted; base: float32 [base_splits, n, width] or null; x: float32 [n, width], the
+// residual stream; w: float32 [width]; rows: int32 [n_out] or null (n_out = n); out: [n_out, width].
+#define WICK_MOE_EXPERTS_NORM(NAME, T)                                                                                          \
+    WICK_API int NAME(const float* y, const int* row_of, const int* choice, const float* weight, int n_experts, int top,         \
+                      const float* base, int base_splits, float* x, float factor, const float* w, float eps, const int* rows,    \
+                      void* out, int n, int n_out, int width, void* s) {                                                         \
+        return moe_experts_norm<T>(y, row_of, choice, weight, n_experts, top, base, base_splits, x, factor, w, eps, rows, out, n, n_out, \
+                                   width, (cudaStream_t)s);                                                                      \
+    }
+WICK_MOE_EXPERTS_NORM(wick_moe_experts_norm_bf16, __nv_bfloat16)
+WICK_MOE_EXPERTS_NORM(wick_moe_experts_norm_f32, float)

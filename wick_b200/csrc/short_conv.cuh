@@ -18,13 +18,13 @@ __device__ __forceinline__ float sum_parts(const float* __restrict__ parts, int 
 
 constexpr int CONV_TOKENS = 4;              // tokens a thread of the convolution takes (their loads are in flight together)
 
-// out[t][c] = bias_c + sum over k of w(c, k) u_(p - (taps - 1) + k) (then silu with SILU), u the partial sums' columns from
-// first_col on, w(c, k) = w[c w_channel + k w_tap].  grid (ceil(tokens / CONV_TOKENS), ceil(channels / 256)).  ONE: the
+// out[t][c] = silu(bias_c + sum over k of w[c][k] u_(p - (taps - 1) + k)), u the partial sums' columns from first_col on.
+// grid (ceil(tokens / CONV_TOKENS), ceil(channels / 256)).  ONE: the
 // projection came as a single set of sums (its loads need no loop and go out together).
-template <bool ONE, bool SILU>
+template <bool ONE>
 __global__ void __launch_bounds__(256)
 short_conv_kernel(const float* __restrict__ parts, int splits, int64_t split_stride, int cols, int first_col, int channels, int taps,
-                const float* __restrict__ w, int w_channel, int w_tap, const float* __restrict__ bias, const float* __restrict__ state, int64_t record,
+                const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ state, int64_t record,
                 const int* __restrict__ slots, const int* __restrict__ seq_of_token, const int* __restrict__ positions,
                 const int* __restrict__ start, float* __restrict__ out, int n) {
     pdl_trigger();
@@ -47,7 +47,7 @@ short_conv_kernel(const float* __restrict__ parts, int splits, int64_t split_str
     }
 #pragma unroll 4
     for (int k = 0; k < taps; ++k) {
-        const float wk = w[(int64_t)c * w_channel + (int64_t)k * w_tap];
+        const float wk = w[(int64_t)c * taps + k];
         float u[CONV_TOKENS];
 #pragma unroll
         for (int j = 0; j < CONV_TOKENS; ++j) {
@@ -63,7 +63,7 @@ short_conv_kernel(const float* __restrict__ parts, int splits, int64_t split_str
 #pragma unroll
     for (int j = 0; j < CONV_TOKENS; ++j) {
         const int t = blockIdx.x * CONV_TOKENS + j;
-        if (t < n) out[(int64_t)t * channels + c] = SILU ? silu_f(acc[j]) : acc[j];
+        if (t < n) out[(int64_t)t * channels + c] = silu_f(acc[j]);
     }
 }
 

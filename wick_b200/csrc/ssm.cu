@@ -429,11 +429,11 @@ WICK_API int wick_ssm_mix(const float* parts, int splits, int n, int cols, int H
     const int64_t stride = (int64_t)n * cols;
     const dim3 conv_grid(ceil_div(n, CONV_TOKENS), ceil_div(channels, 256));
     if (splits == 1) {
-        WICK_CUDA(launch(short_conv_kernel<true, true>, conv_grid, dim3(256), 0, s, parts, splits, stride, cols, inner, channels, taps, conv_w,
-                         taps, 1, conv_b, (const float*)state, record, slots, seq_of_token, positions, start, xbc, n));
+        WICK_CUDA(launch(short_conv_kernel<true>, conv_grid, dim3(256), 0, s, parts, splits, stride, cols, inner, channels, taps, conv_w,
+                         conv_b, (const float*)state, record, slots, seq_of_token, positions, start, xbc, n));
     } else {
-        WICK_CUDA(launch(short_conv_kernel<false, true>, conv_grid, dim3(256), 0, s, parts, splits, stride, cols, inner, channels, taps, conv_w,
-                         taps, 1, conv_b, (const float*)state, record, slots, seq_of_token, positions, start, xbc, n));
+        WICK_CUDA(launch(short_conv_kernel<false>, conv_grid, dim3(256), 0, s, parts, splits, stride, cols, inner, channels, taps, conv_w,
+                         conv_b, (const float*)state, record, slots, seq_of_token, positions, start, xbc, n));
     }
     if (check_launch("ssm_conv")) return 1;
     if (taps > 1) {

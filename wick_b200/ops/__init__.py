@@ -622,27 +622,6 @@ def pool_blocks(kv: torch.Tensor, store: torch.Tensor, batch, *, n_kv: int, d: i
     return (out, tiles) if flat else None
 
 
-def short_conv(parts: torch.Tensor, w: torch.Tensor, records: Optional[torch.Tensor], batch) -> torch.Tensor:
-    """A causal filter over time, channel by channel, of the first columns of the float32 partial sums ``parts`` [splits, n, cols]:
-    y_t = sum_k w[k] u_(t - taps + 1 + k), zeros before a sequence's start.  ``w``: float32 [taps, channels].  ``records``: float32
-    [slots, (taps - 1) * channels], the inputs of earlier steps, oldest first; brought up to date.  Returns float32 [n, channels]."""
-    _cuda("parts", parts, torch.float32)
-    _cuda("w", w, torch.float32)
-    taps, channels = w.shape
-    _need(parts.dim() == 3 and parts.shape[2] >= channels, f"parts must be [splits, n, {channels} or more], is {tuple(parts.shape)}")
-    splits, n, cols = parts.shape
-    _need(n == batch.n_tokens, f"{n} rows, the batch has {batch.n_tokens} tokens")
-    record = (taps - 1) * channels
-    if record:
-        _cuda("records", records, torch.float32)
-        _need(records.dim() == 2 and records.shape[1] == record, f"records must be [slots, {record}], are {tuple(records.shape)}")
-    out = torch.empty((n, channels), dtype=torch.float32, device=parts.device)
-    _layer().call("wick_short_conv", "piiiiipplpippppp" + "p", _p(parts), splits, n, cols, channels, taps, _p(w), _p(records) if record else None,
-                  record, _p(batch.slots), batch.n_seqs, _p(batch.cu_seqlens), _p(batch.start), _p(batch.seq_of_token), _p(batch.positions),
-                  _p(out), _stream(), kernels=2 if taps > 1 else 1)
-    return out
-
-
 def stream_update(x: torch.Tensor, delta: Optional[torch.Tensor], *, scale: Optional[torch.Tensor] = None,
                   rms: Optional[Tuple[torch.Tensor, float]] = None, norm: Optional[tuple] = None,
                   out_dtype: Optional[torch.dtype] = None, rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
@@ -998,9 +977,11 @@ def qkv_finish(parts: torch.Tensor, n_heads: int, n_kv: int, d: int, e: int, *, 
     ``keys_are_values``: the rows hold no values; a head's value is its key as projected, before norm
     and rotation.  Columns behind q, k and v (an output gate's) are left alone.
     ``v_eps``: every head's values are divided by their root mean square.  ``gate`` = (float32 partial sums [splits, n, cols], first
-    column, float32 [n, heads] to write): the sigmoids of the columns' sums.  For steps of one token per sequence only:
-    ``conv`` = (w, records, slots), the filter of :func:`short_conv` over q, k and v before everything else; ``blocks`` = (store, P):
-    the token that completes a block of P positions leaves the block's means (see :func:`pool_blocks`)."""
+    column, float32 [n, heads] to write): the sigmoids of the columns' sums.
+    ``conv`` = (w, records, batch): before everything else every channel of q, k and v passes a causal filter over time,
+    y_t = sum_k w[k] u_(t - taps + 1 + k), zeros before a sequence's start; w float32 [taps, W], records float32 [slots,
+    (taps - 1) W], the inputs of earlier steps, oldest first, brought up to date.  ``blocks`` = (store, P), for steps of one token per
+    sequence only: the token that completes a block of P positions leaves the block's means (see :func:`pool_blocks`)."""
     _cuda("parts", parts, torch.float32)
     W = (n_heads + n_kv) * d + (0 if keys_are_values else n_kv * e)
     _need(parts.dim() == 3 and parts.shape[2] >= W, f"parts must be [splits, n, {W} or more], is {tuple(parts.shape)}")
@@ -1029,10 +1010,13 @@ def qkv_finish(parts: torch.Tensor, n_heads: int, n_kv: int, d: int, e: int, *, 
     q_out = torch.empty((n, n_heads, d), dtype=dtype, device=parts.device)
     _need(maps >= 1 and d % maps == 0, f"a head of {d} numbers is not {maps} vectors")
     flags = (1 if keys_are_values else 0) | (2 if norm_after_rotation else 0)
-    conv_w = conv_rec = slots = None
-    taps = record = 0
+    conv_w = conv_rec = slots = start = cu = None
+    taps = record = n_seqs = 0
     if conv is not None:
-        conv_w, conv_rec, slots = conv
+        conv_w, conv_rec, b = conv
+        slots, n_seqs = b.slots, b.n_seqs
+        if not b.is_decode:
+            start, cu = b.start, b.cu_seqlens
         _cuda("conv's w", conv_w, torch.float32)
         taps = conv_w.shape[0]
         record = (taps - 1) * W
@@ -1040,7 +1024,7 @@ def qkv_finish(parts: torch.Tensor, n_heads: int, n_kv: int, d: int, e: int, *, 
         if record:
             _cuda("conv's records", conv_rec, torch.float32)
             _need(conv_rec.dim() == 2 and conv_rec.shape[1] == record, f"records must be [slots, {record}], are {tuple(conv_rec.shape)}")
-        _cuda("slots", slots, torch.int32, (n,))
+        _need(n == b.n_tokens, f"{n} rows, the batch has {b.n_tokens} tokens")
     gp = g_out = None
     g_splits = g_cols = g_col = g_heads = 0
     if gate is not None:
@@ -1054,13 +1038,13 @@ def qkv_finish(parts: torch.Tensor, n_heads: int, n_kv: int, d: int, e: int, *, 
     if blocks is not None:
         pool, block = blocks
         pool_rows, pool_page = _block_pages("blocks", pool, dtype, n_kv, d, e, block)
-    _layer().call(f"wick_qkv_finish_{_dt(q_out)}", "piipiiiipipifppiiipippppippiii" + "pplpiifppiiiipiil" + "p", _p(parts), parts.shape[0], n, _p(bias),
+    _layer().call(f"wick_qkv_finish_{_dt(q_out)}", "piipiiiipipifppiiipippppippiii" + "pplpippiifppiiiipiil" + "p", _p(parts), parts.shape[0], n, _p(bias),
                   n_heads, n_kv, d, e, _p(q_weight), int(q_span or 0), _p(k_weight), int(k_span or 0), float(eps), _p(cos), _p(sin),
                   rot_dims if cos is not None else 0, PAIRINGS[pairing], int(maps), _p(v_keep), v_mode, _p(blend), _p(q_out),
                   _p(kv) if write_kv else None, _p(page_table), page_table.shape[-1], _p(seq_of_token), _p(positions),
-                  1 if write_kv else 0, int(cols), flags, _p(conv_w), _p(conv_rec) if record else None, record, _p(slots), taps,
+                  1 if write_kv else 0, int(cols), flags, _p(conv_w), _p(conv_rec) if record else None, record, _p(slots), taps, _p(start), _p(cu), n_seqs,
                   1 if v_eps is not None else 0, float(v_eps or 0.0), _p(g_out), _p(gp), g_splits, g_cols, int(g_col), g_heads,
-                  _p(pool), int(block), pool_rows, pool_page, _stream())
+                  _p(pool), int(block), pool_rows, pool_page, _stream(), kernels=2 if start is not None and record else 1)
     return q_out
 
 
@@ -1394,6 +1378,50 @@ def moe_combine_weighted(y: torch.Tensor, row_of: Optional[torch.Tensor], choice
     gate_ptr = _p(base_gate) + 4 * int(base_gate_col) if base_gate is not None else _p(base_gate)
     _layer().call(f"wick_moe_combine_weighted_{dt}", "pppppiipiipipiip", _p(y), _p(row_of), _p(choice), _p(weight), _p(x), int(n_experts),
                   top, _p(out), n, width, _p(base), bs, gate_ptr, gs, gate_ld, _stream())
+    return out
+
+
+class ExpertSum:
+    """What :func:`moe_combine_weighted` adds up (experts' results, their weights, a term beside them), not added up yet: whoever
+    reads the residual stream next may do it in the same kernel (:func:`moe_experts_norm`)."""
+
+    def __init__(self, y: torch.Tensor, row_of: Optional[torch.Tensor], choice: torch.Tensor, weight: torch.Tensor, n_experts: int,
+                 base: Optional[torch.Tensor] = None):
+        self.y, self.row_of, self.choice, self.weight, self.n_experts, self.base = y, row_of, choice, weight, n_experts, base
+
+    def sums(self) -> torch.Tensor:
+        """float32 [1, n, width]."""
+        return moe_combine_weighted(self.y, self.row_of, self.choice, self.weight, None, self.n_experts, self.base).unsqueeze(0)
+
+    def joins_norm(self) -> bool:
+        """Whether :func:`moe_experts_norm` takes these sizes."""
+        return self.y.shape[1] % 4 == 0 and self.y.shape[1] <= 16384 and self.choice.shape[1] <= 64
+
+
+def moe_experts_norm(x: torch.Tensor, d: ExpertSum, factor: float, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
+                     rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x <- x + ``factor`` * (the sum that ``d`` stands for) in float32 and in place, then x / sqrt(mean(x^2) + eps) * ``weight`` in
+    ``out_dtype``.  ``rows`` (int32 indices): only those rows go out, and ``x`` stays as it was."""
+    _cuda("x", x, torch.float32)
+    n, width = x.shape
+    _cuda("weight", weight, torch.float32, (width,))
+    _cuda("y", d.y, torch.float32)
+    top = d.choice.shape[1]
+    _cuda("choice", d.choice, torch.int32, (n, top))
+    _cuda("expert weights", d.weight, torch.float32, (n, top))
+    if d.row_of is not None:
+        _cuda("row_of", d.row_of, torch.int32, (n, top))
+    _need(d.y.shape[1] == width and (d.row_of is not None or d.y.shape[0] == n * top), "the experts' rows have the stream's width")
+    if d.base is not None:
+        _cuda("base", d.base, torch.float32)
+        _need(d.base.dim() == 3 and tuple(d.base.shape[1:]) == (n, width), f"base must be [splits, {n}, {width}]")
+    if rows is not None:
+        _cuda("rows", rows, torch.int32)
+    n_out = n if rows is None else rows.numel()
+    out = torch.empty((n_out, width), dtype=out_dtype, device=x.device)
+    _layer().call(f"wick_moe_experts_norm_{_dt(out)}", "ppppiipipfpfppiiip", _p(d.y), _p(d.row_of), _p(d.choice), _p(d.weight), int(d.n_experts),
+                  top, _p(d.base), 0 if d.base is None else d.base.shape[0], _p(x), float(factor), _p(weight), float(eps), _p(rows), _p(out), n,
+                  n_out, width, _stream())
     return out
 
 

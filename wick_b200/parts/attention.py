@@ -362,24 +362,18 @@ class Attention(Mixer):
         cos, sin = rot.tables(batch) if rot else (None, None)
         kv, blocks, records = self._views(cache)
         cols = self.q_dim + self.k_dim + self.v_all       # (the gate's columns follow)
-        sums, conv = parts, None
-        if self.taps:
-            if not write_cache:
-                raise RuntimeError("filtered projections keep a record of their own; this mixer cannot read another entry's")
-            if batch.is_decode:
-                conv = (self.filters, records, batch.slots)                   # (the finish kernel filters the token itself)
-            else:
-                sums = ops.short_conv(parts, self.filters, records, batch).unsqueeze(0)
+        if self.taps and not write_cache:
+            raise RuntimeError("filtered projections keep a record of their own; this mixer cannot read another entry's")
         gate = torch.empty((n, self.heads), dtype=torch.float32, device=x.device) if self.gate == "head" else None
         pooled = batch.is_decode and blocks is not None and write_cache
         q = ops.qkv_finish(
-            sums, self.heads, self.kv_heads, self.head_dim, self.v_dim, dtype=self.ctx.dtype, bias=self.qkv_bias,
+            parts, self.heads, self.kv_heads, self.head_dim, self.v_dim, dtype=self.ctx.dtype, bias=self.qkv_bias,
             q_weight=self.q_weight, k_weight=self.k_weight, eps=self.eps,
             cos=cos, sin=sin, rot_dims=rot.dims if rot else 0,
             pairing=rot.pairing if rot else "neighbours", v_keep=v_keep, v_mode=v_mode, blend=self.blend_factor,
             kv=kv, page_table=batch.page_table, seq_of_token=batch.seq_of_token, positions=batch.positions,
             write_kv=write_cache, q_span=q_span, k_span=k_span, norm_after_rotation=self.norm_after_rotation,
-            keys_are_values=self.keys_are_values, conv=conv, v_eps=self.eps if self.value_norm else None,
+            keys_are_values=self.keys_are_values, conv=(self.filters, records, batch) if self.taps else None, v_eps=self.eps if self.value_norm else None,
             gate=(parts, cols, gate) if gate is not None else None, blocks=(blocks, self.pool) if pooled else None)
         if self.pooled_kernel:
             att = ops.attention_pooled(q, kv, batch, self.scale, n_kv=self.kv_heads, v_dim=self.v_dim, window=self.mask_size, store=blocks,

@@ -167,7 +167,7 @@ class Norm(Part):
         by the weight first.  A norm without a kernel for these resolves the sum
         into ``x`` with the stream kernel and normalises then."""
         from .. import ops
-        ops.stream_update(x, delta, scale=scale, rms=rms)
+        ops.stream_update(x, delta.sums() if isinstance(delta, ops.ExpertSum) else delta, scale=scale, rms=rms)
         return self.forward(x, out_dtype, rows)
 
     def scaled_add_forward(self, x: torch.Tensor, delta: Optional[torch.Tensor], alpha: float,
@@ -224,7 +224,8 @@ class FeedForward(Part):
         """x: [tokens, width], compute dtype.  Returns float32 [splits, tokens, width].
 
         A feed-forward whose class sets ``JOINS_BESIDE = True`` can also be given ``beside=`` (float32 [splits, tokens,
-        width], what another sublayer made of the same input): its last kernel then adds that to its result."""
+        width], what another sublayer made of the same input): its last kernel then adds that to its result, and it may
+        return an :class:`~wick_b200.ops.ExpertSum` instead, a sum left to whoever reads the stream next."""
         raise NotImplementedError
 
 
@@ -234,7 +235,8 @@ class Hidden:
     (kept apart so that the next norm's kernel can do the addition).  ``scale``
     (float32 [width]) is a factor, element by element, of the pending sum; ``rms``
     (weight, eps) says that the pending sum is divided by its root mean square and
-    multiplied by the weight before it is added; both are None for a plain sum.  ``act``
+    multiplied by the weight before it is added; both are None for a plain sum.  ``pending`` may be
+    an ``ops.ExpertSum`` (a sum over experts that nobody has added up yet).  ``act``
     is ``x`` in the compute dtype where a block has made that copy (blocks whose
     sublayers read the stream itself), else None."""
 
@@ -254,6 +256,8 @@ class Hidden:
         """The stream with everything added; with ``act_dtype`` its copy in that type is
         made on the way and left in ``act``."""
         from .. import ops
+        if isinstance(self.pending, ops.ExpertSum):
+            self.pending = self.pending.sums()
         if self.pending is not None and (self.scale is not None or self.rms is not None or act_dtype is not None):
             self.act = ops.stream_update(self.x, self.pending, scale=self.scale, rms=self.rms, out_dtype=act_dtype)
             self.defer(None)

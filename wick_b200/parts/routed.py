@@ -164,6 +164,7 @@ class RoutedMoE(FeedForward):
     def forward(self, x, batch, beside=None):
         if beside is not None and self.shared is not None:           # (the kernel takes one term beside the experts)
             return ops.weighted_sum([(beside, 1.0), (self.forward(x, batch), 1.0)])
+        defer = beside is not None and not self.identity             # (the sum is left to whoever reads the stream next)
         n = x.shape[0]
         logits = self.router.forward_delta(x)                        # float32 [splits, n, outputs (+ 1: the shared expert's gate)]
         choice, weight, ident = ops.moe_router(logits, self.correction, self.top, renormalize=self.renormalize, scores=self.scores,
@@ -176,12 +177,14 @@ class RoutedMoE(FeedForward):
             if self.has_shared_gate:
                 base_gate = logits                                  # (its last column)
         if self.up_tiles is not None and n >= self.SORTED_FROM:
-            return self._forward_sorted(x, choice, weight, ident, own, base, base_gate)
+            return self._forward_sorted(x, choice, weight, ident, own, base, base_gate, defer)
         hidden = ops.moe_table_up(x, ident, choice, self.gate_up)   # [n, top, ff]; pairs of outputs without matrices are passed over
         y = ops.moe_expert_down(hidden, ident, choice, self.down)
+        if defer:
+            return ops.ExpertSum(y, None, choice, weight, self.experts, base)
         return ops.moe_combine_weighted(y, None, choice, weight, own, self.experts, base, base_gate, self.outputs).unsqueeze(0)
 
-    def _forward_sorted(self, x, choice, weight, ident, own, base=None, base_gate=None):
+    def _forward_sorted(self, x, choice, weight, ident, own, base=None, base_gate=None, defer=False):
         from ..ops import gemm_tc
         n, dt, pad = x.shape[0], self.ctx.dtype, self.ROW_TILE
         counts, row_of, tiles = ops.moe_route(ident, choice, self.experts, pad=pad)
@@ -198,6 +201,8 @@ class RoutedMoE(FeedForward):
             gemm_tc.gemm_tc_pair(xs, self.up_tiles, f, out=hidden, ldo=f, b_packed=True, groups=tiles, group_rows=f_pad)
             ops.relu_squared_(hidden)
         gemm_tc.gemm_tc_pair(hidden, self.down_tiles, w, out=y, ldo=w, b_packed=True, groups=tiles, group_rows=w_pad)
+        if defer:
+            return ops.ExpertSum(y, row_of, choice, weight, self.experts, base)
         return ops.moe_combine_weighted(y, row_of, choice, weight, own, self.experts, base, base_gate, self.outputs).unsqueeze(0)
 
 

@@ -109,6 +109,11 @@ class RMSNorm(Norm):
         return ops.rmsnorm(x, self.weight, self.eps, out_dtype, rows=rows)
 
     def add_forward(self, x, delta, out_dtype, rows=None, *, scale=None, rms=None):
+        if isinstance(delta, ops.ExpertSum):
+            factor = 1.0 if scale is None else getattr(scale, "one_number", None)
+            if rms is None and factor is not None and delta.joins_norm():
+                return ops.moe_experts_norm(x, delta, factor, self.weight, self.eps, out_dtype, rows)
+            delta = delta.sums()
         if scale is not None or rms is not None:              # (the stream's own kernel: the sum's factor or norm, then this norm)
             return ops.stream_update(x, delta, scale=scale, rms=rms, norm=("rms", self.weight, self.eps),
                                      out_dtype=out_dtype, rows=rows)
@@ -179,6 +184,8 @@ class TanhNorm(Norm):
         return ops.stream_update(x, None, norm=self._norm(), out_dtype=out_dtype, rows=rows)
 
     def add_forward(self, x, delta, out_dtype, rows=None, *, scale=None, rms=None):
+        if isinstance(delta, ops.ExpertSum):
+            delta = delta.sums()
         return ops.stream_update(x, delta, scale=scale, rms=rms, norm=self._norm(), out_dtype=out_dtype, rows=rows)
 
     def weight_bytes(self):
@@ -564,7 +571,10 @@ class ParallelResidual(Block):
         if not isinstance(ffn_norm, NoNorm):
             raise ValueError("sublayers side by side share one norm: the second one is of kind 'none'")
         factor = float(params.get("factor", 1.0))
-        self.scale = None if factor == 1.0 else torch.full((int(params["width"]),), factor, dtype=torch.float32, device=ctx.device)
+        self.scale = None
+        if factor != 1.0:
+            self.scale = torch.full((int(params["width"]),), factor, dtype=torch.float32, device=ctx.device)
+            self.scale.one_number = factor           # (for a kernel that takes the factor as a number)
 
     def forward(self, h, batch, cache, write_cache):
         dt = self.ctx.dtype
@@ -579,7 +589,8 @@ class ParallelResidual(Block):
         d = as_splits(self.mixer.forward(xn, batch, cache, write_cache))
         if not getattr(self.ffn, "IS_NONE", False):
             if getattr(self.ffn, "JOINS_BESIDE", False):
-                d = as_splits(self.ffn.forward(xn, batch, beside=d))
+                d = self.ffn.forward(xn, batch, beside=d)
+                d = d if isinstance(d, ops.ExpertSum) else as_splits(d)
             else:
                 d = ops.weighted_sum([(d, 1.0), (as_splits(self.ffn.forward(xn, batch)), 1.0)])
         h.defer(d, self.scale)
