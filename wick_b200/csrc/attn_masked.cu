@@ -330,8 +330,8 @@ qkv_finish_kernel(const float* __restrict__ parts, int splits, int64_t split_str
 // The blocks of `block` positions that a step completes: their mean keys and values go to the store (as above), and, with
 // `flat`, so do all blocks the sequences' tokens can see to arrays whose tiles of 64 blocks lie like cache pages: tile i of sequence b is
 // page b * flat_tiles + i of [G][64][d] keys, then [G][64][e] values (places beyond a sequence's whole blocks hold zeros).
-// grid (most blocks of a sequence, sequences).
-template <typename T>
+// grid (most blocks of a sequence, sequences).  VEC: a thread takes 16 bytes of neighbours at a time.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 pool_blocks_kernel(const T* __restrict__ kv, T* store, T* __restrict__ flat, const int* __restrict__ page_table, int table_width,
                    const int* __restrict__ start, const int* __restrict__ kv_len, int G, int d, int e, int block, int rows,
@@ -348,6 +348,35 @@ pool_blocks_kernel(const T* __restrict__ kv, T* store, T* __restrict__ flat, con
     T* dst = whole ? store + table[pg] * pool_page : nullptr;
     T* out = flat ? flat + (int64_t)(b * flat_tiles + blk / kPage) * W * kPage : nullptr;
     const int at = block_place(blk, block, pg);
+    if (VEC) {
+        constexpr int VN = Vec16<T>::N;
+        for (int c = threadIdx.x * VN; c < W; c += blockDim.x * VN) {
+            const bool key = c < Wk;
+            const int size = key ? d : e, i = key ? c : c - Wk, g = i / size, x = i - g * size;
+            T* s = whole ? dst + (key ? 0 : (int64_t)G * rows * d) + ((int64_t)g * rows + at) * size + x : nullptr;
+            Vec16<T> m;
+#pragma unroll
+            for (int k = 0; k < VN; ++k) m.v[k] = 0.f;
+            if (whole && !old) {
+                const T* from = kv + (key ? 0 : (int64_t)G * kPage * d) + (int64_t)g * kPage * size + x;
+#pragma unroll 8
+                for (int j = 0; j < block; ++j) {
+                    const int p = blk * block + j;
+                    Vec16<T> u;
+                    u.load(from + table[p / kPage] * (int64_t)W * kPage + (int64_t)(p % kPage) * size);
+#pragma unroll
+                    for (int k = 0; k < VN; ++k) m.v[k] += u.v[k];
+                }
+#pragma unroll
+                for (int k = 0; k < VN; ++k) m.v[k] /= (float)block;
+                m.store(s);
+            } else if (whole) {
+                m.load(s);
+            }
+            if (out) m.store(out + (key ? 0 : (int64_t)G * kPage * d) + ((int64_t)g * kPage + blk % kPage) * size + x);
+        }
+        return;
+    }
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
         const bool key = c < Wk;
         const int size = key ? d : e, i = key ? c : c - Wk, g = i / size, x = i - g * size;
@@ -808,7 +837,9 @@ WICK_ATTN_MASKED(wick_attn_masked_f32, float)
                      pool_page == (int64_t)G * rows * (d + e), "pool_blocks: bad sizes");                                      \
         WICK_REQUIRE(n_seqs <= 65535 && (!flat || blocks == flat_tiles * kPage), "pool_blocks: bad numbers of blocks");        \
         if (n_seqs == 0 || blocks == 0) return 0;                                                                              \
-        WICK_CUDA(launch(pool_blocks_kernel<T>, dim3(blocks, n_seqs), dim3(256), 0, (cudaStream_t)s, (const T*)kv, (T*)store, (T*)flat, \
+        const bool vec = d % Vec16<T>::N == 0 && e % Vec16<T>::N == 0 && (((uintptr_t)kv | (uintptr_t)store | (uintptr_t)flat) & 15) == 0; \
+        const int per = vec ? G * (d + e) / Vec16<T>::N : G * (d + e), threads = per >= 256 ? 256 : (per + 31) / 32 * 32;       \
+        WICK_CUDA(launch(vec ? pool_blocks_kernel<T, true> : pool_blocks_kernel<T, false>, dim3(blocks, n_seqs), dim3(threads), 0, (cudaStream_t)s, (const T*)kv, (T*)store, (T*)flat, \
                          page_table, table_width, start, kv_len, G, d, e, block, rows, pool_page, flat_tiles));                 \
         return check_launch("pool_blocks");                                                                                    \
     }
